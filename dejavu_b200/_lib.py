@@ -1,6 +1,7 @@
-"""ctypes binding of libdejavu_b200.so (declared in include/dejavu_b200.h).
+"""ctypes binding of libdejavu_b200.so (declared in include/dejavu_b200.h) and libdejavu_b200_hybrid.so
+(include/dejavu_b200_hybrid.h).
 
-The library is the only compute path of this package: if it is missing the import of any operator
+The libraries are the only compute path of this package: if one is missing the import of any operator
 raises, there is no PyTorch or CPU fallback.
 """
 from __future__ import annotations
@@ -10,9 +11,11 @@ from pathlib import Path
 
 PKG = Path(__file__).resolve().parent
 LIB_PATH = PKG / "libdejavu_b200.so"
+HYBRID_LIB_PATH = PKG / "libdejavu_b200_hybrid.so"
 
 OK, ERR_INVALID, ERR_UNSUPPORTED, ERR_CUDA, ERR_SCRATCH, ERR_TIMEOUT = 0, -1, -2, -3, -4, -5
-ACT = {"id": 0, "relu": 1, "gelu": 2, "gelu_approx": 3, "squared_relu": 4}
+ACT = {"id": 0, "relu": 1, "gelu": 2, "gelu_approx": 3, "squared_relu": 4, "softcap": 5, "clamped_glu": 6}
+DTYPE_F16, DTYPE_BF16, DTYPE_F32 = 0, 1, 2
 MAX_BATCH = 32
 KV_WINDOW = 16
 EXCHANGE_REFILL = 1
@@ -85,36 +88,72 @@ SIGNATURES = {
     "djv_allreduce_add_layernorm": (_i, [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _vp]),
 }
 
+# functions every library has (each keeps its own error message, launch counter and launch mode)
+_PLUMBING = ("djv_version", "djv_last_error", "djv_status_string", "djv_launch_count", "djv_set_early_weight_prefetch",
+             "djv_set_programmatic_launch")
+
+# mirrors include/dejavu_b200_hybrid.h one to one
+HYBRID_SIGNATURES = {
+    "djv_hyper_step": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _i, _i, _i, _i, _vp]),
+    "djv_dense_gemv": (_i, [_i, _i, _vp, _vp, _vp, _i, _i, _i, _ll, _i, _f, _vp]),
+    "djv_clamped_glu": (_i, [_i, _vp, _vp, _ll, _i, _f, _vp]),
+    "djv_softcap": (_i, [_vp, _ll, _f, _vp]),
+    "djv_rotary": (_i, [_i, _vp, _ll, _vp, _f, _vp, _i, _i, _i, _i, _i, _vp]),
+    "djv_window_attn": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp]),
+    "djv_window_store": (_i, [_i, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
+    "djv_window_attn_decode": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _f, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _f,
+                                    _vp]),
+    "djv_gla_scratch_bytes": (_sz, [_i, _i, _i, _i, _i, _i]),
+    "djv_gla_prefill": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _i, _f, _vp, _f, _f, _vp, _vp, _i, _i, _i, _i, _i, _vp, _sz,
+                             _vp]),
+    "djv_gla_decode": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _i, _f, _vp, _f, _f, _vp, _vp, _i, _i, _i, _i, _vp]),
+}
+
 _lib = None
+_hybrid = None
+
+
+def _open(path, signatures) -> C.CDLL:
+    if not path.exists():
+        raise ImportError(
+            f"{path} is missing: build it with `python -m dejavu_b200.build` "
+            "(there is no fallback path)"
+        )
+    lib = C.CDLL(str(path))
+    for name, (res, args) in signatures.items():
+        fn = getattr(lib, name)
+        fn.restype = res
+        fn.argtypes = args
+    return lib
 
 
 def load() -> C.CDLL:
-    """Loads the shared library (once). Raises if it has not been built."""
+    """Loads the sparse path's shared library (once). Raises if it has not been built."""
     global _lib
     if _lib is None:
-        if not LIB_PATH.exists():
-            raise ImportError(
-                f"{LIB_PATH} is missing: build it with `python -m dejavu_b200.build` "
-                "(there is no fallback path)"
-            )
-        lib = C.CDLL(str(LIB_PATH))
-        for name, (res, args) in SIGNATURES.items():
-            fn = getattr(lib, name)
-            fn.restype = res
-            fn.argtypes = args
-        _lib = lib
+        _lib = _open(LIB_PATH, SIGNATURES)
     return _lib
 
 
-def check(fn_name: str, status: int) -> None:
+def load_hybrid() -> C.CDLL:
+    """Loads the hybrid decoders' shared library (once). Raises if it has not been built."""
+    global _hybrid
+    if _hybrid is None:
+        _hybrid = _open(HYBRID_LIB_PATH, {**HYBRID_SIGNATURES, **{n: SIGNATURES[n] for n in _PLUMBING}})
+    return _hybrid
+
+
+def check(fn_name: str, status: int, lib=None) -> None:
     if status != OK:
-        msg = load().djv_last_error().decode(errors="replace")
+        msg = (lib or load()).djv_last_error().decode(errors="replace")
         raise DejavuKernelError(fn_name, status, msg)
 
 
 def call(fn_name: str, *args) -> None:
-    check(fn_name, getattr(load(), fn_name)(*args))
+    lib = load_hybrid() if fn_name in HYBRID_SIGNATURES else load()
+    check(fn_name, getattr(lib, fn_name)(*args), lib)
 
 
 def launch_count() -> int:
-    return int(load().djv_launch_count())
+    """Kernels launched by the loaded libraries since load."""
+    return sum(int(lib.djv_launch_count()) for lib in (_lib, _hybrid) if lib is not None)

@@ -1,9 +1,13 @@
-"""Builds libdejavu_b200.so (the C-ABI library of sm_100a kernels) in-tree with nvcc.
+"""Builds the C-ABI libraries of sm_100a kernels in-tree with nvcc.
 
-    python -m dejavu_b200.build [--force] [--verbose]
+    python -m dejavu_b200.build [--force] [--verbose] [--lib sparse|hybrid]
 
-Each .cu file is compiled to an object in parallel, then linked into one shared library that sits
-next to this file. Nothing is cached outside the package directory.
+  sparse  libdejavu_b200.so         the contextual-sparse OPT decode path
+  hybrid  libdejavu_b200_hybrid.so  gated linear attention, sliding-window attention, hyper-connected streams
+
+Each .cu file is compiled to an object in parallel, then linked into the shared libraries that sit next to this file.
+Nothing is cached outside the package directory. A library can be built alone, so that a program that serves one kind
+of model compiles only what it needs.
 """
 from __future__ import annotations
 
@@ -19,6 +23,8 @@ PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 OBJ = PKG / "build"
 LIB = PKG / "libdejavu_b200.so"
+HYBRID_LIB = PKG / "libdejavu_b200_hybrid.so"
+LIBS = {"sparse": LIB, "hybrid": HYBRID_LIB}
 
 NVCC_FLAGS = [
     "-O3",
@@ -38,8 +44,12 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found; set NVCC=/path/to/nvcc")
 
 
-def sources() -> list[Path]:
-    return sorted(CSRC.glob("*.cu"))
+def sources(lib: str | None = None) -> list[Path]:
+    """Translation units of a library (of all, without a name). api.cu, the plumbing, is part of both."""
+    out = sorted(CSRC.glob("*.cu"))
+    if lib is None:
+        return out
+    return [p for p in out if p.stem == "api" or p.stem.startswith("hybrid_") == (lib == "hybrid")]
 
 
 def _stale(target: Path, deps: list[Path]) -> bool:
@@ -49,15 +59,17 @@ def _stale(target: Path, deps: list[Path]) -> bool:
     return any(d.stat().st_mtime > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """DJV_NVCC_FLAGS in the environment adds flags (e.g. -DDJV_RING_TRACE for the phase stamps of the one-pass
-    MLP kernel; use --force, the flag is not part of the staleness check)."""
+def build(force: bool = False, verbose: bool = False, libs: tuple[str, ...] = ("sparse", "hybrid")) -> Path:
+    """Compiles what is stale of the named libraries and returns the path of the first one. DJV_NVCC_FLAGS in the
+    environment adds flags (e.g. -DDJV_RING_TRACE for the phase stamps of the one-pass MLP kernel; use --force, the
+    flag is not part of the staleness check)."""
     nvcc = _nvcc()
     extra = os.environ.get("DJV_NVCC_FLAGS", "").split()
     OBJ.mkdir(exist_ok=True)
-    headers = sorted(CSRC.glob("*.cuh")) + [PKG.parent / "include" / "dejavu_b200.h"]
+    headers = sorted(CSRC.glob("*.cuh")) + sorted((PKG.parent / "include").glob("*.h"))
+    wanted = sorted({src for lib in libs for src in sources(lib)})
     jobs = []
-    for src in sources():
+    for src in wanted:
         obj = OBJ / (src.stem + ".o")
         if force or _stale(obj, [src] + headers):
             cmd = [nvcc, *NVCC_FLAGS, *extra, "-c", str(src), "-o", str(obj)]
@@ -76,19 +88,26 @@ def build(force: bool = False, verbose: bool = False) -> Path:
                 sys.stderr.write(" ".join(cmd) + "\n" + r.stdout + r.stderr)
             if r.returncode != 0:
                 raise RuntimeError(f"nvcc failed on {cmd[-3]}")
-    objs = [OBJ / (s.stem + ".o") for s in sources()]
-    if force or jobs or _stale(LIB, objs):
-        cmd = [nvcc, "-shared", "-o", str(LIB), *map(str, objs), "-Xcompiler", "-fPIC", "-lcudart"]
-        r = subprocess.run(cmd, capture_output=True, text=True)
-        if r.returncode != 0:
-            sys.stderr.write(r.stdout + r.stderr)
-            raise RuntimeError("link failed")
-    return LIB
+    for lib in libs:
+        objs = [OBJ / (s.stem + ".o") for s in sources(lib)]
+        if force or _stale(LIBS[lib], objs):
+            part = LIBS[lib].with_suffix(f".{os.getpid()}.tmp")
+            cmd = [nvcc, "-shared", "-o", str(part), *map(str, objs), "-Xcompiler", "-fPIC", "-lcudart"]
+            r = subprocess.run(cmd, capture_output=True, text=True)
+            if r.returncode != 0:
+                sys.stderr.write(r.stdout + r.stderr)
+                raise RuntimeError("link failed")
+            os.replace(part, LIBS[lib])
+    return LIBS[libs[0]]
 
 
 if __name__ == "__main__":
     ap = argparse.ArgumentParser()
     ap.add_argument("--force", action="store_true")
     ap.add_argument("--verbose", action="store_true", help="print ptxas register / shared-memory usage")
+    ap.add_argument("--lib", choices=sorted(LIBS), help="build this library only")
     a = ap.parse_args()
-    print(build(force=a.force, verbose=a.verbose))
+    names = (a.lib,) if a.lib else ("sparse", "hybrid")
+    build(force=a.force, verbose=a.verbose, libs=names)
+    for name in names:
+        print(LIBS[name])

@@ -13,7 +13,9 @@ the glob patterns of Decentralized_FM_alpha/modules/hf_opt_sparse_mlp_attention.
 from __future__ import annotations
 
 import glob
+import json
 import math
+import mmap
 import os
 import re
 from collections import OrderedDict
@@ -31,6 +33,51 @@ _RENAMES = [
     (r"^transformer\.layers\.(\d+)\.fc(1|2)\.", r"transformer.layers.\1.mlp.fc\2."),
     (r"^transformer\.layers\.(\d+)\.self_attn\.out_proj\.", r"transformer.layers.\1.mixer.out_proj."),
 ]
+
+
+_SAFETENSORS_DTYPES = {"BF16": torch.bfloat16, "F16": torch.float16, "F32": torch.float32, "F64": torch.float64,
+                       "I8": torch.int8, "U8": torch.uint8, "I16": torch.int16, "I32": torch.int32,
+                       "I64": torch.int64, "BOOL": torch.bool}
+
+
+def read_safetensors(path: str) -> dict:
+    """name -> CPU tensor of a .safetensors file: an 8-byte little-endian length, that many bytes of JSON (name ->
+    dtype, shape, data_offsets from the end of the JSON), then the data."""
+    with open(path, "rb") as f:
+        size = os.fstat(f.fileno()).st_size
+        if size < 8:
+            raise ValueError(f"{path}: too short for a safetensors file")
+        data = mmap.mmap(f.fileno(), 0, access=mmap.ACCESS_COPY)
+    n = int.from_bytes(data[:8], "little")
+    if n > size - 8:
+        raise ValueError(f"{path}: header of {n} bytes in a file of {size}")
+    header = json.loads(data[8:8 + n])
+    out = {}
+    for name, info in header.items():
+        if name == "__metadata__":
+            continue
+        dtype, shape = _SAFETENSORS_DTYPES[info["dtype"]], tuple(info["shape"])
+        begin, end = info["data_offsets"]
+        count = math.prod(shape)
+        if begin < 0 or 8 + n + end > size or end - begin != count * torch.empty(0, dtype=dtype).element_size():
+            raise ValueError(f"{path}: {name} has {end - begin} bytes for shape {shape}")
+        if count == 0:
+            out[name] = torch.empty(shape, dtype=dtype)
+        else:
+            out[name] = torch.frombuffer(data, dtype=torch.uint8, count=end - begin,
+                                         offset=8 + n + begin).clone().view(dtype).view(shape)
+    return out
+
+
+def read_model_tensors(folder: str) -> dict:
+    """All tensors of a model folder (model.safetensors, or the shards beside it)."""
+    files = sorted(glob.glob(os.path.join(folder, "*.safetensors")))
+    if not files:
+        raise FileNotFoundError(f"no .safetensors file in {folder}")
+    out = {}
+    for f in files:
+        out.update(read_safetensors(f))
+    return out
 
 
 def _padded_vocab(config, world_size: int = 1) -> int:

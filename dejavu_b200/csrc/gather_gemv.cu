@@ -10,6 +10,7 @@
 //   rowdot  : M*N*2 + M*2 (bias) + M*4 (idx) + B*N*2 (x) + B*M*2 (y)
 //   rowaxpy : M*N*2 + B*M*2 (x) + N*2 (bias) + B*N*2 (y)
 #include "common.cuh"
+#include "rowdot.cuh"
 #include "rowaxpy.cuh"
 #include "rowdot_mma.cuh"
 #include "rowaxpy_mma.cuh"
@@ -26,173 +27,13 @@ int ring_fc2(__half *y, const __half *w, const __half *h, const void *idx, const
 static int ring_gemv_rows() { return env_int("DJV_RING_GEMV", 0); }
 static bool ring_shape_ok(int B, int N, int M) { return djv_mlp_sparse_fused_supported(B, N, M) != 0; }
 
-// -------------------------------------------------------------------------------------------
-// rowdot. A block has 8 warps split into 8/WPR groups of WPR warps; a group owns ROWS rows at a
-// time and its 32*WPR lanes stride over the 16-byte chunks of those rows, U chunks in flight per
-// lane per row. x is read through L1 (it is tiny and reused by every warp); weights bypass L1.
-// Small M uses large WPR so that the whole device has loads in flight for a handful of rows.
-// -------------------------------------------------------------------------------------------
-constexpr int RD_THREADS = 256;
-constexpr int RD_WARPS = RD_THREADS / WARP;
-
-template <int B, int ACT, int WPR, int ROWS, int U>
-__global__ void __launch_bounds__(RD_THREADS)
-rowdot_kernel(__half *__restrict__ Y, const __half *__restrict__ W, const __half *__restrict__ X,
-              const void *__restrict__ idx, const __half *__restrict__ bias, int M, int N,
-              long long ldw, int idx64, int early) {
-  constexpr int GROUPS = RD_WARPS / WPR;
-  constexpr int GLANES = WARP * WPR;
-  __shared__ float red[WPR > 1 ? RD_WARPS * ROWS * B : 1];
-
-  const int tid = threadIdx.x;
-  const int warp = tid / WARP, lane = tid % WARP;
-  const int group = warp / WPR, wig = warp % WPR;
-  const int glane = wig * WARP + lane;
-  const int nchunks = N / 8;
-  const uint4 *Xv = reinterpret_cast<const uint4 *>(X);
-
-  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  if (early) {
-    // Weights are not produced by any kernel, and the index list is complete (identity, or the caller's
-    // promise): the first 8 KB of the first rows of this group are requested while the kernel before this
-    // one is still running.
-    const int m0 = blockIdx.x * GROUPS * ROWS + group * ROWS;
-    constexpr int LINES = 64;
-    const int row_lines = (int)min((long long)LINES, ((long long)N * 2 + 127) / 128);
-#pragma unroll
-    for (int j = 0; j < ROWS; ++j) {
-      if (m0 + j < M) {
-        const long long r = load_index(idx, m0 + j, idx64);
-        const char *w0 = reinterpret_cast<const char *>(W + r * ldw);
-        for (int l = glane; l < row_lines; l += GLANES) prefetch_l2(w0 + (size_t)l * 128);
-      }
-    }
-  }
-  asm volatile("griddepcontrol.wait;" ::: "memory");
-
-  const int rows_per_pass = gridDim.x * GROUPS * ROWS;
-  // trip count is uniform over the block so that __syncthreads below is legal
-  for (int base = blockIdx.x * GROUPS * ROWS; base < M; base += rows_per_pass) {
-    const int m0 = base + group * ROWS;
-    const uint4 *wp[ROWS];
-    float bv[ROWS];
-#pragma unroll
-    for (int j = 0; j < ROWS; ++j) {
-      const int m = m0 + j;
-      const bool ok = m < M;
-      const long long r = ok ? load_index(idx, m, idx64) : 0;
-      wp[j] = reinterpret_cast<const uint4 *>(W + r * ldw);
-      bv[j] = (bias != nullptr && ok) ? __half2float(bias[r]) : 0.f;
-      if (!ok) wp[j] = nullptr;
-    }
-    float acc[ROWS][B];
-#pragma unroll
-    for (int j = 0; j < ROWS; ++j)
-#pragma unroll
-      for (int b = 0; b < B; ++b) acc[j][b] = 0.f;
-
-    for (int c0 = glane; c0 < nchunks; c0 += GLANES * U) {
-      uint4 wv[ROWS][U];
-#pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const int c = c0 + u * GLANES;
-#pragma unroll
-        for (int j = 0; j < ROWS; ++j) {
-          if (c < nchunks && wp[j] != nullptr)
-            wv[j][u] = ld_stream16(wp[j] + c);
-          else
-            wv[j][u] = make_uint4(0, 0, 0, 0);
-        }
-      }
-#pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const int c = c0 + u * GLANES;
-        if (c < nchunks) {
-#pragma unroll
-          for (int b = 0; b < B; ++b) {
-            const uint4 xv = ld_cached16(Xv + (size_t)b * nchunks + c);
-#pragma unroll
-            for (int j = 0; j < ROWS; ++j) acc[j][b] = dot8(wv[j][u], xv, acc[j][b]);
-          }
-        }
-      }
-    }
-#pragma unroll
-    for (int j = 0; j < ROWS; ++j)
-#pragma unroll
-      for (int b = 0; b < B; ++b) acc[j][b] = warp_sum(acc[j][b]);
-
-    if (WPR > 1) {
-      if (lane == 0) {
-#pragma unroll
-        for (int j = 0; j < ROWS; ++j)
-#pragma unroll
-          for (int b = 0; b < B; ++b) red[(warp * ROWS + j) * B + b] = acc[j][b];
-      }
-      __syncthreads();
-      if (wig == 0 && lane == 0) {
-#pragma unroll
-        for (int j = 0; j < ROWS; ++j)
-#pragma unroll
-          for (int b = 0; b < B; ++b) {
-            float s = 0.f;
-#pragma unroll
-            for (int w2 = 0; w2 < WPR; ++w2) s += red[((group * WPR + w2) * ROWS + j) * B + b];
-            acc[j][b] = s;
-          }
-      }
-    }
-    if (wig == 0 && lane == 0) {
-#pragma unroll
-      for (int j = 0; j < ROWS; ++j) {
-        const int m = m0 + j;
-        if (m < M) {
-#pragma unroll
-          for (int b = 0; b < B; ++b)
-            Y[(size_t)b * M + m] = __float2half_rn(apply_act<ACT>(acc[j][b] + bv[j]));
-        }
-      }
-    }
-    if (WPR > 1) __syncthreads();  // red[] is reused by the next pass
-  }
-}
-
-struct RowdotPlan {
-  int wpr, rows, grid;
-};
-
-static RowdotPlan plan_rowdot(int M, int N, int B) {
-  const int sms = sm_count();
-  const int nchunks = N / 8;
-  const int rows = (B <= 2) ? 2 : 1;
-  static const int k_wpr = env_int("DJV_RD_WPR", 0);  // development knobs
-  static const int k_cap = env_int("DJV_RD_BLOCKS_PER_SM", 6);
-  // As many warps per row as still lets every block be resident at once (4 blocks of 256 threads per SM):
-  // a second, partial wave of blocks costs more than fewer lanes per row (measured: K=4096, d=9216 runs at
-  // 0.77 of the HBM peak with 2 warps per row, 0.71 with 4, 0.67 with 1).
-  const long long resident = (long long)sms * 4;
-  int wpr = 1;
-  while (wpr < 8 && (long long)ceil_div(M, (RD_WARPS / (wpr * 2)) * rows) <= resident && nchunks >= 64 * wpr * 2)
-    wpr *= 2;
-  if (k_wpr > 0) {
-    wpr = k_wpr;
-    while (wpr > 1 && nchunks < 32 * wpr) wpr /= 2;
-  }
-  const int groups = RD_WARPS / wpr;
-  int grid = ceil_div(M, groups * rows);
-  const int cap = sms * k_cap;
-  if (grid > cap) grid = cap;
-  if (grid < 1) grid = 1;
-  return {wpr, rows, grid};
-}
-
 template <int B, int ACT>
 static void launch_rowdot(const RowdotPlan &p, __half *Y, const __half *W, const __half *X,
                           const void *idx, const __half *bias, int M, int N, long long ldw,
                           int idx64, cudaStream_t st) {
 #define DJV_RD(WPR_, ROWS_)                                                               \
-  djv::launch_kernel(rowdot_kernel<B, ACT, WPR_, ROWS_, 4>, p.grid, RD_THREADS, 0, st, Y, W, X, idx, bias, M, N, \
-                     ldw, idx64, (idx == nullptr || early_prefetch()) ? 1 : 0)
+  djv::launch_kernel(rowdot_kernel<__half, __half, B, ACT, WPR_, ROWS_, 4>, p.grid, RD_THREADS, 0, st, Y, W, X, idx, bias, M, N, \
+                     ldw, idx64, (idx == nullptr || early_prefetch()) ? 1 : 0, 0.f)
   constexpr int R = (B <= 2) ? 2 : 1;
   switch (p.wpr) {
     case 1: DJV_RD(1, R); break;
@@ -226,7 +67,7 @@ static int dispatch_act(const RowdotPlan &p, int act, __half *Y, const __half *W
 // (each slice re-reads the gathered rows).
 static int rowdot_slice(int B, int act, __half *Y, const __half *W, const __half *X, const void *idx,
                         const __half *bias, int M, int N, long long ldw, int idx64, cudaStream_t st) {
-  const RowdotPlan p = plan_rowdot(M, N, B);
+  const RowdotPlan p = plan_rowdot(M, N / 8, B, B <= 2 ? 2 : 1);
   switch (B) {
     case 1: return dispatch_act<1>(p, act, Y, W, X, idx, bias, M, N, ldw, idx64, st);
     case 2: return dispatch_act<2>(p, act, Y, W, X, idx, bias, M, N, ldw, idx64, st);
@@ -238,6 +79,49 @@ static int rowdot_slice(int B, int act, __half *Y, const __half *W, const __half
     case 8: return dispatch_act<8>(p, act, Y, W, X, idx, bias, M, N, ldw, idx64, st);
   }
   set_error("gather_gemv: internal batch slice %d", B);
+  return DJV_ERR_INVALID;
+}
+
+template <int NT>
+static int launch_rowdot_mma(int act, __half *Y, const __half *W, const __half *X, const void *idx,
+                             const __half *bias, int M, int N, long long ldw, int idx64, int B, cudaStream_t st) {
+  static const int bps = [] {
+    int n = 0;
+    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, rowdot_mma_kernel<__half, __half, NT, DJV_ACT_RELU>,
+                                                      MM_THREADS, 0) != cudaSuccess) {
+      cudaGetLastError();
+      n = 1;
+    }
+    return n < 1 ? 1 : n;
+  }();
+  const int tiles = ceil_div(M, MM_ROWS);
+  const int S = rowdot_mma_split(M, N, NT, bps);
+  const dim3 grid(tiles, S), cluster(1, S, 1);
+#define DJV_MM(ACT_)                                                                                          \
+  djv::launch_kernel_cluster(rowdot_mma_kernel<__half, __half, NT, ACT_>, grid, dim3(MM_THREADS), 0, st, cluster, \
+                             Y, W, X, idx, bias, M, N, ldw, idx64, B, 0.f)
+  switch (act) {
+    case DJV_ACT_ID: DJV_MM(DJV_ACT_ID); break;
+    case DJV_ACT_RELU: DJV_MM(DJV_ACT_RELU); break;
+    case DJV_ACT_GELU: DJV_MM(DJV_ACT_GELU); break;
+    case DJV_ACT_GELU_APPROX: DJV_MM(DJV_ACT_GELU_APPROX); break;
+    case DJV_ACT_SQUARED_RELU: DJV_MM(DJV_ACT_SQUARED_RELU); break;
+    default: set_error("gather_gemv: unknown activation %d", act); return DJV_ERR_INVALID;
+  }
+#undef DJV_MM
+  return DJV_OK;
+}
+
+// 9 <= B <= 32
+static int rowdot_mma(int B, int act, __half *Y, const __half *W, const __half *X, const void *idx,
+                      const __half *bias, int M, int N, long long ldw, int idx64, cudaStream_t st) {
+  switch ((B + 7) / 8) {
+    case 1: return launch_rowdot_mma<1>(act, Y, W, X, idx, bias, M, N, ldw, idx64, B, st);
+    case 2: return launch_rowdot_mma<2>(act, Y, W, X, idx, bias, M, N, ldw, idx64, B, st);
+    case 3: return launch_rowdot_mma<3>(act, Y, W, X, idx, bias, M, N, ldw, idx64, B, st);
+    case 4: return launch_rowdot_mma<4>(act, Y, W, X, idx, bias, M, N, ldw, idx64, B, st);
+  }
+  set_error("gather_gemv: batch %d outside the tensor-core kernel's range", B);
   return DJV_ERR_INVALID;
 }
 

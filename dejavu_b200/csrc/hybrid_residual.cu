@@ -1,0 +1,222 @@
+// The boundary between two sublayers of a decoder with hyper-connected residual streams: stream update from the
+// previous sublayer's output, weighted sum of the streams, RMS norm. One block per row; every stream element is read
+// and written once. Bytes per row: S*D*4 read + S*D*4 written + D*4 (y) + D*sizeof(T) (h).
+// Also the two small elementwise kernels of the prompt pass (clamped gated unit, logit softcap).
+#include "../../include/dejavu_b200_hybrid.h"
+#include "dtype.cuh"
+#include "rowdot.cuh"
+
+namespace djv {
+
+constexpr int HS_THREADS = 512;
+
+struct HyperArgs {
+  void *h;
+  float *x_out;
+  const float *x_in, *y, *mix, *w_out, *w_in, *gamma;
+  float eps;
+  const int *row_list;
+  const long long *ids;
+  const void *embed;
+  int D, vocab;
+};
+
+template <typename T, int S, int V>  // V columns at a time: 4 (16-byte accesses) or 1
+__global__ void __launch_bounds__(HS_THREADS) hyper_step_kernel(HyperArgs a) {
+  extern __shared__ float u_s[];  // D
+  __shared__ float coef[S * S + 2 * S];
+  __shared__ float red[HS_THREADS / WARP];
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  const int tid = threadIdx.x;
+  // the coefficients are weights: no kernel of the step writes them
+  if (tid < S * S) coef[tid] = a.y ? a.mix[tid] : (tid / S == tid % S ? 1.f : 0.f);
+  if (tid >= 64 && tid < 64 + S) coef[S * S + tid - 64] = a.y ? a.w_out[tid - 64] : 0.f;
+  if (tid >= 96 && tid < 96 + S) coef[S * S + S + tid - 96] = a.w_in ? a.w_in[tid - 96] : 1.f;
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  __syncthreads();
+  const int D = a.D;
+  const int row = a.row_list ? a.row_list[blockIdx.x] : blockIdx.x;
+  const float *x = a.x_in ? a.x_in + (size_t)row * S * D : nullptr;
+  const T *e = nullptr;
+  if (!a.x_in) {
+    const long long id = a.ids[row];
+    e = static_cast<const T *>(a.embed) + (size_t)(id < 0 ? 0 : (id >= a.vocab ? a.vocab - 1 : id)) * D;
+  }
+  float ss = 0.f;
+  for (int c = tid * V; c < D; c += blockDim.x * V) {
+    float xs[S][V], yv[V], u[V];
+    if (x) {
+#pragma unroll
+      for (int s = 0; s < S; ++s) {
+        if (V == 4) {
+          const float4 t = *reinterpret_cast<const float4 *>(x + (size_t)s * D + c);
+          xs[s][0] = t.x; xs[s][1 % V] = t.y; xs[s][2 % V] = t.z; xs[s][3 % V] = t.w;
+        } else {
+          xs[s][0] = x[(size_t)s * D + c];
+        }
+      }
+    } else {
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        const float t = to_f(e[c + v]);
+#pragma unroll
+        for (int s = 0; s < S; ++s) xs[s][v] = t;
+      }
+    }
+#pragma unroll
+    for (int v = 0; v < V; ++v) yv[v] = u[v] = 0.f;
+    if (a.y) {
+      if (V == 4) {
+        const float4 t = *reinterpret_cast<const float4 *>(a.y + (size_t)row * D + c);
+        yv[0] = t.x; yv[1 % V] = t.y; yv[2 % V] = t.z; yv[3 % V] = t.w;
+      } else {
+        yv[0] = a.y[(size_t)row * D + c];
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < S; ++t) {
+      float nv[V];
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        float acc = coef[S * S + t] * yv[v];
+#pragma unroll
+        for (int s = 0; s < S; ++s) acc = fmaf(coef[s * S + t], xs[s][v], acc);
+        nv[v] = acc;
+        u[v] = fmaf(coef[S * S + S + t], acc, u[v]);
+      }
+      if (a.x_out) {
+        float *dst = a.x_out + ((size_t)row * S + t) * D + c;
+        if (V == 4)
+          *reinterpret_cast<float4 *>(dst) = make_float4(nv[0], nv[1 % V], nv[2 % V], nv[3 % V]);
+        else
+          dst[0] = nv[0];
+      }
+    }
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      u_s[c + v] = u[v];
+      ss = fmaf(u[v], u[v], ss);
+    }
+  }
+  if (!a.gamma) return;
+  ss = warp_sum(ss);
+  if (tid % WARP == 0) red[tid / WARP] = ss;
+  __syncthreads();
+  float tot = 0.f;
+  for (int w = 0; w < blockDim.x / WARP; ++w) tot += red[w];
+  const float rstd = 1.f / sqrtf(tot / (float)D + a.eps);
+  T *h = static_cast<T *>(a.h) + (size_t)blockIdx.x * D;
+  for (int c = tid * V; c < D; c += blockDim.x * V) {  // the same columns this thread wrote into u_s
+    T o[V];
+#pragma unroll
+    for (int v = 0; v < V; ++v) o[v] = from_f<T>(u_s[c + v] * rstd * a.gamma[c + v]);
+    if (V == 4 && sizeof(T) == 2)
+      *reinterpret_cast<uint2 *>(h + c) = *reinterpret_cast<uint2 *>(o);
+    else if (V == 4)
+      *reinterpret_cast<uint4 *>(h + c) = *reinterpret_cast<uint4 *>(o);
+    else
+      h[c] = o[0];
+  }
+}
+
+template <typename T, int V>
+static int launch_hyper(const HyperArgs &a, int R, int S, cudaStream_t st) {
+  int threads = ceil_div(ceil_div(a.D, V), WARP) * WARP;
+  if (threads > HS_THREADS) threads = HS_THREADS;
+  if (threads < 128) threads = 128;
+  const size_t smem = (size_t)a.D * 4;
+#define DJV_HS(S_)                                                                                      \
+  case S_:                                                                                              \
+    if (smem > 48 * 1024)                                                                               \
+      cudaFuncSetAttribute(hyper_step_kernel<T, S_, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    djv::launch_kernel(hyper_step_kernel<T, S_, V>, R, threads, smem, st, a);                           \
+    break
+  switch (S) {
+    DJV_HS(1);
+    DJV_HS(2);
+    DJV_HS(3);
+    DJV_HS(4);
+    DJV_HS(5);
+    DJV_HS(6);
+    DJV_HS(7);
+    DJV_HS(8);
+  }
+#undef DJV_HS
+  count_launch();
+  return check_launch("hyper_step");
+}
+
+template <typename T>
+__global__ void clamped_glu_kernel(T *__restrict__ y, const T *__restrict__ gu, long long total, float limit) {
+  pdl_prologue();
+  const long long i0 = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i0 >= total) return;
+  if (total - i0 >= 4 && sizeof(T) == 2) {
+    const uint4 v = *reinterpret_cast<const uint4 *>(gu + i0 * 2);
+    float f[8];
+    unpack_chunk<bf16>(v, f);
+    uint2 o;
+    o.x = pack_bf16(clamped_glu(f[0], f[1], limit), clamped_glu(f[2], f[3], limit));
+    o.y = pack_bf16(clamped_glu(f[4], f[5], limit), clamped_glu(f[6], f[7], limit));
+    *reinterpret_cast<uint2 *>(y + i0) = o;
+  } else {
+    for (long long i = i0; i < total && i < i0 + 4; ++i)
+      y[i] = from_f<T>(clamped_glu(to_f(gu[2 * i]), to_f(gu[2 * i + 1]), limit));
+  }
+}
+
+__global__ void softcap_kernel(float *y, long long n, float cap) {
+  pdl_prologue();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) y[i] = cap * tanhf(y[i] / cap);
+}
+
+}  // namespace djv
+
+using namespace djv;
+
+extern "C" int djv_hyper_step(int dtype, void *h, float *x_out, const float *x_in, const float *y, const float *mix,
+                              const float *w_out, const float *w_in, const float *gamma, float eps,
+                              const int32_t *row_list, const long long *ids, const void *embed, int R, int S, int D,
+                              int vocab, void *stream) {
+  DJV_REQUIRE(dtype == DJV_DTYPE_BF16 || dtype == DJV_DTYPE_F32, "hyper_step: dtype %d", dtype);
+  DJV_REQUIRE(x_in || (ids && embed && vocab > 0), "hyper_step: neither streams nor an embedding given");
+  DJV_REQUIRE(!y || (mix && w_out), "hyper_step: y without mix and out coefficients");
+  DJV_REQUIRE(!gamma || h, "hyper_step: null output");
+  DJV_REQUIRE(S >= 1 && S <= 8, "hyper_step: %d streams (1..8 are supported)", S);
+  DJV_REQUIRE(D >= 1 && D <= 49152 && R >= 0, "hyper_step: D=%d R=%d", D, R);
+  if (R == 0) return DJV_OK;
+  const HyperArgs a{h, x_out, x_in, y, mix, w_out, w_in, gamma, eps, row_list, ids, embed, D, vocab};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool vec = D % 4 == 0 && aligned16(x_in) && aligned16(x_out) && aligned16(y) && aligned16(h);
+  if (dtype == DJV_DTYPE_BF16) return vec ? launch_hyper<bf16, 4>(a, R, S, st) : launch_hyper<bf16, 1>(a, R, S, st);
+  return vec ? launch_hyper<float, 4>(a, R, S, st) : launch_hyper<float, 1>(a, R, S, st);
+}
+
+extern "C" int djv_clamped_glu(int dtype, void *y, const void *gu, long long R, int F, float limit, void *stream) {
+  DJV_REQUIRE(dtype == DJV_DTYPE_BF16 || dtype == DJV_DTYPE_F32, "clamped_glu: dtype %d", dtype);
+  DJV_REQUIRE(y && gu && aligned16(y) && aligned16(gu), "clamped_glu: null or misaligned pointer");
+  DJV_REQUIRE(R >= 0 && F >= 1 && limit >= 0.f, "clamped_glu: R=%lld F=%d limit=%g", R, F, (double)limit);
+  const long long total = R * F;
+  if (total == 0) return DJV_OK;
+  const long long blocks = (total + 1023) / 1024;
+  DJV_REQUIRE(blocks < (1ll << 31), "clamped_glu: too many elements");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (dtype == DJV_DTYPE_BF16)
+    djv::launch_kernel(clamped_glu_kernel<bf16>, (unsigned)blocks, 256, 0, st, static_cast<bf16 *>(y),
+                       static_cast<const bf16 *>(gu), total, limit);
+  else
+    djv::launch_kernel(clamped_glu_kernel<float>, (unsigned)blocks, 256, 0, st, static_cast<float *>(y),
+                       static_cast<const float *>(gu), total, limit);
+  count_launch();
+  return check_launch("clamped_glu");
+}
+
+extern "C" int djv_softcap(float *y, long long n, float cap, void *stream) {
+  DJV_REQUIRE(y && n >= 0 && cap > 0.f, "softcap: null pointer, n=%lld or cap=%g", n, (double)cap);
+  if (n == 0) return DJV_OK;
+  DJV_REQUIRE((n + 255) / 256 < (1ll << 31), "softcap: too many elements");
+  djv::launch_kernel(softcap_kernel, (unsigned)((n + 255) / 256), 256, 0, static_cast<cudaStream_t>(stream), y, n, cap);
+  count_launch();
+  return check_launch("softcap");
+}

@@ -46,29 +46,6 @@ struct RmSmem {
   static constexpr size_t BYTES = RM_IDX_BYTES + (size_t)RM_WARPS * D * RmStage<NTM>::BYTES;
 };
 
-__device__ __forceinline__ void cp_async16_zfill(uint32_t dst_smem, const void *src, int src_bytes) {
-  asm volatile("cp.async.cg.shared.global.L2::128B [%0], [%1], 16, %2;" ::"r"(dst_smem), "l"(src), "r"(src_bytes)
-               : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() {
-  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
-}
-// four 8x8 fp16 matrices: lane (g, t) gets elements [g][2t], [g][2t+1] of each ...
-__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr_smem) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(addr_smem)
-               : "memory");
-}
-// ... or, transposed on the way, elements [2t][g], [2t+1][g]
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr_smem) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(addr_smem)
-               : "memory");
-}
 
 template <int NTM, int D>  // tiles of 16 activation rows; steps in the ring
 __global__ void __launch_bounds__(RM_THREADS, 1)

@@ -1,4 +1,5 @@
-// rowdot_mma: gather GEMV for 9..32 rows of x on the tensor cores (mma.sync m16n8k16, fp16 in, fp32 accumulate).
+// rowdot_mma: gather GEMV for up to 32 rows of x on the tensor cores (mma.sync m16n8k16, fp16 or bf16 in, fp32
+// accumulate).
 //
 //   y[b, m] = act( w[idx[m], :] . x[b, :] + bias[idx[m]] )
 //
@@ -13,19 +14,14 @@
 #include <cooperative_groups.h>
 
 #include "common.cuh"
+#include "mma.cuh"
+#include "rowdot.cuh"
 
 namespace djv {
 
 constexpr int MM_THREADS = 256;
 constexpr int MM_WARPS = MM_THREADS / WARP;
 constexpr int MM_ROWS = 16;
-
-__device__ __forceinline__ void mma_m16n8k16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
-                                             uint32_t b0, uint32_t b1) {
-  asm("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
 
 // Short index lists: M / 16 blocks would leave most of the device idle, so the reduction dimension is also split
 // over the blocks of a thread-block cluster (grid (tiles, S), cluster (1, S), 1 <= S <= 8): block s of a cluster
@@ -40,11 +36,11 @@ struct MmaBlocks {
   static constexpr int PER_SM = NT == 1 ? 5 : 1;  // (1: whatever the compiler's register count allows, 4 here)
 };
 
-template <int NT, int ACT>  // NT groups of 8 activation rows
+template <typename T, typename TO, int NT, int ACT>  // NT groups of 8 activation rows
 __global__ void __launch_bounds__(MM_THREADS, MmaBlocks<NT>::PER_SM)
-rowdot_mma_kernel(__half *__restrict__ Y, const __half *__restrict__ W, const __half *__restrict__ X,
-                  const void *__restrict__ idx, const __half *__restrict__ bias, int M, int N,
-                  long long ldw, int idx64, int B) {
+rowdot_mma_kernel(TO *__restrict__ Y, const T *__restrict__ W, const T *__restrict__ X,
+                  const void *__restrict__ idx, const T *__restrict__ bias, int M, int N,
+                  long long ldw, int idx64, int B, float act_param) {
   pdl_prologue();
   __shared__ float red[MM_WARPS][NT][MM_ROWS][8];
   __shared__ float bsum[NT][MM_ROWS][8];
@@ -55,8 +51,8 @@ rowdot_mma_kernel(__half *__restrict__ Y, const __half *__restrict__ W, const __
   const int m_lo = m0 + g, m_hi = m0 + g + 8;
   const long long r_lo = (m_lo < M) ? load_index(idx, m_lo, idx64) : -1;
   const long long r_hi = (m_hi < M) ? load_index(idx, m_hi, idx64) : -1;
-  const __half *w_lo = W + (r_lo < 0 ? 0 : r_lo) * ldw;
-  const __half *w_hi = W + (r_hi < 0 ? 0 : r_hi) * ldw;
+  const T *w_lo = W + (r_lo < 0 ? 0 : r_lo) * ldw;
+  const T *w_hi = W + (r_hi < 0 ? 0 : r_hi) * ldw;
 
   float acc[NT][4];
 #pragma unroll
@@ -86,8 +82,8 @@ rowdot_mma_kernel(__half *__restrict__ Y, const __half *__restrict__ W, const __
 #pragma unroll
       for (int j = 0; j < NT; ++j) {
         // blocks past the end of the row hold zeros on both sides and add nothing
-        mma_m16n8k16(acc[j], a_lo[u].x, a_hi[u].x, a_lo[u].y, a_hi[u].y, xv[u][j].x, xv[u][j].y);
-        mma_m16n8k16(acc[j], a_lo[u].z, a_hi[u].z, a_lo[u].w, a_hi[u].w, xv[u][j].z, xv[u][j].w);
+        mma_m16n8k16_t<T>(acc[j], a_lo[u].x, a_hi[u].x, a_lo[u].y, a_hi[u].y, xv[u][j].x, xv[u][j].y);
+        mma_m16n8k16_t<T>(acc[j], a_lo[u].z, a_hi[u].z, a_lo[u].w, a_hi[u].w, xv[u][j].z, xv[u][j].w);
       }
     }
   }
@@ -118,35 +114,36 @@ rowdot_mma_kernel(__half *__restrict__ Y, const __half *__restrict__ W, const __
       const int j = o / (MM_ROWS * 8), row = (o / 8) % MM_ROWS, c = o % 8;
       const int m = m0 + row, tok = j * 8 + c;
       if (m < M && tok < B) {
-        float s = 0.f;
-        if (S > 1) {
-          for (int q = 0; q < S; ++q) s += cluster.map_shared_rank(&bsum[0][0][0], q)[o];
-        } else {
+        auto total = [&](int at) {  // sum of one (row, token) over the warps, and over the blocks of the cluster
+          float s = 0.f;
+          if (S > 1) {
+            for (int q = 0; q < S; ++q) s += cluster.map_shared_rank(&bsum[0][0][0], q)[at];
+          } else {
+            const int jj = at / (MM_ROWS * 8), rr = (at / 8) % MM_ROWS, cc = at % 8;
 #pragma unroll
-          for (int w2 = 0; w2 < MM_WARPS; ++w2) s += red[w2][j][row][c];
+            for (int w2 = 0; w2 < MM_WARPS; ++w2) s += red[w2][jj][rr][cc];
+          }
+          return s;
+        };
+        if (ACT == DJV_ACT_CLAMPED_GLU) {
+          // rows 2i, 2i + 1 are the gate and up rows of output i (no bias in this form)
+          if (row % 2 == 0 && m + 1 < M)
+            Y[(size_t)tok * (M / 2) + m / 2] = from_f<TO>(clamped_glu(total(o), total(o + 8), act_param));
+        } else {
+          float s = total(o);
+          if (bias != nullptr) s += to_f(bias[load_index(idx, m, idx64)]);
+          Y[(size_t)tok * M + m] = from_f<TO>(apply_act_param<ACT>(s, act_param));
         }
-        if (bias != nullptr) s += __half2float(bias[load_index(idx, m, idx64)]);
-        Y[(size_t)tok * M + m] = __float2half_rn(apply_act<ACT>(s));
       }
     }
   }
   if (S > 1) cluster.sync();  // no block leaves while block 0 may still read its sums
 }
 
-template <int NT>
-inline int launch_rowdot_mma(int act, __half *Y, const __half *W, const __half *X, const void *idx,
-                             const __half *bias, int M, int N, long long ldw, int idx64, int B, cudaStream_t st) {
+// Blocks of the cluster that split the reduction; `bps` is the kernel's occupancy.
+inline int rowdot_mma_split(int M, int N, int NT, int bps) {
   const int tiles = ceil_div(M, MM_ROWS);
   // Split the reduction over the S blocks of a cluster when the tiles alone leave multiprocessors idle.
-  static const int bps = [] {
-    int n = 0;
-    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, rowdot_mma_kernel<NT, DJV_ACT_RELU>, MM_THREADS, 0) !=
-        cudaSuccess) {
-      cudaGetLastError();
-      n = 1;
-    }
-    return n < 1 ? 1 : n;
-  }();
   const int slots = sm_count() * bps;
   // Measured behaviour: the resident blocks run in waves; a wave costs a fixed ~5 us (row numbers, first loads,
   // reduction, cluster barriers) plus, per k-block of 32 columns a warp walks, the larger of a latency floor that
@@ -172,33 +169,7 @@ inline int launch_rowdot_mma(int act, __half *Y, const __half *W, const __half *
   }
   static const int k_s = env_int("DJV_MMA_S", 0);  // development knob
   if (k_s >= 1 && k_s <= 8) S = k_s;
-  const dim3 grid(tiles, S), cluster(1, S, 1);
-#define DJV_MM(ACT_)                                                                                              \
-  djv::launch_kernel_cluster(rowdot_mma_kernel<NT, ACT_>, grid, dim3(MM_THREADS), 0, st, cluster, Y, W, X, idx, bias, \
-                             M, N, ldw, idx64, B)
-  switch (act) {
-    case DJV_ACT_ID: DJV_MM(DJV_ACT_ID); break;
-    case DJV_ACT_RELU: DJV_MM(DJV_ACT_RELU); break;
-    case DJV_ACT_GELU: DJV_MM(DJV_ACT_GELU); break;
-    case DJV_ACT_GELU_APPROX: DJV_MM(DJV_ACT_GELU_APPROX); break;
-    case DJV_ACT_SQUARED_RELU: DJV_MM(DJV_ACT_SQUARED_RELU); break;
-    default: set_error("gather_gemv: unknown activation %d", act); return DJV_ERR_INVALID;
-  }
-#undef DJV_MM
-  return DJV_OK;
-}
-
-// 9 <= B <= 32
-inline int rowdot_mma(int B, int act, __half *Y, const __half *W, const __half *X, const void *idx,
-                      const __half *bias, int M, int N, long long ldw, int idx64, cudaStream_t st) {
-  switch ((B + 7) / 8) {
-    case 1: return launch_rowdot_mma<1>(act, Y, W, X, idx, bias, M, N, ldw, idx64, B, st);
-    case 2: return launch_rowdot_mma<2>(act, Y, W, X, idx, bias, M, N, ldw, idx64, B, st);
-    case 3: return launch_rowdot_mma<3>(act, Y, W, X, idx, bias, M, N, ldw, idx64, B, st);
-    case 4: return launch_rowdot_mma<4>(act, Y, W, X, idx, bias, M, N, ldw, idx64, B, st);
-  }
-  set_error("gather_gemv: batch %d outside the tensor-core kernel's range", B);
-  return DJV_ERR_INVALID;
+  return S;
 }
 
 }  // namespace djv

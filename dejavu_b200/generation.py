@@ -11,6 +11,11 @@ The K/V caches use the decode kernel's layouts, per layer: K (B, heads_local, he
 V (B, heads_local, S, head_dim). Everything the decode step needs to know about the position (cache
 length, lazy-K/V window) is device-resident state advanced by the kernels, so one captured graph is valid
 for every step; only input_ids and position_ids are rewritten between replays.
+
+A model whose layers keep something else (rings of a window, recurrent states) brings its own `allocate_cache`, and
+everything here works on what that returns: `step` runs the next tokens of every sequence from the caches, `generate`
+is built on it, and `SequencePool` serves independent requests, each from a cache of its own that the next request
+takes over.
 """
 from __future__ import annotations
 
@@ -37,6 +42,8 @@ class InferenceParams:
 
 
 def allocate_kv_cache(model, batch_size: int, max_seqlen: int, device, dtype=torch.float16) -> dict:
+    if hasattr(model, "allocate_cache"):
+        return model.allocate_cache(batch_size, max_seqlen, device)
     cfg = model.config
     hd = cfg.hidden_size // cfg.n_head
     assert hd % 8 == 0
@@ -95,8 +102,7 @@ def update_graph_cache(model, cache, batch_size, seqlen_og, max_seqlen, tensor_p
     cache.input_ids = torch.zeros(batch_size, 1, dtype=torch.long, device=device)
     cache.position_ids = torch.full((batch_size, 1), seqlen_og, dtype=torch.long, device=device)
     # the decode state must describe a decodable position while warming up
-    for layer in model.transformer.layers:
-        layer.mixer.reset_decode_state(seqlen_og, device, max_seqlen, batch_size)
+    model.reset_decode_state(seqlen_og, device, max_seqlen, batch_size)
     s = torch.cuda.Stream()
     s.wait_stream(torch.cuda.current_stream())
     def step():
@@ -128,14 +134,77 @@ def update_graph_cache(model, cache, batch_size, seqlen_og, max_seqlen, tensor_p
     return cache
 
 
+@torch.inference_mode()
+def step(model, params: InferenceParams, input_ids, position_ids=None, logit_rows=None):
+    """Runs the next input_ids (B, n) of every sequence, from what the caches hold after params.sequence_len_offset
+    tokens, and advances the offset. logit_rows: places among the n tokens whose logits are wanted (None: all).
+    Returns logits (B, rows, vocab)."""
+    n = input_ids.size(1)
+    if params.sequence_len_offset + n > params.max_sequence_len:
+        raise ValueError(f"{params.sequence_len_offset} + {n} tokens exceed the cache of {params.max_sequence_len}")
+    if getattr(model, "selects_logit_rows", False):
+        logits = model(input_ids, position_ids=position_ids, inference_params=params, logit_rows=logit_rows).logits
+    else:
+        logits = model(input_ids, position_ids=position_ids, inference_params=params).logits
+        if logit_rows is not None:
+            logits = logits[:, list(logit_rows)]
+    params.sequence_len_offset += n
+    return logits
+
+
+class SequencePool:
+    """Independent requests, one sequence each, run in portions of any size. A request takes a free slot (a cache for
+    one sequence of up to max_seqlen tokens) and gives it back at its end; a new request in a used slot starts at
+    position 0, which is all it takes to forget the old one."""
+
+    def __init__(self, model, max_seqlen: int, device):
+        self.model, self.max_seqlen, self.device = model, max_seqlen, device
+        self.free: list[InferenceParams] = []
+        self.live: dict = {}
+
+    def run(self, request, tokens, logit_rows=()):
+        """The next tokens (a list of ids) of `request`, a new one if it is not live. Returns (len(logit_rows), vocab)
+        logits."""
+        vocab = self.model.config.vocab_size
+        if not tokens:
+            raise ValueError(f"request {request}: no tokens")
+        if min(tokens) < 0 or max(tokens) >= vocab:
+            raise ValueError(f"request {request}: token outside the vocabulary of {vocab}")
+        if any(not 0 <= t < len(tokens) for t in logit_rows):
+            raise ValueError(f"request {request}: logits wanted outside the portion")
+        if request not in self.live:
+            self.live[request] = self._slot()
+        params = self.live[request]
+        if params.sequence_len_offset and len(tokens) > 1 and not getattr(self.model, "takes_portions", False):
+            raise ValueError("this model takes a prompt in one piece")
+        ids = torch.tensor([tokens], dtype=torch.long, device=self.device)
+        pos = torch.full((1, 1), params.sequence_len_offset, dtype=torch.long, device=self.device)
+        first = params.sequence_len_offset == 0 and len(tokens) > 1  # (models number a prompt's tokens themselves)
+        return step(self.model, params, ids, None if first else pos, logit_rows)[0]
+
+    def end(self, request):
+        """Gives the request's slot back."""
+        params = self.live.pop(request)
+        params.sequence_len_offset = 0
+        self.free.append(params)
+
+    def _slot(self) -> InferenceParams:
+        if self.free:
+            return self.free.pop()
+        return InferenceParams(max_sequence_len=self.max_seqlen, max_batch_size=1, fused_ft_kernel=True,
+                               key_value_memory_dict=allocate_kv_cache(self.model, 1, self.max_seqlen, self.device))
+
+
 class GenerationMixin:
     @torch.inference_mode()
     def generate(self, input_ids, max_length, top_k=1, top_p=0.0, temperature=1.0, fused_ft_kernel=True,
                  cg=False, vocab_size=None, return_dict_in_generate=False, output_scores=False, timing=False,
-                 **kwargs):
+                 prompt_chunk=None, **kwargs):
         """Greedy decoding (top_k=1 is the only sampler the benchmarks use). Returns an object with
-        .sequences (B, max_length) and, when asked, .scores (list of (B, vocab) logits per new token)."""
+        .sequences (B, max_length) and, when asked, .scores (list of (B, vocab) logits per new token).
+        prompt_chunk: the prompt runs in portions of at most that many tokens (models that take portions)."""
         assert top_k == 1, "only greedy decoding is implemented"
+        assert prompt_chunk is None or getattr(self, "takes_portions", False), "this model takes a prompt in one piece"
         B, seqlen_og = input_ids.shape
         device = input_ids.device
         if timing:
@@ -151,9 +220,11 @@ class GenerationMixin:
                                  key_value_memory_dict=allocate_kv_cache(self, B, max_length, device))
         ip.sequence_len_offset = 0
         # prompt pass (dense); fills the caches and resets the lazy-K/V state to base = prompt length
-        logits = self(input_ids, inference_params=ip).logits[:, -1]
+        portion = prompt_chunk or seqlen_og
+        for p0 in range(0, seqlen_og, portion):
+            part = input_ids[:, p0:p0 + portion]
+            logits = step(self, ip, part, logit_rows=[part.size(1) - 1])[:, -1]
         scores, sequences = [], [input_ids]
-        ip.sequence_len_offset = seqlen_og
         pos = torch.full((B, 1), seqlen_og, dtype=torch.long, device=device)
         while True:
             if vocab_size is not None:

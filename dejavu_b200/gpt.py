@@ -256,6 +256,10 @@ class GPTLMHeadModel(nn.Module, GenerationMixin):
             lm_logits = torch.cat(parts, dim=-1)
         return CausalLMOutput(logits=lm_logits)
 
+    def reset_decode_state(self, prompt_len, device, max_seqlen, batch=1):
+        for layer in self.transformer.layers:
+            layer.mixer.reset_decode_state(prompt_len, device, max_seqlen, batch)
+
     # ---- synthetic weights ----------------------------------------------------------------------
     @torch.no_grad()
     def init_random(self, seed: int = 0, std: float = 0.02):

@@ -476,3 +476,141 @@ def decode_attention(q, k_cache, v_cache, head_idx, length: int, softmax_scale: 
     call("djv_decode_attn", ctx.data_ptr(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), _ptr(head_idx),
          nnz, B, nheads, hd, S, length, float(softmax_scale), scratch.data_ptr(), scratch.numel(), _stream())
     return ctx
+
+
+# ---- hybrid decoders: gated linear attention, sliding windows, hyper-connected streams (bf16 or fp32) ---------------
+
+def _dtype_code(t: torch.Tensor) -> int:
+    if t.dtype == torch.bfloat16:
+        return _lib.DTYPE_BF16
+    assert t.dtype == torch.float32, f"bf16 or fp32 expected, got {t.dtype}"
+    return _lib.DTYPE_F32
+
+
+def _f32(*tensors):
+    for t in tensors:
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
+
+
+def hyper_step(x, y, mix, w_out, w_in, gamma, eps: float, dtype, *, x_out=None, rows=None, ids=None, embed=None,
+               streams=None):
+    """Boundary between two sublayers of a decoder with S residual streams (djv_hyper_step):
+        new_t = sum_s mix[s, t] x_s + w_out[t] y;  u = sum_t w_in[t] new_t;  h = u / rms(u) * gamma
+    x (rows, S, D) fp32, or None: all streams are embed[ids]. y None: no update. w_in None: plain sum. gamma None: only
+    the update. x_out (may be x) receives the new streams. rows (int32) selects rows. Returns h (R, D) in `dtype`."""
+    src = x if x is not None else ids
+    _require_cuda(src, y, embed)
+    _f32(x, y, mix, w_out, w_in, gamma, x_out)
+    if x is not None:
+        n, S, D = x.shape
+    else:
+        n, S, D = ids.numel(), streams, embed.shape[1]
+        assert ids.dtype == torch.int64 and ids.is_contiguous() and embed.is_contiguous() and embed.dtype == dtype
+    R = n if rows is None else rows.numel()
+    h = None if gamma is None else torch.empty(R, D, dtype=dtype, device=src.device)
+    code = _lib.DTYPE_BF16 if dtype == torch.bfloat16 else _lib.DTYPE_F32
+    call("djv_hyper_step", code, _ptr(h), _ptr(x_out), _ptr(x), _ptr(y), _ptr(mix), _ptr(w_out), _ptr(w_in),
+         _ptr(gamma), float(eps), _ptr(rows), None if x is not None else ids.data_ptr(),
+         None if x is not None else embed.data_ptr(), R, S, D, 0 if x is not None else embed.shape[0], _stream())
+    return h
+
+
+def linear_gemv(x: torch.Tensor, weight: torch.Tensor, out_dtype=None, activation: str = "id",
+                param: float = 0.0) -> torch.Tensor:
+    """y = activation(x @ weight.T) for a few rows of x (decode), bf16 or fp32 weights, result in their type or fp32.
+    activation "softcap" (param * tanh(v / param)) or "clamped_glu" (weight rows 2i, 2i+1 are gate and up of output i)."""
+    M, N = weight.shape
+    B = x.shape[0]
+    assert x.shape == (B, N) and 1 <= B <= _lib.MAX_BATCH and x.dtype == weight.dtype
+    assert weight.stride(1) == 1
+    _require_cuda(x, weight)
+    x = x.contiguous()
+    out_dtype = out_dtype or x.dtype
+    y = torch.empty(B, M // 2 if activation == "clamped_glu" else M, dtype=out_dtype, device=x.device)
+    call("djv_dense_gemv", _dtype_code(x), _dtype_code(y), y.data_ptr(), weight.data_ptr(), x.data_ptr(), B, N, M,
+         weight.stride(0), _lib.ACT[activation], float(param), _stream())
+    return y
+
+
+def clamped_glu(gu: torch.Tensor, limit: float) -> torch.Tensor:
+    """(R, 2F) with gate and up interleaved -> (R, F): min(g, limit) * sigmoid(1.702 .) * (clamp(u) + 1)."""
+    R, F2 = gu.shape
+    _require_cuda(gu)
+    assert gu.is_contiguous()
+    y = torch.empty(R, F2 // 2, dtype=gu.dtype, device=gu.device)
+    call("djv_clamped_glu", _dtype_code(gu), y.data_ptr(), gu.data_ptr(), R, F2 // 2, float(limit), _stream())
+    return y
+
+
+def softcap_(y: torch.Tensor, cap: float) -> torch.Tensor:
+    _require_cuda(y)
+    _f32(y)
+    call("djv_softcap", y.data_ptr(), y.numel(), float(cap), _stream())
+    return y
+
+
+def rotary_(buf: torch.Tensor, freqs: torch.Tensor, amp: float, pos: torch.Tensor, n: int, heads: int, dim: int):
+    """Rotates the first `heads` heads of `dim` elements of every row of buf (B*n, ld) in place; pos (B,) int64 is the
+    position of each sequence's first row."""
+    _require_cuda(buf, freqs, pos)
+    assert buf.stride(1) == 1 and pos.dtype == torch.int64 and buf.shape[0] == pos.numel() * n
+    call("djv_rotary", _dtype_code(buf), buf.data_ptr(), buf.stride(0), freqs.data_ptr(), float(amp), pos.data_ptr(),
+         pos.numel(), n, heads, dim, freqs.numel(), _stream())
+
+
+def _window_shapes(qkv, k_ring, v_ring, pos, n, heads):
+    B, G, cap, dk = k_ring.shape
+    dv = v_ring.shape[3]
+    assert v_ring.shape == (B, G, cap, dv) and k_ring.is_contiguous() and v_ring.is_contiguous()
+    b = pos.numel()
+    assert b <= B and qkv.shape[0] == b * n and qkv.shape[1] >= (heads + G) * dk + G * dv and qkv.stride(1) == 1
+    assert qkv.dtype == k_ring.dtype == v_ring.dtype and pos.dtype == torch.int64
+    _require_cuda(qkv, k_ring, v_ring, pos)
+    return b, G, cap, dk, dv
+
+
+def window_attention(qkv, k_ring, v_ring, sink, pos, n: int, heads: int, window: int, scale: float):
+    """n new tokens per sequence over the rings and themselves, then the new tokens enter the rings.
+    qkv (B*n, (H+G)*dk + G*dv), rotated. Returns (B*n, H*dv)."""
+    b, G, cap, dk, dv = _window_shapes(qkv, k_ring, v_ring, pos, n, heads)
+    _f32(sink)
+    out = torch.empty(b * n, heads * dv, dtype=qkv.dtype, device=qkv.device)
+    code = _dtype_code(qkv)
+    call("djv_window_attn", code, out.data_ptr(), qkv.data_ptr(), qkv.stride(0), k_ring.data_ptr(), v_ring.data_ptr(),
+         _ptr(sink), pos.data_ptr(), b, n, heads, G, dk, dv, cap, window, float(scale), _stream())
+    call("djv_window_store", code, k_ring.data_ptr(), v_ring.data_ptr(), qkv.data_ptr(), qkv.stride(0), pos.data_ptr(),
+         b, n, heads, G, dk, dv, cap, _stream())
+    return out
+
+
+def window_attention_decode(qkv, k_ring, v_ring, sink, freqs, amp: float, pos, heads: int, window: int, scale: float):
+    """One token per sequence, qkv not rotated: rotation, ring store and attention in one kernel."""
+    b, G, cap, dk, dv = _window_shapes(qkv, k_ring, v_ring, pos, 1, heads)
+    _f32(sink, freqs)
+    out = torch.empty(b, heads * dv, dtype=qkv.dtype, device=qkv.device)
+    call("djv_window_attn_decode", _dtype_code(qkv), out.data_ptr(), qkv.data_ptr(), qkv.stride(0), k_ring.data_ptr(),
+         v_ring.data_ptr(), _ptr(sink), _ptr(freqs), float(amp), 0 if freqs is None else freqs.numel(), pos.data_ptr(),
+         b, heads, G, dk, dv, cap, window, float(scale), _stream())
+    return out
+
+
+def gated_linear_attention(proj, a2, a2_bias, tau: float, norm, eps: float, scale: float, state, pos, n: int):
+    """proj (B*n, q | k | v | gate | low-rank decay input) -> (B*n, H*dv), normed and gated; state (B, H, dk, dv) fp32
+    is advanced in place (a sequence at position 0 starts from zero)."""
+    _, H, dk, dv = state.shape
+    b, rank = pos.numel(), a2.shape[1]
+    assert proj.shape[0] == b * n and proj.shape[1] >= 2 * H * (dk + dv) + rank and proj.stride(1) == 1
+    assert b <= state.shape[0] and a2.shape[0] == H * dk and pos.dtype == torch.int64
+    _require_cuda(proj, a2, state, pos)
+    _f32(a2, a2_bias, norm, state)
+    out = torch.empty(b * n, H * dv, dtype=proj.dtype, device=proj.device)
+    code = _dtype_code(proj)
+    args = (code, out.data_ptr(), proj.data_ptr(), proj.stride(0), a2.data_ptr(), a2_bias.data_ptr(), rank, 1.0 / tau,
+            norm.data_ptr(), float(eps), float(scale), state.data_ptr(), pos.data_ptr(), b)
+    if n == 1:
+        call("djv_gla_decode", *args, H, dk, dv, _stream())
+    else:
+        need = _lib.load_hybrid().djv_gla_scratch_bytes(code, b, n, H, dk, dv)
+        scratch = torch.empty(max(need, 256), dtype=torch.uint8, device=proj.device)
+        call("djv_gla_prefill", *args, n, H, dk, dv, scratch.data_ptr(), scratch.numel(), _stream())
+    return out

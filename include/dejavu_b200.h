@@ -36,6 +36,15 @@ extern "C" {
 #define DJV_ACT_GELU 2
 #define DJV_ACT_GELU_APPROX 3
 #define DJV_ACT_SQUARED_RELU 4
+/* activations with a constant, only of the entry points that take one */
+#define DJV_ACT_SOFTCAP 5     /* c * tanh(v / c)                                                          */
+#define DJV_ACT_CLAMPED_GLU 6 /* rows 2i, 2i+1 = gate, up: g = min(gate, c), u = clamp(up, -c, c),        */
+                              /* g * sigmoid(1.702 g) * (u + 1)                                           */
+
+/* element types of the entry points that are compiled for several */
+#define DJV_DTYPE_F16 0
+#define DJV_DTYPE_BF16 1
+#define DJV_DTYPE_F32 2
 
 /* Limits shared with the host-side shims. */
 #define DJV_MAX_BATCH 32        /* rows of x for the GEMV kernels                        */

@@ -7,10 +7,11 @@ import pytest
 
 ROOT = Path(__file__).resolve().parents[1]
 HEADER = ROOT / "include" / "dejavu_b200.h"
+HYBRID_HEADER = ROOT / "include" / "dejavu_b200_hybrid.h"
 
 
-def declared_functions():
-    text = re.sub(r"/\*.*?\*/", "", HEADER.read_text(), flags=re.S)
+def declared_functions(header=HEADER):
+    text = re.sub(r"/\*.*?\*/", "", header.read_text(), flags=re.S)
     return sorted(set(re.findall(r"\b(djv_[a-z0-9_]+)\s*\(", text)))
 
 
@@ -36,6 +37,17 @@ def test_binding_table_matches_header(lib):
     from dejavu_b200 import _lib
 
     assert sorted(_lib.SIGNATURES) == declared_functions()
+
+
+def test_hybrid_library_matches_its_header(lib):
+    from dejavu_b200 import _lib
+
+    names = declared_functions(HYBRID_HEADER)
+    hybrid = _lib.load_hybrid()
+    assert sorted(_lib.HYBRID_SIGNATURES) == names and "djv_gla_prefill" in names
+    for name in names:
+        assert hasattr(hybrid, name)
+    assert hybrid.djv_version() >= 100
 
 
 def test_host_only_calls_work_without_a_gpu(lib):
