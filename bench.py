@@ -15,6 +15,8 @@ uniform-random prompt) after a dense prompt pass. Prints one JSON line:
   dense          the same model and weights with every head and neuron (dense comparator)
   cpu_baseline   the reference's torch formulation on the host cores (bounded sample, N=1 only)
 `--impl reference` times only that CPU formulation (all host threads) and prints it in the same format.
+`--hybrid 1b,7b` instead times the Ninolorn design beside the dense OPT decoder at those sizes (one GPU; see
+dejavu_b200/hybrid_bench.py) and prints one JSON line of its own.
 """
 from __future__ import annotations
 
@@ -324,6 +326,20 @@ def run_reference(args, cfg, mlp_K, att_K, world, rank):
     emit(line)
 
 
+def run_hybrid(args):
+    """Throughput and kernels of the hybrid design beside dense OPT, one JSON line."""
+    from dejavu_b200 import _lib, hybrid_bench
+
+    _lib.load(), _lib.load_hybrid()  # fail loudly if a CUDA library is missing
+    peak, kind = measured_peaks()
+    p = ROOT / "MEASURED_PEAKS.json"
+    tflops = float(json.loads(p.read_text())["bf16_tflops"]) if p.exists() else 1590.0
+    with ClockSampler(0) as clocks:
+        res = hybrid_bench.run(args.hybrid.split(","), kernel_timing, peak, tflops, prompt=args.promptlen or 4096)
+    emit({"metric": "hybrid_decoder_throughput", "peak_gbs": peak, "peak_tflops": tflops, "peak_kind": kind,
+          "data": "synthetic", "sizes": res, "clocks": clocks.summary()})
+
+
 def base_line(args, cfg, mlp_K, att_K, world):
     return {
         "metric": "decode_ms_per_token", "value": None, "unit": "ms/token", "n_gpus": world, "steps": args.steps,
@@ -383,8 +399,12 @@ def main():
     ap.add_argument("--no-dense", action="store_true")
     ap.add_argument("--no-cpu", action="store_true")
     ap.add_argument("--fused-allreduce", type=int, default=1)
+    ap.add_argument("--hybrid", default=None, help="comma-separated sizes (1b, 7b, 30b): time the hybrid design beside dense OPT")
     args = ap.parse_args()
 
+    if args.hybrid:
+        run_hybrid(args)
+        return
     if args.model_name:
         args.workload = args.model_name.split("/")[-1].lower()
         assert args.workload in WORKLOADS, f"unknown model {args.model_name}"
