@@ -103,6 +103,7 @@ HYBRID_SIGNATURES = {
     "djv_window_store": (_i, [_i, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "djv_window_attn_decode": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _f, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _f,
                                     _vp]),
+    "djv_window_timeouts": (C.c_uint, []),
     "djv_gla_scratch_bytes": (_sz, [_i, _i, _i, _i, _i, _i]),
     "djv_gla_prefill": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _i, _f, _vp, _f, _f, _vp, _vp, _i, _i, _i, _i, _i, _vp, _sz,
                              _vp]),

@@ -463,7 +463,7 @@ extern "C" int djv_window_attn(int dtype, void *out, const void *qkv, long long 
   if (window > cap) window = cap;  // a ring that is shorter than the window holds the longest sequence
   const WindowArgs a{out, qkv, ld, k_ring, v_ring, sink, pos, B, n, H, G, dk, dv, cap, window, scale};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dtype == DJV_DTYPE_BF16) return launch_simple<bf16>(a, st);
+  if (dtype == DJV_DTYPE_BF16) return window_prefill_supported(a) ? window_prefill(a, st) : launch_simple<bf16>(a, st);
   return launch_simple<float>(a, st);
 }
 

@@ -15,4 +15,8 @@ struct WindowArgs {
   float scale;
 };
 
+// tensor-core form for prompt portions (bf16)
+bool window_prefill_supported(const WindowArgs &a);
+int window_prefill(const WindowArgs &a, cudaStream_t st);
+
 }  // namespace djv

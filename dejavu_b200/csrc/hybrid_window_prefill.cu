@@ -1,0 +1,292 @@
+// Sliding-window attention of a prompt portion on the 5th-generation tensor cores (bf16).
+//
+// A block takes 128 queries of one head and walks the key tiles of 128 that their windows touch:
+//   S (TMEM, 128 x 128 fp32) = Q K^T;  softmax in registers, one query row per thread, no shuffles;
+//   P goes back to TMEM over S as two bf16 terms, p = hi + lo, so that the weights keep their fp32 value to 2^-17;
+//   O (TMEM, 128 x dv fp32) += P_hi V + P_lo V.
+// O is only rescaled when a row's maximum grows by more than 2^8 (the final division by the sum makes up for the rest).
+// Keys come from the ring (tokens before the portion) or from the projection's output (the portion's own), row by row,
+// with 16-byte asynchronous copies into the swizzled operand layout. Two blocks share a multiprocessor: one computes
+// its softmax while the other's products run. K of the next tile loads behind the scores, V behind the values.
+#include "../../include/dejavu_b200_hybrid.h"
+#include "hybrid_attention.cuh"
+#include "tcgen05.cuh"
+
+namespace djv {
+
+constexpr int WP_THREADS = 128;
+constexpr int WP_TILE = 128;  // queries per block, keys per tile
+
+__device__ unsigned g_window_timeouts;  // bounded waits that ran out (never, in a healthy run)
+
+__device__ __forceinline__ float exp2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int KB, int VB>  // 64-element blocks of a query/key row and of a value row
+__global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a) {
+  extern __shared__ unsigned char smem_raw[];
+  __shared__ __align__(8) uint64_t bar_s, bar_o;
+  __shared__ uint32_t tmem_slot;
+  constexpr uint32_t COLS = VB > 2 ? 512 : 256;
+  constexpr uint32_t KT = KB * WP_TILE * 128;
+  const int tid = threadIdx.x, warp = tid / WARP;
+  const int h = blockIdx.y, b = blockIdx.z, g = h / (a.H / a.G);
+  const int t0 = blockIdx.x * WP_TILE;
+  unsigned char *base = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+  const uint32_t q_sm = smem_u32(base), k_sm = q_sm + KT, v_sm = k_sm + KT;
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+
+  if (tid == 0) {
+    mbar_init(&bar_s, 1);
+    mbar_init(&bar_o, 1);
+    mbar_fence_init();
+  }
+  __syncwarp();
+  if (warp == 0) tmem_alloc(&tmem_slot, COLS);
+
+  const bf16 *rows = static_cast<const bf16 *>(a.qkv) + (size_t)b * a.n * a.ld;
+  const bf16 *kr = static_cast<const bf16 *>(a.k_ring) + ((size_t)b * a.G + g) * a.cap * a.dk;
+  const bf16 *vr = static_cast<const bf16 *>(a.v_ring) + ((size_t)b * a.G + g) * a.cap * a.dv;
+  const long long p0 = a.pos[b];
+  const int last = min(t0 + WP_TILE, a.n) - 1;
+  // everything below is relative to the portion: key j of the portion is token j, the ring holds j < 0
+  const long long reach = p0 < (long long)a.window - 1 ? p0 : (long long)a.window - 1;  // ring tokens the portion can see
+  int lo = t0 - (a.window - 1);
+  if (lo < -(int)reach) lo = -(int)reach;
+  const int tiles = (last - lo) / WP_TILE + 1;
+  const int ring_slot0 = (int)((p0 - reach) % a.cap);  // slot of token -reach
+
+  auto load = [&](uint32_t dst, int j0, const bf16 *ring, int dim, const bf16 *fresh, int blocks) {
+    const int per_row = blocks * 8;  // chunks, a power of two
+    const int ch = tid & (per_row - 1);
+    const bool inside = ch * 8 < dim;
+    for (int r = tid / per_row; r < WP_TILE; r += WP_THREADS / per_row) {
+      const int j = j0 + r;
+      const bf16 *src = fresh;
+      bool ok = inside && j <= last;
+      if (ok) {
+        if (j >= 0) {
+          src = fresh + (size_t)j * a.ld + ch * 8;
+        } else {
+          int slot = ring_slot0 + (j + (int)reach);
+          if (slot >= a.cap) slot -= a.cap;
+          src = ring + (size_t)slot * dim + ch * 8;
+        }
+      }
+      cp_async16_zfill(dst + sw128_offset(WP_TILE, r, ch), src, ok ? 16 : 0);
+    }
+    cp_async_commit();
+  };
+  const bf16 *k_new = rows + (size_t)(a.H + g) * a.dk;
+  const bf16 *v_new = rows + (size_t)(a.H + a.G) * a.dk + (size_t)g * a.dv;
+  {  // queries
+    constexpr int PER_ROW = KB * 8;
+    const int ch = tid & (PER_ROW - 1);
+    for (int r = tid / PER_ROW; r < WP_TILE; r += WP_THREADS / PER_ROW) {
+      const bool ok = ch * 8 < a.dk && t0 + r <= last;
+      cp_async16_zfill(q_sm + sw128_offset(WP_TILE, r, ch),
+                       ok ? rows + (size_t)(t0 + r) * a.ld + (size_t)h * a.dk + ch * 8 : rows, ok ? 16 : 0);
+    }
+  }
+  load(k_sm, lo, kr, a.dk, k_new, KB);
+
+  const float sink = a.sink ? a.sink[h] * 1.4426950408889634f : 0.f;
+  const float c = a.scale * 1.4426950408889634f;  // scores in units of log 2
+  float m = -1e30f, l = 0.f;
+  const int row = t0 + tid;
+  const uint32_t idesc_s = mma_idesc(WP_TILE, WP_TILE, false, false);
+  const int dvp = (a.dv + 15) / 16 * 16;
+  const uint32_t idesc_o = mma_idesc(WP_TILE, dvp, false, true);
+  const int k_steps = (a.dk + 15) / 16;
+  bool dead = false;  // a wait ran out: wait no more, finish and report
+  __syncthreads();
+  tmem_fence_after();
+  const uint32_t tm = tmem_slot;
+  const uint32_t tm_s = tm, tm_o = tm + WP_TILE;
+  const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
+
+  for (int i = 0; i < tiles; ++i) {
+    const int j0 = lo + i * WP_TILE;
+    if (i > 0) {  // the last tile's values: P (over S), V and O are free
+      if (!dead) dead = !mbar_wait(&bar_o, (i - 1) & 1);
+      __syncwarp();  // (TMEM accesses are whole-warp instructions)
+      tmem_fence_after();
+    }
+    cp_async_wait<0>();
+    fence_proxy_async_smem();
+    __syncthreads();
+    if (tid == 0) {
+      tmem_fence_after();
+      for (int k = 0; k < k_steps; ++k)
+        mma_ss(tm_s, desc_k_major(q_sm, WP_TILE, k), desc_k_major(k_sm, WP_TILE, k), idesc_s, k > 0);
+      mma_commit(&bar_s);
+    }
+    load(v_sm, j0, vr, a.dv, v_new, VB);
+    if (!dead) dead = !mbar_wait(&bar_s, i & 1);
+    __syncwarp();
+    tmem_fence_after();
+    if (i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, KB);
+
+    __syncwarp();
+    uint32_t s[4][32];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) tmem_ld32(s[q], tm_s + lane_base + q * 32);
+    tmem_wait_ld();
+    // keys outside this row's window: those after it and those more than window - 1 before it
+    const bool edge = j0 + WP_TILE - 1 > t0 || j0 < t0 + WP_TILE - a.window;
+    if (edge) {
+      const int hi_c = row - j0, lo_c = row - a.window + 1 - j0;  // columns lo_c .. hi_c are seen
+#pragma unroll
+      for (int q = 0; q < 4; ++q)
+#pragma unroll
+        for (int e = 0; e < 32; ++e)
+          if (q * 32 + e > hi_c || q * 32 + e < lo_c) s[q][e] = 0xff800000u;  // -inf
+    }
+    // (a negative scale turns the maximum round; masked entries stay at -inf below)
+    float mx = -INFINITY;
+    if (c >= 0.f) {
+#pragma unroll
+      for (int q = 0; q < 4; ++q)
+#pragma unroll
+        for (int e = 0; e < 32; ++e) mx = fmaxf(mx, __uint_as_float(s[q][e]));
+    } else {
+#pragma unroll
+      for (int q = 0; q < 4; ++q)
+#pragma unroll
+        for (int e = 0; e < 32; ++e)
+          if (s[q][e] != 0xff800000u) {
+            mx = fmaxf(mx, -__uint_as_float(s[q][e]));
+            s[q][e] ^= 0x80000000u;
+          }
+    }
+    const float ca = fabsf(c);
+    mx *= ca;
+    if (a.sink && i == 0) mx = fmaxf(mx, sink);
+    const bool grow = mx > m + 8.f;
+    if (i == 0) {
+      m = fmaxf(mx, m);
+      l = a.sink ? exp2_approx(sink - m) : 0.f;
+    } else if (__any_sync(0xffffffffu, grow)) {
+      const float corr = grow ? exp2_approx(m - mx) : 1.f;
+      if (grow) m = mx;
+      l *= corr;
+      for (int q = 0; q < dvp; q += 32) {  // (TMEM columns up to the next multiple of 32 belong to this block)
+        uint32_t o[32];
+        tmem_ld32(o, tm_o + lane_base + q);
+        tmem_wait_ld();
+#pragma unroll
+        for (int e = 0; e < 32; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * corr);
+        tmem_st32(tm_o + lane_base + q, o);
+      }
+    }
+    const float nm = -m;
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      uint32_t hi[16], lw[16];
+#pragma unroll
+      for (int e = 0; e < 16; ++e) {
+        const float x = exp2_approx(fmaf(__uint_as_float(s[q][2 * e]), ca, nm));
+        const float y = exp2_approx(fmaf(__uint_as_float(s[q][2 * e + 1]), ca, nm));
+        l += x + y;
+        hi[e] = pack_bf16(x, y);
+        const float2 r = b2f(hi[e]);
+        lw[e] = pack_bf16(x - r.x, y - r.y);
+      }
+      tmem_st16(tm_s + lane_base + q * 16, hi);
+      tmem_st16(tm_s + lane_base + 64 + q * 16, lw);
+    }
+    tmem_wait_st();
+    tmem_fence_before();
+    if (i + 1 < tiles)
+      cp_async_wait<1>();  // V is there; K of the next tile may still be on its way
+    else
+      cp_async_wait<0>();
+    fence_proxy_async_smem();
+    __syncthreads();
+    if (tid == 0) {
+      tmem_fence_after();
+      for (int k = 0; k < WP_TILE / 16; ++k)
+        mma_ts(tm_o, tm_s + k * 8, desc_mn_major(v_sm, WP_TILE, k), idesc_o, i > 0 || k > 0);
+      for (int k = 0; k < WP_TILE / 16; ++k)
+        mma_ts(tm_o, tm_s + 64 + k * 8, desc_mn_major(v_sm, WP_TILE, k), idesc_o, true);
+      mma_commit(&bar_o);
+    }
+  }
+  if (!dead) dead = !mbar_wait(&bar_o, (tiles - 1) & 1);
+  __syncwarp();
+  tmem_fence_after();
+  const float inv = 1.f / l;
+  bf16 *out = static_cast<bf16 *>(a.out) + (((size_t)b * a.n + row) * a.H + h) * a.dv;
+  for (int q = 0; q < dvp; q += 32) {
+    uint32_t o[32];
+    tmem_ld32(o, tm_o + lane_base + q);
+    tmem_wait_ld();
+    if (row <= last) {
+#pragma unroll
+      for (int e = 0; e < 32; e += 8) {
+        if (q + e < a.dv) {  // dv % 8 == 0
+          uint4 v;
+          v.x = pack_bf16(__uint_as_float(o[e]) * inv, __uint_as_float(o[e + 1]) * inv);
+          v.y = pack_bf16(__uint_as_float(o[e + 2]) * inv, __uint_as_float(o[e + 3]) * inv);
+          v.z = pack_bf16(__uint_as_float(o[e + 4]) * inv, __uint_as_float(o[e + 5]) * inv);
+          v.w = pack_bf16(__uint_as_float(o[e + 6]) * inv, __uint_as_float(o[e + 7]) * inv);
+          *reinterpret_cast<uint4 *>(out + q + e) = v;
+        }
+      }
+    }
+    __syncwarp();
+  }
+  if (dead && tid == 0) atomicAdd(&g_window_timeouts, 1u);
+  tmem_fence_before();
+  __syncthreads();
+  if (warp == 0) tmem_dealloc(tm, COLS);
+}
+
+template <int KB, int VB>
+static int launch_window_prefill(const WindowArgs &a, cudaStream_t st) {
+  size_t smem = 1024 + (size_t)(2 * KB + VB) * WP_TILE * 128;
+  // as many blocks per multiprocessor as TMEM has room for: two, or one with wide values
+  const size_t least = (VB > 2 ? 120 : 80) * 1024;
+  if (smem < least) smem = least;
+  cudaFuncSetAttribute(window_prefill_kernel<KB, VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  djv::launch_kernel(window_prefill_kernel<KB, VB>, dim3(ceil_div(a.n, WP_TILE), a.H, a.B), dim3(WP_THREADS), smem, st,
+                     a);
+  count_launch();
+  return check_launch("window_attn");
+}
+
+bool window_prefill_supported(const WindowArgs &a) {
+  return a.dk % 8 == 0 && a.dv % 8 == 0 && a.dk <= 256 && a.dv <= 256 && a.ld % 8 == 0 && aligned16(a.qkv) &&
+         aligned16(a.k_ring) && aligned16(a.v_ring) && aligned16(a.out);
+}
+
+int window_prefill(const WindowArgs &a, cudaStream_t st) {
+  const int kb = a.dk <= 64 ? 1 : (a.dk <= 128 ? 2 : 4), vb = a.dv <= 64 ? 1 : (a.dv <= 128 ? 2 : 4);
+#define DJV_WP(K_, V_) \
+  if (kb == K_ && vb == V_) return launch_window_prefill<K_, V_>(a, st)
+  DJV_WP(1, 1);
+  DJV_WP(1, 2);
+  DJV_WP(1, 4);
+  DJV_WP(2, 1);
+  DJV_WP(2, 2);
+  DJV_WP(2, 4);
+  DJV_WP(4, 1);
+  DJV_WP(4, 2);
+  return launch_window_prefill<4, 4>(a, st);
+#undef DJV_WP
+}
+
+}  // namespace djv
+
+extern "C" unsigned djv_window_timeouts(void) {
+  unsigned v = 0;
+  if (cudaMemcpyFromSymbol(&v, djv::g_window_timeouts, sizeof(v)) != cudaSuccess) {
+    cudaGetLastError();
+    return 0;
+  }
+  return v;
+}

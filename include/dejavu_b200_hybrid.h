@@ -57,6 +57,8 @@ int djv_window_attn(int dtype, void *out, const void *qkv, long long ld, const v
                     int window, float scale, void *stream);
 int djv_window_store(int dtype, void *k_ring, void *v_ring, const void *qkv, long long ld, const long long *pos, int B,
                      int n, int H, int G, int dk, int dv, int cap, void *stream);
+/* Waits of the tensor-core kernels on their own products that ran out since load (0 in a healthy process; synchronises). */
+unsigned djv_window_timeouts(void);
 /* The decode step of the same in one kernel: rotates q and k of one token per sequence, stores k and v into the rings
  * and attends. qkv rows are not rotated yet; freqs NULL: no rotation. */
 int djv_window_attn_decode(int dtype, void *out, const void *qkv, long long ld, void *k_ring, void *v_ring,
