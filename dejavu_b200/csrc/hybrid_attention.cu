@@ -11,7 +11,7 @@
 
 #include "../../include/dejavu_b200_hybrid.h"
 #include "hybrid_attention.cuh"
-#include "mma.cuh"
+#include "dtype.cuh"
 
 namespace djv {
 
@@ -19,7 +19,7 @@ namespace cg = cooperative_groups;
 
 // ---- rotary positions ------------------------------------------------------------------------------------------
 // One block per row; the angles of the row's position are shared by its heads.
-template <typename T>
+template <typename T, bool VEC>
 __global__ void rotary_kernel(T *__restrict__ buf, long long ld, const float *__restrict__ freqs, float amp,
                               const long long *__restrict__ pos, int n, int heads, int dim, int half) {
   extern __shared__ float cs[];  // cos[half], sin[half]
@@ -35,6 +35,28 @@ __global__ void rotary_kernel(T *__restrict__ buf, long long ld, const float *__
   }
   __syncthreads();
   T *x = buf + row * ld;
+  if (VEC) {  // half is a multiple of the 16-byte chunk
+    constexpr int N = Chunk<T>::N;
+    const int per = half / N;
+    for (int k = threadIdx.x; k < heads * per; k += blockDim.x) {
+      const int h = k / per, i = (k - h * per) * N;
+      uint4 *pu = reinterpret_cast<uint4 *>(x + (size_t)h * dim + i);
+      uint4 *pv = reinterpret_cast<uint4 *>(x + (size_t)h * dim + half + i);
+      float u[N], v[N];
+      T ru[N], rv[N];
+      unpack_chunk<T>(*pu, u);
+      unpack_chunk<T>(*pv, v);
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        const float c = cs[i + e], s = cs[half + i + e];
+        ru[e] = from_f<T>(u[e] * c - v[e] * s);
+        rv[e] = from_f<T>(v[e] * c + u[e] * s);
+      }
+      *pu = *reinterpret_cast<uint4 *>(ru);
+      *pv = *reinterpret_cast<uint4 *>(rv);
+    }
+    return;
+  }
   for (int k = threadIdx.x; k < heads * half; k += blockDim.x) {
     const int h = k / half, i = k % half;
     T *e = x + (size_t)h * dim + i;
@@ -119,10 +141,10 @@ __global__ void window_store_kernel(T *__restrict__ k_ring, T *__restrict__ v_ri
 }
 
 // ---- decode ----------------------------------------------------------------------------------------------------
-// grid (G * head subgroups, B, splits); the splits of the window form a cluster, rank 0 combines them through
-// distributed shared memory. A block takes RT query heads of one kv head, so K and V are read once for all of them,
-// and streams tiles of up to `tile` tokens through shared memory: every load of a tile is in flight at once.
-constexpr int WD_THREADS = 128;
+// grid (G * head subgroups, B, splits); the splits of the window form a cluster and push their partial sums into rank
+// 0's shared memory, which combines them. A block takes RT query heads of one kv head, so K and V are read once for all
+// of them. A pass covers TILE tokens: all its K and V loads are issued before anything waits on them.
+constexpr int WD_THREADS = 256;
 constexpr int WD_MAX_SPLITS = 8;
 
 struct DecodeArgs {
@@ -130,7 +152,7 @@ struct DecodeArgs {
   void *k_ring, *v_ring;
   const float *freqs;
   float amp;
-  int half, subs, tile, k_pitch, v_pitch, vrows;  // pitches in elements; vrows: rows of V per pass of the threads
+  int half, subs;
 };
 
 // rotated element i of a head vector (fp32)
@@ -142,25 +164,34 @@ __device__ __forceinline__ float rotated(const T *x, int i, const float *cs, int
   return u;
 }
 
-template <typename T, int RT, bool VEC>
+// KL: 16-byte chunks of a key per lane (8 lanes per key); VI: 16-byte chunks of values per thread and pass.
+// KL == 0: any head size and alignment, element by element, one token of K and one column of V per thread at a time.
+template <typename T, int RT, int KL, int VI>
 __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(DecodeArgs d) {
   const WindowArgs &a = d.w;
+  constexpr bool VEC = KL > 0;
   constexpr int N = VEC ? Chunk<T>::N : 1;
-  extern __shared__ __align__(16) unsigned char sm_raw[];
-  const int dk = a.dk, dv = a.dv, tile = d.tile;
-  T *k_sm = reinterpret_cast<T *>(sm_raw);
-  T *v_sm = k_sm + (size_t)tile * d.k_pitch;
-  float *qs = reinterpret_cast<float *>(v_sm + (size_t)tile * d.v_pitch);  // RT * dk
-  float *sc = qs + RT * dk;                                               // RT * tile
-  float *cs = sc + RT * tile;                                             // 2 * half
-  float *part = cs + 2 * d.half;                                          // RT * (dv + 2): m, l, o
-  float *osum = part + RT * (dv + 2);                                     // vrows * RT * dv
+  constexpr int TILE = sizeof(T) == 2 ? 128 : 64;
+  constexpr int KT = TILE / (WD_THREADS / 8);  // keys per group of 8 lanes and pass
+  extern __shared__ __align__(16) float sm[];
+  const int dk = a.dk, dv = a.dv, ps = RT * (dv + 2);
+  float *qs = sm;                        // RT * dk
+  float *sc = qs + RT * ((dk + 3) & ~3); // RT * TILE
+  T *kn = reinterpret_cast<T *>(sc + RT * TILE);                        // the new token's rotated key
+  float *cs = reinterpret_cast<float *>(kn) + ((dk + 3) & ~3);          // 2 * half
+  float *part = cs + 2 * ((d.half + 1) & ~1);                           // splits * RT * (m, l, o[dv])
+  const int nvc = VEC ? dv / N : min(dv, WD_THREADS);
+  const int vrows = WD_THREADS / nvc;
+  float *osum = part + WD_MAX_SPLITS * ps;  // vrows * RT * dv
   __shared__ float m_run[RT], l_run[RT], corr[RT];
-  pdl_prologue();
+  cg::cluster_group cluster = cg::this_cluster();
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  const int nsplit = gridDim.z;
+  if (nsplit > 1) cluster.barrier_arrive();  // (waited for before the first access to another block's memory)
+  asm volatile("griddepcontrol.wait;" ::: "memory");
 
   const int tid = threadIdx.x, lane = tid % WARP, warp = tid / WARP;
-  const int g = blockIdx.x / d.subs, sub = blockIdx.x % d.subs, b = blockIdx.y;
-  const int sp = blockIdx.z, nsplit = gridDim.z;
+  const int g = blockIdx.x / d.subs, sub = blockIdx.x % d.subs, b = blockIdx.y, sp = blockIdx.z;
   const int rep = a.H / a.G, r0 = sub * RT, nr = min(RT, rep - r0), h0 = g * rep + r0;
   const long long p = a.pos[b];
   const T *row = static_cast<const T *>(a.qkv) + (size_t)b * a.ld;
@@ -175,6 +206,38 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(DecodeArgs d)
   const int chunk = (len + nsplit - 1) / nsplit;
   const int t_begin = min(len, sp * chunk), t_end = min(len, t_begin + chunk);
   const int slot0 = (int)(lo % a.cap);  // slot of the window's first token
+  auto slot_of = [&](int t) {
+    const int s = slot0 + t;
+    return (size_t)(s >= a.cap ? s - a.cap : s);
+  };
+
+  const int ksub = tid % 8, kgrp = tid / 8;
+  const int vch = tid % nvc, vrow = tid / nvc;
+  const bool vmine = vrow < vrows;
+  const int nkc = dk / N;
+  uint4 kreg[KT][VEC ? KL : 1], vreg[VEC ? VI : 1];
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  auto fetch = [&](int p0) {
+    if (VEC) {
+#pragma unroll
+      for (int x = 0; x < KT; ++x) {
+        const int t = p0 + x * (WD_THREADS / 8) + kgrp;
+        const uint4 *src = reinterpret_cast<const uint4 *>(kr + slot_of(t) * dk);
+#pragma unroll
+        for (int c = 0; c < KL; ++c)  // the last token of the window is not in the ring yet
+          kreg[x][c] = (t < t_end && t < len - 1 && ksub + c * 8 < nkc) ? src[ksub + c * 8] : zero;
+      }
+#pragma unroll
+      for (int x = 0; x < VI; ++x) {
+        const int i = x * vrows + vrow, t = p0 + i;
+        vreg[x] = zero;
+        if (vmine && i < TILE && t < t_end)
+          vreg[x] = t < len - 1 ? *reinterpret_cast<const uint4 *>(vr + slot_of(t) * dv + vch * N)
+                                : *reinterpret_cast<const uint4 *>(v_new + vch * N);
+      }
+    }
+  };
+  fetch(t_begin);
 
   for (int i = tid; i < d.half; i += WD_THREADS) {
     float s, c;
@@ -186,86 +249,98 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(DecodeArgs d)
     m_run[tid] = -INFINITY;
     l_run[tid] = 0.f;
   }
-  const int nkc = dk / N, nvc = dv / N;
-  const int vch = tid % nvc, vrow = tid / nvc;  // value columns of this thread, and its first row
+  __syncthreads();
+  for (int i = tid; i < RT * dk; i += WD_THREADS) {
+    const int r = i / dk;
+    qs[i] = r < nr ? to_f(from_f<T>(rotated(row + (size_t)(h0 + r) * dk, i - r * dk, cs, d.half))) : 0.f;
+  }
+  if (t_end == len && t_begin < t_end) {  // this block holds the new token: the first head subgroup stores it
+    const size_t slot = (size_t)(p % a.cap);
+    for (int i = tid; i < dk; i += WD_THREADS) {
+      const T k = from_f<T>(rotated(k_new, i, cs, d.half));
+      kn[i] = k;
+      if (sub == 0) kr[slot * dk + i] = k;
+    }
+    if (sub == 0)
+      for (int i = tid; i < dv; i += WD_THREADS) vr[slot * dv + i] = v_new[i];
+  }
+  __syncthreads();
+
   float acc[RT][N];
 #pragma unroll
   for (int r = 0; r < RT; ++r)
 #pragma unroll
     for (int e = 0; e < N; ++e) acc[r][e] = 0.f;
-  const bool wide_v = nvc > WD_THREADS;  // (element-wise form only: a thread then owns several columns, below)
 
-  for (int p0 = t_begin; p0 < t_end; p0 += tile) {
-    const int pn = min(tile, t_end - p0);
-    for (int c = tid; c < pn * nkc; c += WD_THREADS) {
-      const int t = c / nkc, j = c % nkc;
-      if (p0 + t == len - 1) continue;  // the new token is not in the ring yet
-      int slot = slot0 + p0 + t;
-      if (slot >= a.cap) slot -= a.cap;
-      if (VEC)
-        cp_async16_zfill(smem_addr(k_sm + (size_t)t * d.k_pitch + j * N), kr + (size_t)slot * dk + j * N, 16);
-      else
-        k_sm[(size_t)t * d.k_pitch + j] = kr[(size_t)slot * dk + j];
-    }
-    for (int c = tid; c < pn * nvc; c += WD_THREADS) {
-      const int t = c / nvc, j = c % nvc;
-      if (p0 + t == len - 1) continue;
-      int slot = slot0 + p0 + t;
-      if (slot >= a.cap) slot -= a.cap;
-      if (VEC)
-        cp_async16_zfill(smem_addr(v_sm + (size_t)t * d.v_pitch + j * N), vr + (size_t)slot * dv + j * N, 16);
-      else
-        v_sm[(size_t)t * d.v_pitch + j] = vr[(size_t)slot * dv + j];
-    }
-    if (VEC) cp_async_commit();
-    if (p0 == t_begin) __syncthreads();  // cs[] is complete
-    if (p0 == t_begin)
-      for (int i = tid; i < nr * dk; i += WD_THREADS)
-        qs[i] = to_f(from_f<T>(rotated(row + (size_t)(h0 + i / dk) * dk, i % dk, cs, d.half)));
-    if (p0 + pn == len) {  // this block holds the new token: the first head subgroup stores it
-      const size_t slot = (size_t)(p % a.cap);
-      for (int i = tid; i < dk; i += WD_THREADS) {
-        const T k = from_f<T>(rotated(k_new, i, cs, d.half));
-        k_sm[(size_t)(pn - 1) * d.k_pitch + i] = k;
-        if (sub == 0) kr[slot * dk + i] = k;
-      }
-      for (int i = tid; i < dv; i += WD_THREADS) {
-        v_sm[(size_t)(pn - 1) * d.v_pitch + i] = v_new[i];
-        if (sub == 0) vr[slot * dv + i] = v_new[i];
-      }
-    }
-    if (VEC) cp_async_wait<0>();
-    __syncthreads();
-    // scores: a thread per token
-    for (int t = tid; t < tile; t += WD_THREADS) {
-      float s[RT];
+  for (int p0 = t_begin; p0 < t_end; p0 += TILE) {
+    const int pn = min(TILE, t_end - p0);
+    if (VEC) {
+      if (p0 != t_begin) fetch(p0);
+      float s[KT][RT];
 #pragma unroll
-      for (int r = 0; r < RT; ++r) s[r] = 0.f;
-      if (t < pn) {
-        for (int c = 0; c < nkc; ++c) {
-          float kf[N];
-          if (VEC)
-            unpack_chunk<T>(*reinterpret_cast<const uint4 *>(k_sm + (size_t)t * d.k_pitch + c * N), kf);
-          else
-            kf[0] = to_f(k_sm[(size_t)t * d.k_pitch + c]);
+      for (int x = 0; x < KT; ++x)
 #pragma unroll
-          for (int r = 0; r < RT; ++r)
+        for (int r = 0; r < RT; ++r) s[x][r] = 0.f;
 #pragma unroll
-            for (int e = 0; e < N; ++e) s[r] = fmaf(kf[e], r < nr ? qs[r * dk + c * N + e] : 0.f, s[r]);
+      for (int c = 0; c < (VEC ? KL : 1); ++c) {
+        const int ch = ksub + c * 8;
+        if (ch >= nkc) continue;
+        float kf[KT][N];
+#pragma unroll
+        for (int x = 0; x < KT; ++x) {
+          if (p0 + x * (WD_THREADS / 8) + kgrp == len - 1) kreg[x][c] = *reinterpret_cast<const uint4 *>(kn + ch * N);
+          if constexpr (VEC) unpack_chunk<T>(kreg[x][c], kf[x]);
+        }
+#pragma unroll
+        for (int r = 0; r < RT; ++r) {
+          float qf[N];
+#pragma unroll
+          for (int e = 0; e < N; ++e) qf[e] = qs[r * dk + ch * N + e];
+#pragma unroll
+          for (int x = 0; x < KT; ++x)
+#pragma unroll
+            for (int e = 0; e < N; ++e) s[x][r] = fmaf(kf[x][e], qf[e], s[x][r]);
         }
       }
 #pragma unroll
-      for (int r = 0; r < RT; ++r) sc[r * tile + t] = t < pn ? s[r] * a.scale : -INFINITY;
+      for (int x = 0; x < KT; ++x) {
+        const int t = x * (WD_THREADS / 8) + kgrp;
+#pragma unroll
+        for (int r = 0; r < RT; ++r) {
+          float v = s[x][r];
+          v += __shfl_xor_sync(0xffffffffu, v, 4);
+          v += __shfl_xor_sync(0xffffffffu, v, 2);
+          v += __shfl_xor_sync(0xffffffffu, v, 1);
+          if (ksub == 0) sc[r * TILE + t] = t < pn ? v * a.scale : -INFINITY;
+        }
+      }
+    } else {
+      for (int i = tid; i < RT * TILE; i += WD_THREADS) {
+        const int r = i / TILE, t = i % TILE;
+        float v = -INFINITY;
+        if (t < pn && r < nr) {
+          const T *k = p0 + t == len - 1 ? kn : kr + slot_of(p0 + t) * dk;
+          v = 0.f;
+          for (int c = 0; c < dk; ++c) v = fmaf(to_f(k[c]), qs[r * dk + c], v);
+          v *= a.scale;
+        }
+        sc[i] = v;
+      }
     }
     __syncthreads();
     for (int r = warp; r < nr; r += WD_THREADS / WARP) {
-      float mx = m_run[r];
-      for (int t = lane; t < pn; t += WARP) mx = fmaxf(mx, sc[r * tile + t]);
+      float x[TILE / WARP], mx = m_run[r];
+#pragma unroll
+      for (int i = 0; i < TILE / WARP; ++i) {
+        x[i] = sc[r * TILE + i * WARP + lane];
+        mx = fmaxf(mx, x[i]);
+      }
       mx = warp_max(mx);
       float sum = 0.f;
-      for (int t = lane; t < pn; t += WARP) {
-        const float w = expf(sc[r * tile + t] - mx);
-        sc[r * tile + t] = w;
+#pragma unroll
+      for (int i = 0; i < TILE / WARP; ++i) {
+        const float w = expf(x[i] - mx);  // 0 past the end of the pass
+        sc[r * TILE + i * WARP + lane] = w;
         sum += w;
       }
       sum = warp_sum(sum);
@@ -276,132 +351,131 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(DecodeArgs d)
       }
     }
     __syncthreads();
-    if (!wide_v && vrow < d.vrows) {
-#pragma unroll
-      for (int r = 0; r < RT; ++r)
-        if (r < nr) {
-#pragma unroll
-          for (int e = 0; e < N; ++e) acc[r][e] *= corr[r];
-        }
-      for (int t = vrow; t < pn; t += d.vrows) {
-        float vf[N];
-        if (VEC)
-          unpack_chunk<T>(*reinterpret_cast<const uint4 *>(v_sm + (size_t)t * d.v_pitch + vch * N), vf);
-        else
-          vf[0] = to_f(v_sm[(size_t)t * d.v_pitch + vch]);
+    if (VEC) {
+      if (p0 != t_begin) {
 #pragma unroll
         for (int r = 0; r < RT; ++r) {
-          if (r < nr) {
-            const float w = sc[r * tile + t];
+          const float w = r < nr ? corr[r] : 0.f;
+#pragma unroll
+          for (int e = 0; e < N; ++e) acc[r][e] *= w;
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < (VEC ? VI : 1); ++x) {
+        const int i = x * vrows + vrow;
+        float vf[N];
+        if constexpr (VEC) unpack_chunk<T>(vreg[x], vf);
+        if (vmine && i < pn) {
+#pragma unroll
+          for (int r = 0; r < RT; ++r) {
+            const float w = r < nr ? sc[r * TILE + i] : 0.f;
 #pragma unroll
             for (int e = 0; e < N; ++e) acc[r][e] = fmaf(w, vf[e], acc[r][e]);
           }
         }
       }
-    } else if (wide_v) {
-      // more value columns than threads: sums live in shared memory (vrows == 1)
-      for (int j = tid; j < nvc; j += WD_THREADS)
+    } else {
+      for (int j = tid; j < dv; j += WD_THREADS)  // sums in shared memory, one thread per column
         for (int r = 0; r < nr; ++r) {
           float o = p0 == t_begin ? 0.f : osum[r * dv + j] * corr[r];
-          for (int t = 0; t < pn; ++t) o = fmaf(sc[r * tile + t], to_f(v_sm[(size_t)t * d.v_pitch + j]), o);
+          for (int t = 0; t < pn; ++t) {
+            const T *v = p0 + t == len - 1 ? v_new : vr + slot_of(p0 + t) * dv;
+            o = fmaf(sc[r * TILE + t], to_f(v[j]), o);
+          }
           osum[r * dv + j] = o;
         }
     }
-    __syncthreads();  // the tile and sc[] are reused
+    __syncthreads();  // sc[] is reused
   }
-  if (!wide_v && vrow < d.vrows) {
+  const bool empty = t_begin >= t_end;
+  if (VEC && vmine) {
 #pragma unroll
     for (int r = 0; r < RT; ++r)
 #pragma unroll
       for (int e = 0; e < N; ++e) osum[((size_t)vrow * RT + r) * dv + vch * N + e] = acc[r][e];
   }
   __syncthreads();
-  const bool empty = t_begin >= t_end;
+  if (nsplit > 1) cluster.barrier_wait();
+  float *dst = (nsplit > 1 ? cluster.map_shared_rank(part, 0) : part) + sp * ps;
   for (int i = tid; i < nr * dv; i += WD_THREADS) {
-    const int r = i / dv, j = i % dv;
+    const int r = i / dv, j = i - r * dv;
     float o = 0.f;
     if (!empty)
-      for (int v = 0; v < d.vrows; ++v) o += osum[((size_t)v * RT + r) * dv + j];
-    part[r * (dv + 2) + 2 + j] = o;
+      for (int v = 0; v < (VEC ? vrows : 1); ++v) o += osum[((size_t)v * RT + r) * dv + j];
+    dst[r * (dv + 2) + 2 + j] = o;
   }
   if (tid < nr) {
-    part[tid * (dv + 2)] = m_run[tid];
-    part[tid * (dv + 2) + 1] = l_run[tid];
+    dst[tid * (dv + 2)] = m_run[tid];
+    dst[tid * (dv + 2) + 1] = l_run[tid];
   }
-  cg::cluster_group cluster = cg::this_cluster();
   if (nsplit > 1)
     cluster.sync();
   else
     __syncthreads();
-  if (sp == 0) {
-    for (int i = tid; i < nr * dv; i += WD_THREADS) {
-      const int r = i / dv, j = i % dv;
-      const float sink = a.sink ? a.sink[h0 + r] : -INFINITY;
-      float ms[WD_MAX_SPLITS], m = sink;
+  if (sp != 0) return;
+  for (int i = tid; i < nr * dv; i += WD_THREADS) {
+    const int r = i / dv, j = i - r * dv;
+    const float sink = a.sink ? a.sink[h0 + r] : -INFINITY;
+    float ms[WD_MAX_SPLITS], m = sink;
 #pragma unroll
-      for (int s = 0; s < WD_MAX_SPLITS; ++s) {
-        ms[s] = -INFINITY;
-        if (s < nsplit) ms[s] = *(nsplit > 1 ? cluster.map_shared_rank(part + r * (dv + 2), s) : part + r * (dv + 2));
-        m = fmaxf(m, ms[s]);
-      }
-      float l = a.sink ? expf(sink - m) : 0.f, o = 0.f;
-#pragma unroll
-      for (int s = 0; s < WD_MAX_SPLITS; ++s) {
-        if (s < nsplit && ms[s] != -INFINITY) {
-          const float *q = (nsplit > 1 ? cluster.map_shared_rank(part, s) : part) + r * (dv + 2);
-          const float w = expf(ms[s] - m);
-          l = fmaf(w, q[1], l);
-          o = fmaf(w, q[2 + j], o);
-        }
-      }
-      static_cast<T *>(a.out)[((size_t)b * a.H + h0 + r) * dv + j] = from_f<T>(o / l);
+    for (int s = 0; s < WD_MAX_SPLITS; ++s) {
+      ms[s] = s < nsplit ? part[s * ps + r * (dv + 2)] : -INFINITY;
+      m = fmaxf(m, ms[s]);
     }
+    float l = a.sink ? expf(sink - m) : 0.f, o = 0.f;
+#pragma unroll
+    for (int s = 0; s < WD_MAX_SPLITS; ++s) {
+      if (s < nsplit && ms[s] != -INFINITY) {
+        const float *q = part + s * ps + r * (dv + 2);
+        const float w = expf(ms[s] - m);
+        l = fmaf(w, q[1], l);
+        o = fmaf(w, q[2 + j], o);
+      }
+    }
+    static_cast<T *>(a.out)[((size_t)b * a.H + h0 + r) * dv + j] = from_f<T>(o / l);
   }
-  if (nsplit > 1) cluster.sync();  // no block leaves while rank 0 may still read its shared memory
 }
 
-template <typename T, int RT, bool VEC>
+template <typename T, int RT, int KL, int VI>
 static int launch_decode(DecodeArgs d, int nsplit, cudaStream_t st) {
   const WindowArgs &a = d.w;
-  constexpr int N = VEC ? Chunk<T>::N : 1;
+  constexpr int TILE = sizeof(T) == 2 ? 128 : 64;
   d.subs = ceil_div(a.H / a.G, RT);
-  // an odd number of 16-byte units per row: rows of one column then fall into different banks
-  auto pitch = [](int dim) {
-    if (!VEC) return dim | 1;
-    const int units = dim / N;
-    return (units | 1) * N;
-  };
-  d.k_pitch = pitch(a.dk);
-  d.v_pitch = pitch(a.dv);
-  const int nvc = a.dv / N;
-  d.vrows = nvc > WD_THREADS ? 1 : WD_THREADS / nvc;
-  size_t smem = 0;
-  for (d.tile = 128;; d.tile /= 2) {
-    size_t kv = (size_t)d.tile * (d.k_pitch + d.v_pitch) * sizeof(T);
-    kv = (kv + 15) / 16 * 16;
-    smem = kv + 4 * ((size_t)RT * a.dk + (size_t)RT * d.tile + 2 * d.half + (size_t)RT * (a.dv + 2) +
-                     (size_t)d.vrows * RT * a.dv);
-    if (smem <= 200 * 1024) break;
-    if (d.tile == 16) {
-      set_error("window_attn_decode: head sizes %d / %d are too large", a.dk, a.dv);
-      return DJV_ERR_UNSUPPORTED;
-    }
+  const int nvc = KL > 0 ? a.dv / Chunk<T>::N : WD_THREADS;
+  const size_t dk4 = (a.dk + 3) & ~3;
+  const size_t smem = 4 * (RT * dk4 + (size_t)RT * TILE + dk4 + 2 * ((d.half + 1) & ~1) +
+                           (size_t)WD_MAX_SPLITS * RT * (a.dv + 2) + (size_t)(WD_THREADS / nvc) * RT * a.dv);
+  if (smem > 220 * 1024) {
+    set_error("window_attn_decode: head sizes %d / %d are too large", a.dk, a.dv);
+    return DJV_ERR_UNSUPPORTED;
   }
-  if (!VEC && ((size_t)d.tile * (d.k_pitch + d.v_pitch) * sizeof(T)) % 4 != 0) return DJV_ERR_UNSUPPORTED;
-  cudaFuncSetAttribute(window_decode_kernel<T, RT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-  djv::launch_kernel_cluster(window_decode_kernel<T, RT, VEC>, dim3(a.G * d.subs, a.B, nsplit), dim3(WD_THREADS), smem,
+  cudaFuncSetAttribute(window_decode_kernel<T, RT, KL, VI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+  djv::launch_kernel_cluster(window_decode_kernel<T, RT, KL, VI>, dim3(a.G * d.subs, a.B, nsplit), dim3(WD_THREADS), smem,
                              st, dim3(1, 1, nsplit), d);
   count_launch();
   return check_launch("window_attn_decode");
 }
 
-template <typename T, bool VEC>
-static int dispatch_decode(const DecodeArgs &d, int nsplit, cudaStream_t st) {
+template <typename T, int RT>
+static int dispatch_decode(const DecodeArgs &d, int nsplit, bool vec, cudaStream_t st) {
+  if (!vec) return launch_decode<T, RT, 0, 0>(d, nsplit, st);
+  constexpr int N = Chunk<T>::N, TILE = sizeof(T) == 2 ? 128 : 64;
+  const int kl = ceil_div(d.w.dk / N, 8);
+  const int vi = ceil_div(TILE, WD_THREADS / (d.w.dv / N));
+  // (the larger instance of each pair serves the sizes between)
+  if (kl <= 2 && vi <= 8) return launch_decode<T, RT, 2, 8>(d, nsplit, st);
+  if (kl <= 4 && vi <= 16) return launch_decode<T, RT, 4, 16>(d, nsplit, st);
+  if (sizeof(T) == 4 && kl <= 8 && vi <= 16) return launch_decode<T, RT, sizeof(T) == 4 ? 8 : 4, 16>(d, nsplit, st);
+  return launch_decode<T, RT, 0, 0>(d, nsplit, st);
+}
+
+template <typename T>
+static int dispatch_decode(const DecodeArgs &d, int nsplit, bool vec, cudaStream_t st) {
   const int rep = d.w.H / d.w.G;
-  if (rep == 1) return launch_decode<T, 1, VEC>(d, nsplit, st);
-  if (rep == 2) return launch_decode<T, 2, VEC>(d, nsplit, st);
-  if (rep <= 4) return launch_decode<T, 4, VEC>(d, nsplit, st);
-  return launch_decode<T, 8, VEC>(d, nsplit, st);
+  if (rep == 1) return dispatch_decode<T, 1>(d, nsplit, vec, st);
+  if (rep == 2) return dispatch_decode<T, 2>(d, nsplit, vec, st);
+  if (rep <= 4) return dispatch_decode<T, 4>(d, nsplit, vec, st);
+  return dispatch_decode<T, 8>(d, nsplit, vec, st);
 }
 
 template <typename T>
@@ -442,14 +516,21 @@ extern "C" int djv_rotary(int dtype, void *buf, long long ld, const float *freqs
                   ld >= (long long)heads * dim && (long long)B * n < (1ll << 31),
               "rotary: B=%d n=%d heads=%d dim=%d half=%d", B, n, heads, dim, half);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  int threads = ceil_div(heads * half, 4 * WARP) * WARP;
+  const int chunk = 16 / (int)dtype_bytes(dtype);
+  const bool vec = half % chunk == 0 && dim % chunk == 0 && ld % chunk == 0 && aligned16(buf);
+  int threads = ceil_div(vec ? heads * half / chunk : ceil_div(heads * half, 4), WARP) * WARP;
   threads = threads > 512 ? 512 : threads;
-  if (dtype == DJV_DTYPE_BF16)
-    djv::launch_kernel(rotary_kernel<bf16>, B * n, threads, half * 8, st, static_cast<bf16 *>(buf), ld, freqs, amp, pos,
-                       n, heads, dim, half);
-  else
-    djv::launch_kernel(rotary_kernel<float>, B * n, threads, half * 8, st, static_cast<float *>(buf), ld, freqs, amp,
-                       pos, n, heads, dim, half);
+#define DJV_ROT(T_, VEC_)                                                                                             \
+  djv::launch_kernel(rotary_kernel<T_, VEC_>, B * n, threads, half * 8, st, static_cast<T_ *>(buf), ld, freqs, amp, pos, \
+                     n, heads, dim, half)
+  if (dtype == DJV_DTYPE_BF16) {
+    if (vec) DJV_ROT(bf16, true);
+    else DJV_ROT(bf16, false);
+  } else {
+    if (vec) DJV_ROT(float, true);
+    else DJV_ROT(float, false);
+  }
+#undef DJV_ROT
   count_launch();
   return check_launch("rotary");
 }
@@ -507,10 +588,9 @@ extern "C" int djv_window_attn_decode(int dtype, void *out, const void *qkv, lon
   int nsplit = 1;
   while (nsplit < WD_MAX_SPLITS && window > 64 * nsplit) nsplit *= 2;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dtype == DJV_DTYPE_BF16) {
-    const bool vec = dk % 8 == 0 && dv % 8 == 0 && dv / 8 <= WD_THREADS && aligned16(k_ring) && aligned16(v_ring);
-    return vec ? dispatch_decode<bf16, true>(d, nsplit, st) : dispatch_decode<bf16, false>(d, nsplit, st);
-  }
-  const bool vec = dk % 4 == 0 && dv % 4 == 0 && dv / 4 <= WD_THREADS && aligned16(k_ring) && aligned16(v_ring);
-  return vec ? dispatch_decode<float, true>(d, nsplit, st) : dispatch_decode<float, false>(d, nsplit, st);
+  const int chunk = 16 / (int)dtype_bytes(dtype);
+  const bool vec = dk % chunk == 0 && dv % chunk == 0 && dv / chunk <= WD_THREADS && ld % chunk == 0 &&
+                   aligned16(qkv) && aligned16(k_ring) && aligned16(v_ring);
+  if (dtype == DJV_DTYPE_BF16) return dispatch_decode<bf16>(d, nsplit, vec, st);
+  return dispatch_decode<float>(d, nsplit, vec, st);
 }

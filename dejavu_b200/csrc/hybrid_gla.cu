@@ -7,32 +7,16 @@
 //   S_out[c, :] = exp(B_C[c]) S_in[c, :] + sum_s k_s[c] exp(B_C[c] - B_s[c]) v_s
 // All exponents are <= 0, whatever the decays are. Three kernels: every chunk's own contribution to the state (chunks
 // in parallel), a scan over the chunks that turns contributions into incoming states, every chunk's outputs (in
-// parallel, norm and gate included).
+// parallel, norm and gate included). The kernels here do the chunks' products in fp32 on the CUDA cores, for any head
+// size and both element types; the tensor-core form for bf16 is in hybrid_gla_mma.cu.
 #include <cooperative_groups.h>
 
 #include "../../include/dejavu_b200_hybrid.h"
-#include "mma.cuh"
+#include "hybrid_gla.cuh"
 
 namespace djv {
 
 namespace cg = cooperative_groups;
-
-constexpr int GLA_THREADS = 256;
-
-struct GlaArgs {
-  void *out;
-  const void *proj;
-  long long ld;
-  const float *a2, *a2_bias, *norm;
-  float inv_tau, eps, scale;
-  float *state;
-  const long long *pos;
-  int B, n, H, dk, dv, rank;
-  int C, nc;      // chunk length, number of chunks
-  float *contrib; // (B, H, nc, dk, dv): contributions, then incoming states
-  float *decay;   // (B, H, nc, dk): B_C
-  float *cum;     // (B*n, H, dk): B_t
-};
 
 // log of the decay of channel c (in 0 .. H*dk) from the low-rank activations of one token
 template <typename T>
@@ -113,11 +97,22 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_state_scan_kernel(GlaArgs a) 
   float s = a.pos[b] == 0 ? 0.f : a.state[bh * per + e];
   float *U = a.contrib + bh * a.nc * per + e;
   const float *D = a.decay + bh * a.nc * a.dk + e / a.dv;
-#pragma unroll 4
-  for (int c = 0; c < a.nc; ++c) {
-    const float u = U[(size_t)c * per], d = expf(D[(size_t)c * a.dk]);
-    U[(size_t)c * per] = s;
-    s = fmaf(d, s, u);
+  constexpr int U8 = 8;  // chunks whose loads are in flight together
+  for (int c0 = 0; c0 < a.nc; c0 += U8) {
+    float u[U8], d[U8];
+#pragma unroll
+    for (int c = 0; c < U8; ++c) {
+      const bool ok = c0 + c < a.nc;
+      u[c] = ok ? U[(size_t)(c0 + c) * per] : 0.f;
+      d[c] = ok ? D[(size_t)(c0 + c) * a.dk] : 0.f;
+    }
+#pragma unroll
+    for (int c = 0; c < U8; ++c) {
+      if (c0 + c < a.nc) {
+        U[(size_t)(c0 + c) * per] = s;
+        s = fmaf(expf(d[c]), s, u[c]);
+      }
+    }
   }
   a.state[bh * per + e] = s;
 }
@@ -213,62 +208,86 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_chunk_out_kernel(GlaArgs a) {
 
 // ---- decode: one token per sequence ------------------------------------------------------------------------------
 // grid (column blocks, H, B), a cluster over the column blocks of a head (the norm needs all of dv). A block reads,
-// updates and writes its (dk, columns) part of the state once.
+// updates and writes its (dk, columns) part of the state once; the first batch of state loads is in flight while the
+// decays are computed, and the decay weights are fetched before the kernel waits for its predecessor.
 constexpr int GD_THREADS = 128;
 constexpr int GD_MAX_BLOCKS = 8;
+constexpr int GD_ROWS = 8;  // state rows of a thread per batch of loads
 
 template <typename T, int V>
 __global__ void __launch_bounds__(GD_THREADS) gla_decode_kernel(GlaArgs a, int cols) {
   extern __shared__ float sm[];
   __shared__ float red[GD_THREADS / WARP];
-  __shared__ float ss_s;
-  pdl_prologue();
+  __shared__ float ss_all[GD_MAX_BLOCKS];
   const int tid = threadIdx.x;
-  const int cb = blockIdx.x, h = blockIdx.y, b = blockIdx.z, dk = a.dk, dv = a.dv;
+  const int cb = blockIdx.x, h = blockIdx.y, b = blockIdx.z, dk = a.dk, dv = a.dv, nb = gridDim.x;
   const int j0 = cb * cols, jn = max(0, min(cols, dv - j0));
-  float *q = sm, *k = q + dk, *al = k + dk, *osum = al + dk;  // osum: [row groups][cols]
+  const int wp = a.rank + 1;
+  float *q = sm, *k = q + dk, *al = k + dk, *w = al + dk, *osum = w + dk * wp;  // osum: [row groups][cols]
+  cg::cluster_group cluster = cg::this_cluster();
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  if (nb > 1) cluster.barrier_arrive();  // (waited for before the first access to another block's memory)
+  for (int i = tid; i < dk * a.rank; i += GD_THREADS)
+    w[i / a.rank * wp + i % a.rank] = a.a2[(size_t)h * dk * a.rank + i];
+  asm volatile("griddepcontrol.wait;" ::: "memory");
   const T *row = static_cast<const T *>(a.proj) + (size_t)b * a.ld;
   const T *v = row + 2 * a.H * dk + h * dv + j0, *gate = v + a.H * dv;
   const T *tr = row + 2 * a.H * dk + 2 * a.H * dv;
+  const bool fresh = a.pos[b] == 0;
+  float *S = a.state + ((size_t)b * a.H + h) * dk * dv + j0;
+  const int groups = jn / V;                                  // column groups (V divides cols and dv)
+  const int rows = max(1, GD_THREADS / max(1, groups));       // row groups
+  const int cg0 = tid % max(1, groups) * V, r = tid / max(1, groups);
+  const bool mine = r < rows && groups > 0;
+  float st[GD_ROWS][V];
+  auto fetch = [&](int c0) {
+#pragma unroll
+    for (int x = 0; x < GD_ROWS; ++x) {
+      const int c = c0 + x * rows;
+      const bool ok = mine && c < dk && !fresh;
+      const float *p = S + (size_t)c * dv + cg0;
+      if (V == 4) {
+        float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (ok) t = *reinterpret_cast<const float4 *>(p);
+        st[x][0] = t.x; st[x][1 % V] = t.y; st[x][2 % V] = t.z; st[x][3 % V] = t.w;
+      } else {
+        st[x][0] = ok ? p[0] : 0.f;
+      }
+    }
+  };
+  fetch(r);
+  __syncthreads();  // w[] is complete
   for (int c = tid; c < dk; c += GD_THREADS) {
     q[c] = to_f(row[h * dk + c]) * a.scale;
     k[c] = to_f(row[a.H * dk + h * dk + c]);
-    al[c] = expf(log_decay(tr, a.a2 + (size_t)(h * dk + c) * a.rank, a.a2_bias + h * dk + c, a.rank, a.inv_tau));
+    al[c] = expf(log_decay(tr, w + c * wp, a.a2_bias + h * dk + c, a.rank, a.inv_tau));
   }
   __syncthreads();
-  const bool fresh = a.pos[b] == 0;
-  float *S = a.state + ((size_t)b * a.H + h) * dk * dv + j0;
-  const int groups = jn / V;                                    // column groups (V divides cols and dv)
-  const int rows = groups ? max(1, GD_THREADS / groups) : 1;    // row groups
-  for (int gi = tid; gi < groups * rows; gi += GD_THREADS) {
-    const int cg0 = gi % groups * V, r = gi / groups;
-    float vv[V], acc[V];
+  float vv[V], acc[V];
 #pragma unroll
-    for (int e = 0; e < V; ++e) {
-      vv[e] = to_f(v[cg0 + e]);
-      acc[e] = 0.f;
-    }
-#pragma unroll 4
-    for (int c = r; c < dk; c += rows) {
-      float s[V];
+  for (int e = 0; e < V; ++e) {
+    vv[e] = mine ? to_f(v[cg0 + e]) : 0.f;
+    acc[e] = 0.f;
+  }
+  for (int c0 = r; c0 < dk; c0 += GD_ROWS * rows) {
+    if (c0 != r) fetch(c0);
+#pragma unroll
+    for (int x = 0; x < GD_ROWS; ++x) {
+      const int c = c0 + x * rows;
+      if (!mine || c >= dk) continue;
       float *p = S + (size_t)c * dv + cg0;
-      if (V == 4) {
-        float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (!fresh) t = *reinterpret_cast<const float4 *>(p);
-        s[0] = t.x; s[1 % V] = t.y; s[2 % V] = t.z; s[3 % V] = t.w;
-      } else {
-        s[0] = fresh ? 0.f : p[0];
-      }
 #pragma unroll
       for (int e = 0; e < V; ++e) {
-        s[e] = fmaf(k[c], vv[e], al[c] * s[e]);
-        acc[e] = fmaf(q[c], s[e], acc[e]);
+        st[x][e] = fmaf(k[c], vv[e], al[c] * st[x][e]);
+        acc[e] = fmaf(q[c], st[x][e], acc[e]);
       }
       if (V == 4)
-        *reinterpret_cast<float4 *>(p) = make_float4(s[0], s[1 % V], s[2 % V], s[3 % V]);
+        *reinterpret_cast<float4 *>(p) = make_float4(st[x][0], st[x][1 % V], st[x][2 % V], st[x][3 % V]);
       else
-        p[0] = s[0];
+        p[0] = st[x][0];
     }
+  }
+  if (mine) {
 #pragma unroll
     for (int e = 0; e < V; ++e) osum[r * cols + cg0 + e] = acc[e];
   }
@@ -276,33 +295,29 @@ __global__ void __launch_bounds__(GD_THREADS) gla_decode_kernel(GlaArgs a, int c
   float ss = 0.f;
   for (int j = tid; j < jn; j += GD_THREADS) {
     float o = 0.f;
-    for (int r = 0; r < rows; ++r) o += osum[r * cols + j];
+    for (int x = 0; x < rows; ++x) o += osum[x * cols + j];
     osum[j] = o;  // row group 0's slot of the same column, read by this thread only
     ss = fmaf(o, o, ss);
   }
   ss = warp_sum(ss);
   if (tid % WARP == 0) red[tid / WARP] = ss;
   __syncthreads();
-  if (tid == 0) {
-    float t = 0.f;
-    for (int w = 0; w < GD_THREADS / WARP; ++w) t += red[w];
-    ss_s = t;
-  }
-  cg::cluster_group cluster = cg::this_cluster();
-  const int nb = gridDim.x;
-  if (nb > 1)
-    cluster.sync();
-  else
-    __syncthreads();
   float tot = 0.f;
-  for (int i = 0; i < nb; ++i) tot += nb > 1 ? *cluster.map_shared_rank(&ss_s, i) : ss_s;
+#pragma unroll
+  for (int x = 0; x < GD_THREADS / WARP; ++x) tot += red[x];
+  if (nb > 1) {
+    cluster.barrier_wait();
+    if (tid < nb) cluster.map_shared_rank(ss_all, tid)[cb] = tot;  // this block's sum to every block
+    cluster.sync();
+    tot = 0.f;
+    for (int x = 0; x < nb; ++x) tot += ss_all[x];
+  }
   const float rn = 1.f / sqrtf(tot / (float)dv + a.eps);
   T *out = static_cast<T *>(a.out) + ((size_t)b * a.H + h) * dv + j0;
   for (int j = tid; j < jn; j += GD_THREADS) {
     const float g = to_f(gate[j]);
     out[j] = from_f<T>(osum[j] * rn * a.norm[j0 + j] * (g * sigmoid_f(g)));
   }
-  if (nb > 1) cluster.sync();  // no block leaves while another may still read its sum
 }
 
 // ---- host ----------------------------------------------------------------------------------------------------------
@@ -322,17 +337,32 @@ static int chunk_len(int dk, int dv) {
 }
 static size_t al256(size_t v) { return (v + 255) / 256 * 256; }
 
+// the tensor-core chunk kernels also need rows that 16-byte copies can read
+static bool use_mma(int dtype, const GlaArgs &a) {
+  return gla_mma_supported(dtype, a.dk, a.dv) && a.ld % 8 == 0 && aligned16(a.proj) && aligned16(a.out) &&
+         aligned16(a.norm);
+}
+
 template <typename T>
-static int launch_prefill(const GlaArgs &a, cudaStream_t st) {
+static int launch_prefill(const GlaArgs &a, bool mma, cudaStream_t st) {
   const size_t s1 = state_smem(a.C, a.dk, a.dv), s3 = out_smem(a.C, a.dk, a.dv);
-  cudaFuncSetAttribute(gla_chunk_state_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GLA_SMEM);
-  cudaFuncSetAttribute(gla_chunk_out_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GLA_SMEM);
   const dim3 grid(a.nc, a.H, a.B);
-  djv::launch_kernel(gla_chunk_state_kernel<T>, grid, dim3(GLA_THREADS), s1, st, a);
+  int rc = DJV_OK;
+  if (mma) {
+    rc = gla_mma_chunk_state(a, st);
+  } else {
+    cudaFuncSetAttribute(gla_chunk_state_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GLA_SMEM);
+    djv::launch_kernel(gla_chunk_state_kernel<T>, grid, dim3(GLA_THREADS), s1, st, a);
+    count_launch();
+  }
+  if (rc) return rc;
   djv::launch_kernel(gla_state_scan_kernel, dim3(ceil_div(a.dk * a.dv, GLA_THREADS), a.H, a.B), dim3(GLA_THREADS), 0, st,
                      a);
+  count_launch();
+  if (mma) return gla_mma_chunk_out(a, st);
+  cudaFuncSetAttribute(gla_chunk_out_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GLA_SMEM);
   djv::launch_kernel(gla_chunk_out_kernel<T>, grid, dim3(GLA_THREADS), s3, st, a);
-  count_launch(3);
+  count_launch();
   return check_launch("gla_prefill");
 }
 
@@ -350,8 +380,8 @@ static int launch_gla_decode(const GlaArgs &a, cudaStream_t st) {
   const int last = a.dv - (nb - 1) * cols;
   const int last_rows = GD_THREADS / (last / V > 0 ? last / V : 1) > 1 ? GD_THREADS / (last / V > 0 ? last / V : 1) : 1;
   if ((size_t)last_rows * cols > osum) osum = (size_t)last_rows * cols;
-  const size_t smem = 4 * ((size_t)3 * a.dk + osum);
-  DJV_REQUIRE(smem <= 200 * 1024, "gla_decode: head sizes %d / %d are too large", a.dk, a.dv);
+  const size_t smem = 4 * ((size_t)a.dk * (3 + a.rank + 1) + osum);
+  DJV_REQUIRE(smem <= 200 * 1024, "gla_decode: head sizes %d / %d, rank %d are too large", a.dk, a.dv, a.rank);
   const dim3 grid(nb, a.H, a.B), cluster(nb, 1, 1);
   if (vec) {
     cudaFuncSetAttribute(gla_decode_kernel<T, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
@@ -379,9 +409,9 @@ static int check_gla(const char *op, int dtype, const GlaArgs &a) {
 }
 
 extern "C" size_t djv_gla_scratch_bytes(int dtype, int B, int n, int H, int dk, int dv) {
-  (void)dtype;
   if (B < 1 || n < 1 || H < 1 || dk < 1 || dv < 1) return 0;
-  const int C = chunk_len(dk, dv);
+  int C = chunk_len(dk, dv);
+  if (gla_mma_supported(dtype, dk, dv) && (C == 0 || C > GLA_MMA_CHUNK)) C = GLA_MMA_CHUNK;
   if (C == 0) return 0;
   const size_t nc = ceil_div(n, C), bh = (size_t)B * H;
   return al256(bh * nc * dk * dv * 4) + al256(bh * nc * dk * 4) + al256(bh * n * dk * 4);
@@ -395,7 +425,8 @@ extern "C" int djv_gla_prefill(int dtype, void *out, const void *proj, long long
             nullptr, nullptr};
   int rc = check_gla("gla_prefill", dtype, a);
   if (rc) return rc;
-  a.C = chunk_len(dk, dv);
+  const bool mma = use_mma(dtype, a);
+  a.C = mma ? GLA_MMA_CHUNK : chunk_len(dk, dv);
   if (a.C == 0) {
     set_error("gla_prefill: head sizes %d / %d are too large", dk, dv);
     return DJV_ERR_UNSUPPORTED;
@@ -414,7 +445,7 @@ extern "C" int djv_gla_prefill(int dtype, void *out, const void *proj, long long
   p += al256(bh * a.nc * dk * 4);
   a.cum = reinterpret_cast<float *>(p);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return dtype == DJV_DTYPE_BF16 ? launch_prefill<bf16>(a, st) : launch_prefill<float>(a, st);
+  return dtype == DJV_DTYPE_BF16 ? launch_prefill<bf16>(a, mma, st) : launch_prefill<float>(a, false, st);
 }
 
 extern "C" int djv_gla_decode(int dtype, void *out, const void *proj, long long ld, const float *a2,

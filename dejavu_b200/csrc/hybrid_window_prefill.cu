@@ -12,6 +12,8 @@
 #include "hybrid_attention.cuh"
 #include "tcgen05.cuh"
 
+#include <type_traits>
+
 namespace djv {
 
 constexpr int WP_THREADS = 128;
@@ -23,6 +25,31 @@ __device__ __forceinline__ float exp2_approx(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// pairs of floats: one instruction for two
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+  uint64_t v;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(lo), "f"(hi));
+  return v;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float &lo, float &hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ uint64_t sub2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("sub.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
 }
 
 template <int KB, int VB>  // 64-element blocks of a query/key row and of a value row
@@ -60,27 +87,42 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
   const int tiles = (last - lo) / WP_TILE + 1;
   const int ring_slot0 = (int)((p0 - reach) % a.cap);  // slot of token -reach
 
-  auto load = [&](uint32_t dst, int j0, const bf16 *ring, int dim, const bf16 *fresh, int blocks) {
-    const int per_row = blocks * 8;  // chunks, a power of two
-    const int ch = tid & (per_row - 1);
+  // One tile of keys or values. The chunk a thread copies is the same in every row, so a tile of the portion's own
+  // tokens is a pointer that advances by a fixed number of rows.
+  auto load = [&](uint32_t dst, int j0, const bf16 *ring, int dim, const bf16 *fresh, auto blocks) {
+    constexpr int PER_ROW = decltype(blocks)::value * 8, STEP = WP_THREADS / PER_ROW;
+    const int ch = tid & (PER_ROW - 1), r0 = tid / PER_ROW;
     const bool inside = ch * 8 < dim;
-    for (int r = tid / per_row; r < WP_TILE; r += WP_THREADS / per_row) {
-      const int j = j0 + r;
-      const bf16 *src = fresh;
-      bool ok = inside && j <= last;
-      if (ok) {
-        if (j >= 0) {
-          src = fresh + (size_t)j * a.ld + ch * 8;
-        } else {
-          int slot = ring_slot0 + (j + (int)reach);
-          if (slot >= a.cap) slot -= a.cap;
-          src = ring + (size_t)slot * dim + ch * 8;
-        }
+    if (j0 >= 0 && j0 + WP_TILE - 1 <= last) {
+      const bf16 *src = fresh + (size_t)(j0 + r0) * a.ld + ch * 8;
+      const size_t step = (size_t)STEP * a.ld;
+      if (!inside) src = fresh;  // (not read)
+#pragma unroll
+      for (int it = 0; it < PER_ROW; ++it) {
+        cp_async16_zfill(dst + sw128_offset(WP_TILE, r0 + it * STEP, ch), src, inside ? 16 : 0);
+        if (inside) src += step;
       }
-      cp_async16_zfill(dst + sw128_offset(WP_TILE, r, ch), src, ok ? 16 : 0);
+    } else {
+      for (int r = r0; r < WP_TILE; r += STEP) {
+        const int j = j0 + r;
+        const bf16 *src = fresh;
+        const bool ok = inside && j <= last;
+        if (ok) {
+          if (j >= 0) {
+            src = fresh + (size_t)j * a.ld + ch * 8;
+          } else {
+            int slot = ring_slot0 + (j + (int)reach);
+            if (slot >= a.cap) slot -= a.cap;
+            src = ring + (size_t)slot * dim + ch * 8;
+          }
+        }
+        cp_async16_zfill(dst + sw128_offset(WP_TILE, r, ch), src, ok ? 16 : 0);
+      }
     }
     cp_async_commit();
   };
+  const std::integral_constant<int, KB> kb;
+  const std::integral_constant<int, VB> vb;
   const bf16 *k_new = rows + (size_t)(a.H + g) * a.dk;
   const bf16 *v_new = rows + (size_t)(a.H + a.G) * a.dk + (size_t)g * a.dv;
   {  // queries
@@ -92,7 +134,7 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
                        ok ? rows + (size_t)(t0 + r) * a.ld + (size_t)h * a.dk + ch * 8 : rows, ok ? 16 : 0);
     }
   }
-  load(k_sm, lo, kr, a.dk, k_new, KB);
+  load(k_sm, lo, kr, a.dk, k_new, kb);
 
   const float sink = a.sink ? a.sink[h] * 1.4426950408889634f : 0.f;
   const float c = a.scale * 1.4426950408889634f;  // scores in units of log 2
@@ -125,11 +167,11 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
         mma_ss(tm_s, desc_k_major(q_sm, WP_TILE, k), desc_k_major(k_sm, WP_TILE, k), idesc_s, k > 0);
       mma_commit(&bar_s);
     }
-    load(v_sm, j0, vr, a.dv, v_new, VB);
+    load(v_sm, j0, vr, a.dv, v_new, vb);
     if (!dead) dead = !mbar_wait(&bar_s, i & 1);
     __syncwarp();
     tmem_fence_after();
-    if (i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, KB);
+    if (i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, kb);
 
     __syncwarp();
     uint32_t s[4][32];
@@ -184,20 +226,34 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
       }
     }
     const float nm = -m;
+    const uint64_t ca2 = pack2(ca, ca), nm2 = pack2(nm, nm);
+    uint64_t l2 = 0;
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
       uint32_t hi[16], lw[16];
 #pragma unroll
       for (int e = 0; e < 16; ++e) {
-        const float x = exp2_approx(fmaf(__uint_as_float(s[q][2 * e]), ca, nm));
-        const float y = exp2_approx(fmaf(__uint_as_float(s[q][2 * e + 1]), ca, nm));
-        l += x + y;
-        hi[e] = pack_bf16(x, y);
-        const float2 r = b2f(hi[e]);
-        lw[e] = pack_bf16(x - r.x, y - r.y);
+        float x, y;
+        unpack2(fma2(pack2(__uint_as_float(s[q][2 * e]), __uint_as_float(s[q][2 * e + 1])), ca2, nm2), x, y);
+        x = exp2_approx(x);
+        y = exp2_approx(y);
+        const uint64_t p = pack2(x, y);
+        l2 = add2(l2, p);
+        // hi: the upper halves; the rest, which a float holds exactly, is rounded to bf16
+        hi[e] = __byte_perm(__float_as_uint(x), __float_as_uint(y), 0x7632);
+        const uint64_t top = pack2(__uint_as_float(__float_as_uint(x) & 0xffff0000u),
+                                   __uint_as_float(__float_as_uint(y) & 0xffff0000u));
+        float rx, ry;
+        unpack2(sub2(p, top), rx, ry);
+        lw[e] = pack_bf16(rx, ry);
       }
       tmem_st16(tm_s + lane_base + q * 16, hi);
       tmem_st16(tm_s + lane_base + 64 + q * 16, lw);
+    }
+    {
+      float x, y;
+      unpack2(l2, x, y);
+      l += x + y;
     }
     tmem_wait_st();
     tmem_fence_before();
