@@ -155,12 +155,11 @@ struct DecodeArgs {
   int half, subs;
 };
 
-// rotated element i of a head vector (fp32)
-template <typename T>
-__device__ __forceinline__ float rotated(const T *x, int i, const float *cs, int half) {
-  const float u = to_f(x[i]);
-  if (i < half) return u * cs[i] - to_f(x[i + half]) * cs[half + i];
-  if (i < 2 * half) return u * cs[i - half] + to_f(x[i - half]) * cs[i];
+// rotated element i of a head vector
+__device__ __forceinline__ float rotated(const float *x, int i, const float *cs, int half) {
+  const float u = x[i];
+  if (i < half) return u * cs[i] - x[i + half] * cs[half + i];
+  if (i < 2 * half) return u * cs[i - half] + x[i - half] * cs[i];
   return u;
 }
 
@@ -179,7 +178,8 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(DecodeArgs d)
   float *sc = qs + RT * ((dk + 3) & ~3); // RT * TILE
   T *kn = reinterpret_cast<T *>(sc + RT * TILE);                        // the new token's rotated key
   float *cs = reinterpret_cast<float *>(kn) + ((dk + 3) & ~3);          // 2 * half
-  float *part = cs + 2 * ((d.half + 1) & ~1);                           // splits * RT * (m, l, o[dv])
+  float *raw = cs + 2 * ((d.half + 1) & ~1);                            // the heads' queries and the key, not rotated
+  float *part = raw + (RT + 1) * dk;                                    // splits * RT * (m, l, o[dv])
   const int nvc = VEC ? dv / N : min(dv, WD_THREADS);
   const int vrows = WD_THREADS / nvc;
   float *osum = part + WD_MAX_SPLITS * ps;  // vrows * RT * dv
@@ -238,6 +238,8 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(DecodeArgs d)
     }
   };
   fetch(t_begin);
+  for (int i = tid; i < nr * dk; i += WD_THREADS) raw[i] = to_f(row[(size_t)h0 * dk + i]);
+  for (int i = tid; i < dk; i += WD_THREADS) raw[RT * dk + i] = to_f(k_new[i]);
 
   for (int i = tid; i < d.half; i += WD_THREADS) {
     float s, c;
@@ -252,12 +254,12 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(DecodeArgs d)
   __syncthreads();
   for (int i = tid; i < RT * dk; i += WD_THREADS) {
     const int r = i / dk;
-    qs[i] = r < nr ? to_f(from_f<T>(rotated(row + (size_t)(h0 + r) * dk, i - r * dk, cs, d.half))) : 0.f;
+    qs[i] = r < nr ? to_f(from_f<T>(rotated(raw + r * dk, i - r * dk, cs, d.half))) : 0.f;
   }
   if (t_end == len && t_begin < t_end) {  // this block holds the new token: the first head subgroup stores it
     const size_t slot = (size_t)(p % a.cap);
     for (int i = tid; i < dk; i += WD_THREADS) {
-      const T k = from_f<T>(rotated(k_new, i, cs, d.half));
+      const T k = from_f<T>(rotated(raw + RT * dk, i, cs, d.half));
       kn[i] = k;
       if (sub == 0) kr[slot * dk + i] = k;
     }
@@ -443,7 +445,7 @@ static int launch_decode(DecodeArgs d, int nsplit, cudaStream_t st) {
   d.subs = ceil_div(a.H / a.G, RT);
   const int nvc = KL > 0 ? a.dv / Chunk<T>::N : WD_THREADS;
   const size_t dk4 = (a.dk + 3) & ~3;
-  const size_t smem = 4 * (RT * dk4 + (size_t)RT * TILE + dk4 + 2 * ((d.half + 1) & ~1) +
+  const size_t smem = 4 * (RT * dk4 + (size_t)RT * TILE + dk4 + 2 * ((d.half + 1) & ~1) + (size_t)(RT + 1) * a.dk +
                            (size_t)WD_MAX_SPLITS * RT * (a.dv + 2) + (size_t)(WD_THREADS / nvc) * RT * a.dv);
   if (smem > 220 * 1024) {
     set_error("window_attn_decode: head sizes %d / %d are too large", a.dk, a.dv);
@@ -471,10 +473,14 @@ static int dispatch_decode(const DecodeArgs &d, int nsplit, bool vec, cudaStream
 
 template <typename T>
 static int dispatch_decode(const DecodeArgs &d, int nsplit, bool vec, cudaStream_t st) {
+  // query heads per block: few while the blocks of all of them still fit the device at once (K and V then come from L2
+  // for the second and later blocks of a kv head), all of a kv head's otherwise
   const int rep = d.w.H / d.w.G;
-  if (rep == 1) return dispatch_decode<T, 1>(d, nsplit, vec, st);
-  if (rep == 2) return dispatch_decode<T, 2>(d, nsplit, vec, st);
-  if (rep <= 4) return dispatch_decode<T, 4>(d, nsplit, vec, st);
+  int rt = 1;
+  while (rt < 8 && rt < rep && (long long)d.w.G * ceil_div(rep, rt) * d.w.B * nsplit > sm_count()) rt *= 2;
+  if (rt == 1) return dispatch_decode<T, 1>(d, nsplit, vec, st);
+  if (rt == 2) return dispatch_decode<T, 2>(d, nsplit, vec, st);
+  if (rt == 4) return dispatch_decode<T, 4>(d, nsplit, vec, st);
   return dispatch_decode<T, 8>(d, nsplit, vec, st);
 }
 

@@ -86,35 +86,57 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_chunk_state_kernel(GlaArgs a)
   }
 }
 
-// contributions -> incoming states, one thread per state element, chunks in order
+// contributions -> incoming states, V neighbouring state elements of one row per thread, chunks in order
+template <int V>
 __global__ void __launch_bounds__(GLA_THREADS) gla_state_scan_kernel(GlaArgs a) {
   pdl_prologue();
   const int per = a.dk * a.dv;
-  const int e = blockIdx.x * GLA_THREADS + threadIdx.x;
+  const int e = (blockIdx.x * GLA_THREADS + threadIdx.x) * V;
   const int h = blockIdx.y, b = blockIdx.z;
   if (e >= per) return;
   const size_t bh = (size_t)b * a.H + h;
-  float s = a.pos[b] == 0 ? 0.f : a.state[bh * per + e];
+  auto get = [](const float *p, float (&v)[V]) {
+    if (V == 4) {
+      const float4 t = *reinterpret_cast<const float4 *>(p);
+      v[0] = t.x; v[1 % V] = t.y; v[2 % V] = t.z; v[3 % V] = t.w;
+    } else {
+      v[0] = *p;
+    }
+  };
+  auto put = [](float *p, const float (&v)[V]) {
+    if (V == 4)
+      *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
+    else
+      *p = v[0];
+  };
+  float s[V];
+#pragma unroll
+  for (int v = 0; v < V; ++v) s[v] = 0.f;
+  if (a.pos[b] != 0) get(a.state + bh * per + e, s);
   float *U = a.contrib + bh * a.nc * per + e;
   const float *D = a.decay + bh * a.nc * a.dk + e / a.dv;
-  constexpr int U8 = 8;  // chunks whose loads are in flight together
-  for (int c0 = 0; c0 < a.nc; c0 += U8) {
-    float u[U8], d[U8];
+  constexpr int CH = 8;  // chunks whose loads are in flight together
+  for (int c0 = 0; c0 < a.nc; c0 += CH, U += (size_t)CH * per, D += CH * a.dk) {
+    const int cn = min(CH, a.nc - c0);
+    float u[CH][V], d[CH];
 #pragma unroll
-    for (int c = 0; c < U8; ++c) {
-      const bool ok = c0 + c < a.nc;
-      u[c] = ok ? U[(size_t)(c0 + c) * per] : 0.f;
-      d[c] = ok ? D[(size_t)(c0 + c) * a.dk] : 0.f;
+    for (int c = 0; c < CH; ++c) {
+      if (c < cn) {
+        get(U + (size_t)c * per, u[c]);
+        d[c] = D[c * a.dk];
+      }
     }
 #pragma unroll
-    for (int c = 0; c < U8; ++c) {
-      if (c0 + c < a.nc) {
-        U[(size_t)(c0 + c) * per] = s;
-        s = fmaf(expf(d[c]), s, u[c]);
+    for (int c = 0; c < CH; ++c) {
+      if (c < cn) {
+        put(U + (size_t)c * per, s);
+        const float f = expf(d[c]);
+#pragma unroll
+        for (int v = 0; v < V; ++v) s[v] = fmaf(f, s[v], u[c][v]);
       }
     }
   }
-  a.state[bh * per + e] = s;
+  put(a.state + bh * per + e, s);
 }
 
 template <typename T>
@@ -356,8 +378,12 @@ static int launch_prefill(const GlaArgs &a, bool mma, cudaStream_t st) {
     count_launch();
   }
   if (rc) return rc;
-  djv::launch_kernel(gla_state_scan_kernel, dim3(ceil_div(a.dk * a.dv, GLA_THREADS), a.H, a.B), dim3(GLA_THREADS), 0, st,
-                     a);
+  if (a.dv % 4 == 0 && aligned16(a.state))
+    djv::launch_kernel(gla_state_scan_kernel<4>, dim3(ceil_div(a.dk * a.dv, 4 * GLA_THREADS), a.H, a.B),
+                       dim3(GLA_THREADS), 0, st, a);
+  else
+    djv::launch_kernel(gla_state_scan_kernel<1>, dim3(ceil_div(a.dk * a.dv, GLA_THREADS), a.H, a.B), dim3(GLA_THREADS),
+                       0, st, a);
   count_launch();
   if (mma) return gla_mma_chunk_out(a, st);
   cudaFuncSetAttribute(gla_chunk_out_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GLA_SMEM);

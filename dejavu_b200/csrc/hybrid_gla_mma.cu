@@ -28,13 +28,21 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
 // rows x cols of bf16 from global (row stride ld) into shared memory, zeros up to pad_rows / pad_cols. 16-byte chunks.
 __device__ __forceinline__ void stage_rows(bf16 *dst, int pitch, const bf16 *src, long long ld, int rows, int cols,
                                            int pad_cols) {
-  const int chunks = pad_cols / 8;
-  for (int i = threadIdx.x; i < GC * chunks; i += GLA_THREADS) {
-    const int r = i / chunks, c = i - r * chunks;
-    const bool ok = r < rows && c * 8 < cols;
-    cp_async16_zfill(smem_addr(dst + r * pitch + c * 8), ok ? src + (size_t)r * ld + c * 8 : src, ok ? 16 : 0);
+  const int chunks = pad_cols / 8, step = GLA_THREADS / chunks;  // (pad_cols <= 256)
+  const int r0 = threadIdx.x / chunks, c = threadIdx.x - r0 * chunks;
+  if (r0 >= step) return;
+  const bool inside = c * 8 < cols;
+  const bf16 *s = src + (size_t)r0 * ld + c * 8;
+  uint32_t d = smem_addr(dst + r0 * pitch + c * 8);
+  for (int r = r0; r < GC; r += step, s += (size_t)step * ld, d += step * pitch * 2) {
+    const bool ok = inside && r < rows;
+    cp_async16_zfill(d, ok ? s : src, ok ? 16 : 0);
   }
 }
+
+// exp, log and sigmoid on the fast units: absolute errors near 2^-23, for quantities that end in bf16 products
+__device__ __forceinline__ float log_sigmoid_fast(float z) { return fminf(z, 0.f) - __logf(1.f + __expf(-fabsf(z))); }
+__device__ __forceinline__ float silu_fast(float g) { return __fdividef(g, 1.f + __expf(-g)); }
 
 // ---- a chunk's own contribution to the state: U = sum_t (k_t exp(B_C - B_t)) v_t^T, and the sums B_t ----------------
 __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_state_kernel(GlaArgs a) {
@@ -85,37 +93,56 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_state_kernel(Gla
           z = fmaf(x.w, w[r + 3], z);
         }
         // tokens past the end change nothing: their decay is 1
-        bs[t * dkp + tc] = last ? (t < cl ? log_sigmoid_f(z) * a.inv_tau : 0.f) : z;
+        bs[t * dkp + tc] = last ? (t < cl ? log_sigmoid_fast(z) * a.inv_tau : 0.f) : z;
       }
     }
   }
   __syncthreads();
-  for (int c = tid; c < dk; c += GLA_THREADS) {
+  // sums along the chunk: `parts` threads per channel, each over its own stretch first
+  const int parts = steps >= 4 ? 4 : (steps >= 2 ? 2 : 1), len = GC / parts;
+  float *tot = a2s;  // (parts, dkp)
+  if (tc < dk && tr < parts) {
     float run = 0.f;
-#pragma unroll 8
-    for (int t = 0; t < GC; ++t) {
-      run += bs[t * dkp + c];
-      bs[t * dkp + c] = run;
+#pragma unroll 16
+    for (int t = tr * len; t < tr * len + len; ++t) {
+      run += bs[t * dkp + tc];
+      bs[t * dkp + tc] = run;
     }
-    a.decay[(((size_t)b * a.H + h) * a.nc + ci) * dk + c] = run;
+    tot[tr * dkp + tc] = run;
   }
   __syncthreads();
-  const int kc = dkp / 2;
-  for (int i = tid; i < GC * kc; i += GLA_THREADS) {
-    const int t = i / kc, c = (i - t * kc) * 2;
-    float x = 0.f, y = 0.f;
-    if (t < cl && c < dk) {  // dk is even
-      const float2 s = *reinterpret_cast<const float2 *>(bs + t * dkp + c);
-      const float2 e = *reinterpret_cast<const float2 *>(bs + (GC - 1) * dkp + c);
-      const float2 k = b2f(*reinterpret_cast<const uint32_t *>(rows + (size_t)t * a.ld + koff + c));
-      x = k.x * expf(e.x - s.x);
-      y = k.y * expf(e.y - s.y);
-      *reinterpret_cast<float2 *>(a.cum + (((size_t)b * a.n + t0 + t) * a.H + h) * dk + c) = s;
+  if (tc < dk && tr < parts) {
+    float before = 0.f;
+    for (int x = 0; x < tr; ++x) before += tot[x * dkp + tc];
+    if (tr > 0) {
+#pragma unroll 16
+      for (int t = tr * len; t < tr * len + len; ++t) bs[t * dkp + tc] += before;
     }
-    uint32_t hi, lo;
-    split2(x, y, hi, lo);
-    *reinterpret_cast<uint32_t *>(k_hi + t * kp + c) = hi;
-    *reinterpret_cast<uint32_t *>(k_lo + t * kp + c) = lo;
+    if (tr == parts - 1) a.decay[(((size_t)b * a.H + h) * a.nc + ci) * dk + tc] = before + tot[tr * dkp + tc];
+  }
+  __syncthreads();
+  const int kc = dkp / 2, kstep = GLA_THREADS / kc;  // pairs of channels, rows at a time
+  const int kt0 = tid / kc, c2 = (tid - kt0 * kc) * 2;
+  if (kt0 < kstep) {
+    const bool inside = c2 < dk;  // dk is even
+    const float2 e = inside ? *reinterpret_cast<const float2 *>(bs + (GC - 1) * dkp + c2) : make_float2(0.f, 0.f);
+    const bf16 *kr = rows + (size_t)kt0 * a.ld + koff + c2;
+    float *cum = a.cum + (((size_t)b * a.n + t0 + kt0) * a.H + h) * dk + c2;
+#pragma unroll 4
+    for (int t = kt0; t < GC; t += kstep, kr += (size_t)kstep * a.ld, cum += (size_t)kstep * a.H * dk) {
+      float x = 0.f, y = 0.f;
+      if (t < cl && inside) {
+        const float2 s = *reinterpret_cast<const float2 *>(bs + t * dkp + c2);
+        const float2 k = b2f(*reinterpret_cast<const uint32_t *>(kr));
+        x = k.x * __expf(e.x - s.x);
+        y = k.y * __expf(e.y - s.y);
+        *reinterpret_cast<float2 *>(cum) = s;
+      }
+      uint32_t hi, lo;
+      split2(x, y, hi, lo);
+      *reinterpret_cast<uint32_t *>(k_hi + t * kp + c2) = hi;
+      *reinterpret_cast<uint32_t *>(k_lo + t * kp + c2) = lo;
+    }
   }
   cp_async_wait<0>();
   __syncthreads();
@@ -177,18 +204,20 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_out_kernel(GlaAr
   stage_rows(qs, kp, rows + qoff, a.ld, cl, dk, dkp);
   stage_rows(ks, kp, rows + koff, a.ld, cl, dk, dkp);
   stage_rows(vs, vp, rows + voff, a.ld, cl, dv, dvp);
-  cp_async_commit();
   {
     const float *cum = a.cum + (((size_t)b * a.n + t0) * a.H + h) * dk;
-    const int per = dkp / 4;  // dk % 8 == 0
-    for (int i = tid; i < GC * per; i += GLA_THREADS) {
-      const int t = i / per, c = (i - t * per) * 4;
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      // (rows past the end repeat the last sum; columns past the end are zero)
-      if (c < dk) v = *reinterpret_cast<const float4 *>(cum + (size_t)min(t, cl - 1) * a.H * dk + c);
-      *reinterpret_cast<float4 *>(bs + t * bp + c) = v;
+    const int per = dkp / 4, step = GLA_THREADS / per;  // dk % 8 == 0
+    const int r0 = tid / per, c = (tid - r0 * per) * 4;
+    if (r0 < step) {
+#pragma unroll 4
+      for (int t = r0; t < GC; t += step) {
+        // (rows past the end repeat the last sum; columns past the end are zero)
+        const bool ok = c < dk;
+        cp_async16_zfill(smem_addr(bs + t * bp + c), ok ? cum + (size_t)min(t, cl - 1) * a.H * dk + c : cum, ok ? 16 : 0);
+      }
     }
   }
+  cp_async_commit();
   cp_async_wait<0>();
   __syncthreads();
 
@@ -263,15 +292,18 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_out_kernel(GlaAr
   }
   __syncthreads();
   // queries for the incoming state: q exp(B_t), split, over q and k
-  const int kc = dkp / 2;
-  for (int i = tid; i < GC * kc; i += GLA_THREADS) {
-    const int t = i / kc, c = (i - t * kc) * 2;
-    const float2 q = b2f(*reinterpret_cast<const uint32_t *>(qs + t * kp + c));
-    const float2 s = *reinterpret_cast<const float2 *>(bs + t * bp + c);
-    uint32_t hi, lo;
-    split2(q.x * a.scale * expf(s.x), q.y * a.scale * expf(s.y), hi, lo);
-    *reinterpret_cast<uint32_t *>(qs + t * kp + c) = hi;
-    *reinterpret_cast<uint32_t *>(ks + t * kp + c) = lo;
+  const int kc = dkp / 2, kstep = GLA_THREADS / kc;
+  const int kt0 = tid / kc, c2 = (tid - kt0 * kc) * 2;
+  if (kt0 < kstep) {
+#pragma unroll 4
+    for (int t = kt0; t < GC; t += kstep) {
+      const float2 q = b2f(*reinterpret_cast<const uint32_t *>(qs + t * kp + c2));
+      const float2 s = *reinterpret_cast<const float2 *>(bs + t * bp + c2);
+      uint32_t hi, lo;
+      split2(q.x * a.scale * __expf(s.x), q.y * a.scale * __expf(s.y), hi, lo);
+      *reinterpret_cast<uint32_t *>(qs + t * kp + c2) = hi;
+      *reinterpret_cast<uint32_t *>(ks + t * kp + c2) = lo;
+    }
   }
   __syncthreads();
 #pragma unroll
@@ -384,8 +416,7 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_out_kernel(GlaAr
           const float2 gt = b2f(*reinterpret_cast<const uint32_t *>(gate + j));
           const float2 w = *reinterpret_cast<const float2 *>(a.norm + j);
           *reinterpret_cast<uint32_t *>(out + j) =
-              pack_bf16(acc[m][x][2 * e] * rn * w.x * (gt.x * sigmoid_f(gt.x)),
-                        acc[m][x][2 * e + 1] * rn * w.y * (gt.y * sigmoid_f(gt.y)));
+              pack_bf16(acc[m][x][2 * e] * rn * w.x * silu_fast(gt.x), acc[m][x][2 * e + 1] * rn * w.y * silu_fast(gt.y));
         }
       }
     }

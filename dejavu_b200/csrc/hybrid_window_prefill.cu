@@ -1,7 +1,7 @@
 // Sliding-window attention of a prompt portion on the 5th-generation tensor cores (bf16).
 //
 // A block takes 128 queries of one head and walks the key tiles of 128 that their windows touch:
-//   S (TMEM, 128 x 128 fp32) = Q K^T;  softmax in registers, one query row per thread, no shuffles;
+//   S (TMEM, 128 x 128 fp32) = Q K^T;  softmax in registers, two threads per query row (64 keys each), no shuffles;
 //   P goes back to TMEM over S as two bf16 terms, p = hi + lo, so that the weights keep their fp32 value to 2^-17;
 //   O (TMEM, 128 x dv fp32) += P_hi V + P_lo V.
 // O is only rescaled when a row's maximum grows by more than 2^8 (the final division by the sum makes up for the rest).
@@ -16,7 +16,7 @@
 
 namespace djv {
 
-constexpr int WP_THREADS = 128;
+constexpr int WP_THREADS = 256;
 constexpr int WP_TILE = 128;  // queries per block, keys per tile
 
 __device__ unsigned g_window_timeouts;  // bounded waits that ran out (never, in a healthy run)
@@ -53,13 +53,15 @@ __device__ __forceinline__ uint64_t sub2(uint64_t a, uint64_t b) {
 }
 
 template <int KB, int VB>  // 64-element blocks of a query/key row and of a value row
-__global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a) {
+__global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_kernel(WindowArgs a) {
   extern __shared__ unsigned char smem_raw[];
   __shared__ __align__(8) uint64_t bar_s, bar_o;
   __shared__ uint32_t tmem_slot;
+  __shared__ float exch[2][WP_TILE];  // maxima, and in the end sums, of the two halves of a row
   constexpr uint32_t COLS = VB > 2 ? 512 : 256;
   constexpr uint32_t KT = KB * WP_TILE * 128;
   const int tid = threadIdx.x, warp = tid / WARP;
+  const int half = tid / WP_TILE, r = tid % WP_TILE;  // keys of a tile, query row; warps w and w + 4 share TMEM lanes
   const int h = blockIdx.y, b = blockIdx.z, g = h / (a.H / a.G);
   const int t0 = blockIdx.x * WP_TILE;
   unsigned char *base = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -90,7 +92,7 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
   // One tile of keys or values. The chunk a thread copies is the same in every row, so a tile of the portion's own
   // tokens is a pointer that advances by a fixed number of rows.
   auto load = [&](uint32_t dst, int j0, const bf16 *ring, int dim, const bf16 *fresh, auto blocks) {
-    constexpr int PER_ROW = decltype(blocks)::value * 8, STEP = WP_THREADS / PER_ROW;
+    constexpr int PER_ROW = decltype(blocks)::value * 8, STEP = WP_THREADS / PER_ROW, ROUNDS = WP_TILE / STEP;
     const int ch = tid & (PER_ROW - 1), r0 = tid / PER_ROW;
     const bool inside = ch * 8 < dim;
     if (j0 >= 0 && j0 + WP_TILE - 1 <= last) {
@@ -98,13 +100,13 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
       const size_t step = (size_t)STEP * a.ld;
       if (!inside) src = fresh;  // (not read)
 #pragma unroll
-      for (int it = 0; it < PER_ROW; ++it) {
+      for (int it = 0; it < ROUNDS; ++it) {
         cp_async16_zfill(dst + sw128_offset(WP_TILE, r0 + it * STEP, ch), src, inside ? 16 : 0);
         if (inside) src += step;
       }
     } else {
-      for (int r = r0; r < WP_TILE; r += STEP) {
-        const int j = j0 + r;
+      for (int x = r0; x < WP_TILE; x += STEP) {
+        const int j = j0 + x;
         const bf16 *src = fresh;
         const bool ok = inside && j <= last;
         if (ok) {
@@ -116,7 +118,7 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
             src = ring + (size_t)slot * dim + ch * 8;
           }
         }
-        cp_async16_zfill(dst + sw128_offset(WP_TILE, r, ch), src, ok ? 16 : 0);
+        cp_async16_zfill(dst + sw128_offset(WP_TILE, x, ch), src, ok ? 16 : 0);
       }
     }
     cp_async_commit();
@@ -128,10 +130,10 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
   {  // queries
     constexpr int PER_ROW = KB * 8;
     const int ch = tid & (PER_ROW - 1);
-    for (int r = tid / PER_ROW; r < WP_TILE; r += WP_THREADS / PER_ROW) {
-      const bool ok = ch * 8 < a.dk && t0 + r <= last;
-      cp_async16_zfill(q_sm + sw128_offset(WP_TILE, r, ch),
-                       ok ? rows + (size_t)(t0 + r) * a.ld + (size_t)h * a.dk + ch * 8 : rows, ok ? 16 : 0);
+    for (int x = tid / PER_ROW; x < WP_TILE; x += WP_THREADS / PER_ROW) {
+      const bool ok = ch * 8 < a.dk && t0 + x <= last;
+      cp_async16_zfill(q_sm + sw128_offset(WP_TILE, x, ch),
+                       ok ? rows + (size_t)(t0 + x) * a.ld + (size_t)h * a.dk + ch * 8 : rows, ok ? 16 : 0);
     }
   }
   load(k_sm, lo, kr, a.dk, k_new, kb);
@@ -139,7 +141,7 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
   const float sink = a.sink ? a.sink[h] * 1.4426950408889634f : 0.f;
   const float c = a.scale * 1.4426950408889634f;  // scores in units of log 2
   float m = -1e30f, l = 0.f;
-  const int row = t0 + tid;
+  const int row = t0 + r;
   const uint32_t idesc_s = mma_idesc(WP_TILE, WP_TILE, false, false);
   const int dvp = (a.dv + 15) / 16 * 16;
   const uint32_t idesc_o = mma_idesc(WP_TILE, dvp, false, true);
@@ -149,7 +151,7 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
   tmem_fence_after();
   const uint32_t tm = tmem_slot;
   const uint32_t tm_s = tm, tm_o = tm + WP_TILE;
-  const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
+  const uint32_t lane_base = (uint32_t)(warp % 4 * 32) << 16;
 
   for (int i = 0; i < tiles; ++i) {
     const int j0 = lo + i * WP_TILE;
@@ -174,16 +176,16 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
     if (i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, kb);
 
     __syncwarp();
-    uint32_t s[4][32];
+    uint32_t s[2][32];
 #pragma unroll
-    for (int q = 0; q < 4; ++q) tmem_ld32(s[q], tm_s + lane_base + q * 32);
+    for (int q = 0; q < 2; ++q) tmem_ld32(s[q], tm_s + lane_base + half * 64 + q * 32);
     tmem_wait_ld();
     // keys outside this row's window: those after it and those more than window - 1 before it
     const bool edge = j0 + WP_TILE - 1 > t0 || j0 < t0 + WP_TILE - a.window;
     if (edge) {
-      const int hi_c = row - j0, lo_c = row - a.window + 1 - j0;  // columns lo_c .. hi_c are seen
+      const int hi_c = row - j0 - half * 64, lo_c = hi_c - a.window + 1;  // columns lo_c .. hi_c are seen
 #pragma unroll
-      for (int q = 0; q < 4; ++q)
+      for (int q = 0; q < 2; ++q)
 #pragma unroll
         for (int e = 0; e < 32; ++e)
           if (q * 32 + e > hi_c || q * 32 + e < lo_c) s[q][e] = 0xff800000u;  // -inf
@@ -191,13 +193,15 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
     // (a negative scale turns the maximum round; masked entries stay at -inf below)
     float mx = -INFINITY;
     if (c >= 0.f) {
+      float mm[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};  // independent chains
 #pragma unroll
-      for (int q = 0; q < 4; ++q)
+      for (int q = 0; q < 2; ++q)
 #pragma unroll
-        for (int e = 0; e < 32; ++e) mx = fmaxf(mx, __uint_as_float(s[q][e]));
+        for (int e = 0; e < 32; ++e) mm[e % 4] = fmaxf(mm[e % 4], __uint_as_float(s[q][e]));
+      mx = fmaxf(fmaxf(mm[0], mm[1]), fmaxf(mm[2], mm[3]));
     } else {
 #pragma unroll
-      for (int q = 0; q < 4; ++q)
+      for (int q = 0; q < 2; ++q)
 #pragma unroll
         for (int e = 0; e < 32; ++e)
           if (s[q][e] != 0xff800000u) {
@@ -205,31 +209,36 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
             s[q][e] ^= 0x80000000u;
           }
     }
+    exch[half][r] = mx;
+    tmem_fence_before();  // both halves have read S before either puts P over it
+    __syncthreads();
+    tmem_fence_after();
+    mx = fmaxf(mx, exch[half ^ 1][r]);
     const float ca = fabsf(c);
     mx *= ca;
     if (a.sink && i == 0) mx = fmaxf(mx, sink);
     const bool grow = mx > m + 8.f;
     if (i == 0) {
       m = fmaxf(mx, m);
-      l = a.sink ? exp2_approx(sink - m) : 0.f;
+      l = a.sink && half == 0 ? exp2_approx(sink - m) : 0.f;
     } else if (__any_sync(0xffffffffu, grow)) {
       const float corr = grow ? exp2_approx(m - mx) : 1.f;
       if (grow) m = mx;
       l *= corr;
-      for (int q = 0; q < dvp; q += 32) {  // (TMEM columns up to the next multiple of 32 belong to this block)
-        uint32_t o[32];
-        tmem_ld32(o, tm_o + lane_base + q);
+      for (int q = half * 16; q < dvp; q += 32) {
+        uint32_t o[16];
+        tmem_ld16(o, tm_o + lane_base + q);
         tmem_wait_ld();
 #pragma unroll
-        for (int e = 0; e < 32; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * corr);
-        tmem_st32(tm_o + lane_base + q, o);
+        for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * corr);
+        tmem_st16(tm_o + lane_base + q, o);
       }
     }
     const float nm = -m;
     const uint64_t ca2 = pack2(ca, ca), nm2 = pack2(nm, nm);
-    uint64_t l2 = 0;
+    uint64_t l2[2] = {0, 0};
 #pragma unroll
-    for (int q = 0; q < 4; ++q) {
+    for (int q = 0; q < 2; ++q) {
       uint32_t hi[16], lw[16];
 #pragma unroll
       for (int e = 0; e < 16; ++e) {
@@ -238,7 +247,7 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
         x = exp2_approx(x);
         y = exp2_approx(y);
         const uint64_t p = pack2(x, y);
-        l2 = add2(l2, p);
+        l2[e % 2] = add2(l2[e % 2], p);
         // hi: the upper halves; the rest, which a float holds exactly, is rounded to bf16
         hi[e] = __byte_perm(__float_as_uint(x), __float_as_uint(y), 0x7632);
         const uint64_t top = pack2(__uint_as_float(__float_as_uint(x) & 0xffff0000u),
@@ -247,12 +256,12 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
         unpack2(sub2(p, top), rx, ry);
         lw[e] = pack_bf16(rx, ry);
       }
-      tmem_st16(tm_s + lane_base + q * 16, hi);
-      tmem_st16(tm_s + lane_base + 64 + q * 16, lw);
+      tmem_st16(tm_s + lane_base + half * 32 + q * 16, hi);
+      tmem_st16(tm_s + lane_base + 64 + half * 32 + q * 16, lw);
     }
     {
       float x, y;
-      unpack2(l2, x, y);
+      unpack2(add2(l2[0], l2[1]), x, y);
       l += x + y;
     }
     tmem_wait_st();
@@ -275,15 +284,18 @@ __global__ void __launch_bounds__(WP_THREADS) window_prefill_kernel(WindowArgs a
   if (!dead) dead = !mbar_wait(&bar_o, (tiles - 1) & 1);
   __syncwarp();
   tmem_fence_after();
-  const float inv = 1.f / l;
+  __syncthreads();
+  exch[half][r] = l;
+  __syncthreads();
+  const float inv = 1.f / (l + exch[half ^ 1][r]);
   bf16 *out = static_cast<bf16 *>(a.out) + (((size_t)b * a.n + row) * a.H + h) * a.dv;
-  for (int q = 0; q < dvp; q += 32) {
-    uint32_t o[32];
-    tmem_ld32(o, tm_o + lane_base + q);
+  for (int q = half * 16; q < dvp; q += 32) {
+    uint32_t o[16];
+    tmem_ld16(o, tm_o + lane_base + q);
     tmem_wait_ld();
     if (row <= last) {
 #pragma unroll
-      for (int e = 0; e < 32; e += 8) {
+      for (int e = 0; e < 16; e += 8) {
         if (q + e < a.dv) {  // dv % 8 == 0
           uint4 v;
           v.x = pack_bf16(__uint_as_float(o[e]) * inv, __uint_as_float(o[e + 1]) * inv);

@@ -2,6 +2,7 @@
 
     python -m dejavu_b200.profile_cases <case>
         case: qkv | out_proj | attn | topk | exchange | ring | fc1 | fc2 | fc1_b16 | fc2_b16 | ring_trace
+              hybrid_window | hybrid_gla | hybrid_decode   (shapes of the 7b size of bench.py --hybrid)
 
 Every case launches ONE kind of kernel a dozen times at the per-rank shapes of an OPT-175B layer under 8-way
 tensor parallelism (d 12288, 12 local heads of which 4 are active, 512 of 6144 ffn rows), rotating several weight
@@ -71,6 +72,28 @@ def main(case: str) -> None:
             for i in range(4):
                 if case == "fc1_b16": ops.gather_gemv(x, Ws[i], idxs[i], b1, "relu")
                 else: ops.gather_transposed_gemv(h, Ws[i], idxs[i], b2)
+    elif case in ("hybrid_window", "hybrid_gla", "hybrid_decode"):
+        H, G, dk, dv, W, GH, gk, gv, rank, n = 32, 8, 128, 128, 1024, 16, 128, 256, 16, 4096
+        def bf(*shape): return torch.randn(*shape, device=dev, generator=g).bfloat16()
+        def f32(*shape): return torch.randn(*shape, device=dev, generator=g)
+        gla = (f32(GH * gk, rank) * 0.1, torch.ones(GH * gk, device=dev), 16.0, torch.ones(gv, device=dev), 1e-6, gk ** -0.5)
+        pos = torch.zeros(1, dtype=torch.int64, device=dev)
+        sink = torch.ones(H, device=dev)
+        if case == "hybrid_window":
+            rows = [bf(n, (H + G) * dk + G * dv) for _ in range(3)]
+            ring = (bf(1, G, W, dk), bf(1, G, W, dv))
+            for r in rows * 2: ops.window_attention(r, *ring, sink, pos, n, H, W, dk ** -0.5)
+        elif case == "hybrid_gla":
+            rows, st = [bf(n, 2 * GH * (gk + gv) + rank) for _ in range(2)], f32(1, GH, gk, gv)
+            for r in rows * 2: ops.gated_linear_attention(r, *gla, st, pos, n)
+        else:
+            far = pos + 5000
+            row, prow = bf(1, (H + G) * dk + G * dv), bf(1, 2 * GH * (gk + gv) + rank)
+            rings = [(bf(1, G, W, dk), bf(1, G, W, dv)) for _ in range(40)]
+            states = [f32(1, GH, gk, gv) for _ in range(70)]
+            freqs = torch.rand(dk // 2, device=dev)
+            for r in rings: ops.window_attention_decode(row, *r, sink, freqs, 1.0, far, H, W, dk ** -0.5)
+            for s in states: ops.gated_linear_attention(prow, *gla, s, far, 1)
     torch.cuda.synchronize()
     if case == "ring_trace":
         lib = _lib.load()
