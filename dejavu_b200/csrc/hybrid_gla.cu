@@ -96,16 +96,16 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_state_scan_kernel(GlaArgs a) 
   if (e >= per) return;
   const size_t bh = (size_t)b * a.H + h;
   auto get = [](const float *p, float (&v)[V]) {
-    if (V == 4) {
-      const float4 t = *reinterpret_cast<const float4 *>(p);
-      v[0] = t.x; v[1 % V] = t.y; v[2 % V] = t.z; v[3 % V] = t.w;
+    if (V == 2) {
+      const float2 t = *reinterpret_cast<const float2 *>(p);
+      v[0] = t.x; v[1 % V] = t.y;
     } else {
       v[0] = *p;
     }
   };
   auto put = [](float *p, const float (&v)[V]) {
-    if (V == 4)
-      *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
+    if (V == 2)
+      *reinterpret_cast<float2 *>(p) = make_float2(v[0], v[1 % V]);
     else
       *p = v[0];
   };
@@ -378,8 +378,8 @@ static int launch_prefill(const GlaArgs &a, bool mma, cudaStream_t st) {
     count_launch();
   }
   if (rc) return rc;
-  if (a.dv % 4 == 0 && aligned16(a.state))
-    djv::launch_kernel(gla_state_scan_kernel<4>, dim3(ceil_div(a.dk * a.dv, 4 * GLA_THREADS), a.H, a.B),
+  if (a.dv % 2 == 0 && aligned16(a.state))
+    djv::launch_kernel(gla_state_scan_kernel<2>, dim3(ceil_div(a.dk * a.dv, 2 * GLA_THREADS), a.H, a.B),
                        dim3(GLA_THREADS), 0, st, a);
   else
     djv::launch_kernel(gla_state_scan_kernel<1>, dim3(ceil_div(a.dk * a.dv, GLA_THREADS), a.H, a.B), dim3(GLA_THREADS),

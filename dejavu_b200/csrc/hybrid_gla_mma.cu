@@ -55,22 +55,20 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_state_kernel(Gla
   const int t0 = ci * GC, cl = min(GC, a.n - t0);
   bf16 *k_hi = reinterpret_cast<bf16 *>(sm_raw), *k_lo = k_hi + GC * kp, *vs = k_lo + GC * kp;
   float *bs = reinterpret_cast<float *>(vs + GC * vp);  // [GC][dkp]
-  float *a2s = bs + GC * dkp, *ts = a2s + 16 * dkp;     // 16 ranks at a time: [16][dkp], [GC][16]
+  float *tot = bs + GC * dkp, *ts = tot + 4 * dkp;      // [4][dkp]; 16 ranks of the decay input at a time: [GC][16]
   const bf16 *rows = static_cast<const bf16 *>(a.proj) + ((size_t)b * a.n + t0) * a.ld;
   const int koff = a.H * dk + h * dk, voff = 2 * a.H * dk + h * dv, toff = 2 * a.H * dk + 2 * a.H * dv;
 
+  stage_rows(k_lo, kp, rows + koff, a.ld, cl, dk, dkp);  // (split in place below)
   stage_rows(vs, vp, rows + voff, a.ld, cl, dv, dvp);
   cp_async_commit();
   // log decays: thread = channel, the rows in steps
   const int cpr = min(dkp, GLA_THREADS), steps = GLA_THREADS / cpr;  // (dk <= 256)
   const int tc = tid % cpr, tr = tid / cpr;
+  const float *wr = a.a2 + (size_t)(h * dk + min(tc, dk - 1)) * a.rank;
   for (int r0 = 0; r0 < a.rank; r0 += 16) {
     const int rn = min(16, a.rank - r0);
     __syncthreads();
-    for (int i = tid; i < dk * rn; i += GLA_THREADS) {
-      const int c = i / rn, r = i - c * rn;
-      a2s[r * dkp + c] = a.a2[(size_t)(h * dk + c) * a.rank + r0 + r];
-    }
     for (int i = tid; i < GC * 16; i += GLA_THREADS) {
       const int t = i / 16, r = i % 16;
       ts[i] = (t < cl && r < rn) ? to_f(rows[(size_t)t * a.ld + toff + r0 + r]) : 0.f;
@@ -79,7 +77,7 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_state_kernel(Gla
     if (tc < dk && tr < steps) {
       float w[16];
 #pragma unroll
-      for (int r = 0; r < 16; ++r) w[r] = r < rn ? a2s[r * dkp + tc] : 0.f;
+      for (int r = 0; r < 16; ++r) w[r] = r < rn ? __ldg(wr + r0 + r) : 0.f;
       const float bias = a.a2_bias[h * dk + tc];
       const bool last = r0 + 16 >= a.rank;
       for (int t = tr; t < GC; t += steps) {
@@ -100,7 +98,6 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_state_kernel(Gla
   __syncthreads();
   // sums along the chunk: `parts` threads per channel, each over its own stretch first
   const int parts = steps >= 4 ? 4 : (steps >= 2 ? 2 : 1), len = GC / parts;
-  float *tot = a2s;  // (parts, dkp)
   if (tc < dk && tr < parts) {
     float run = 0.f;
 #pragma unroll 16
@@ -120,20 +117,20 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_state_kernel(Gla
     }
     if (tr == parts - 1) a.decay[(((size_t)b * a.H + h) * a.nc + ci) * dk + tc] = before + tot[tr * dkp + tc];
   }
+  cp_async_wait<0>();
   __syncthreads();
   const int kc = dkp / 2, kstep = GLA_THREADS / kc;  // pairs of channels, rows at a time
   const int kt0 = tid / kc, c2 = (tid - kt0 * kc) * 2;
   if (kt0 < kstep) {
     const bool inside = c2 < dk;  // dk is even
     const float2 e = inside ? *reinterpret_cast<const float2 *>(bs + (GC - 1) * dkp + c2) : make_float2(0.f, 0.f);
-    const bf16 *kr = rows + (size_t)kt0 * a.ld + koff + c2;
     float *cum = a.cum + (((size_t)b * a.n + t0 + kt0) * a.H + h) * dk + c2;
 #pragma unroll 4
-    for (int t = kt0; t < GC; t += kstep, kr += (size_t)kstep * a.ld, cum += (size_t)kstep * a.H * dk) {
+    for (int t = kt0; t < GC; t += kstep, cum += (size_t)kstep * a.H * dk) {
       float x = 0.f, y = 0.f;
       if (t < cl && inside) {
         const float2 s = *reinterpret_cast<const float2 *>(bs + t * dkp + c2);
-        const float2 k = b2f(*reinterpret_cast<const uint32_t *>(kr));
+        const float2 k = b2f(*reinterpret_cast<const uint32_t *>(k_lo + t * kp + c2));
         x = k.x * __expf(e.x - s.x);
         y = k.y * __expf(e.y - s.y);
         *reinterpret_cast<float2 *>(cum) = s;
@@ -144,7 +141,6 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_state_kernel(Gla
       *reinterpret_cast<uint32_t *>(k_lo + t * kp + c2) = lo;
     }
   }
-  cp_async_wait<0>();
   __syncthreads();
   // U (channels x values): a warp takes 16 channels and walks the value columns 16 at a time
   float *U = a.contrib + (((size_t)b * a.H + h) * a.nc + ci) * (size_t)dk * dv;
@@ -201,6 +197,9 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_out_kernel(GlaAr
   const bf16 *rows = static_cast<const bf16 *>(a.proj) + ((size_t)b * a.n + t0) * a.ld;
   const int qoff = h * dk, koff = a.H * dk + h * dk, voff = 2 * a.H * dk + h * dv, goff = voff + a.H * dv;
 
+  // the incoming state is needed last: have it in L2 by then
+  const float *S = a.contrib + (((size_t)b * a.H + h) * a.nc + ci) * (size_t)dk * dv;
+  for (int i = tid * 32; i < dk * dv; i += GLA_THREADS * 32) prefetch_l2(S + i);
   stage_rows(qs, kp, rows + qoff, a.ld, cl, dk, dkp);
   stage_rows(ks, kp, rows + koff, a.ld, cl, dk, dkp);
   stage_rows(vs, vp, rows + voff, a.ld, cl, dv, dvp);
@@ -321,7 +320,6 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_out_kernel(GlaAr
   __syncthreads();
 
   // outputs: a warp takes NT * 8 value columns of all 64 rows
-  const float *S = a.contrib + (((size_t)b * a.H + h) * a.nc + ci) * (size_t)dk * dv;
   const int n0 = warp * NT * 8;
   float acc[GC / 16][NT][4];
 #pragma unroll
@@ -424,7 +422,7 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_out_kernel(GlaAr
 
 static size_t mma_state_smem(int dk, int dv) {
   const int dkp = up16(dk), dvp = up16(dv);
-  return (size_t)GC * ((2 * (dkp + 8) + dvp + 8) * 2 + dkp * 4) + 16 * dkp * 4 + GC * 16 * 4;
+  return (size_t)GC * ((2 * (dkp + 8) + dvp + 8) * 2 + dkp * 4) + 4 * dkp * 4 + GC * 16 * 4;
 }
 static size_t mma_out_smem(int dk, int dv) {
   const int dkp = up16(dk), dvp = up16(dv);

@@ -7,7 +7,8 @@
 // O is only rescaled when a row's maximum grows by more than 2^8 (the final division by the sum makes up for the rest).
 // Keys come from the ring (tokens before the portion) or from the projection's output (the portion's own), row by row,
 // with 16-byte asynchronous copies into the swizzled operand layout. Two blocks share a multiprocessor: one computes
-// its softmax while the other's products run. K of the next tile loads behind the scores, V behind the values.
+// its softmax while the other's products run. V of a tile loads behind its scores, K of the next one behind the
+// values' products.
 #include "../../include/dejavu_b200_hybrid.h"
 #include "hybrid_attention.cuh"
 #include "tcgen05.cuh"
@@ -62,8 +63,9 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
   constexpr uint32_t KT = KB * WP_TILE * 128;
   const int tid = threadIdx.x, warp = tid / WARP;
   const int half = tid / WP_TILE, r = tid % WP_TILE;  // keys of a tile, query row; warps w and w + 4 share TMEM lanes
-  const int h = blockIdx.y, b = blockIdx.z, g = h / (a.H / a.G);
-  const int t0 = blockIdx.x * WP_TILE;
+  // the first queries of a sequence have short windows: their blocks come last and fill the tail of the grid
+  const int h = blockIdx.x, b = blockIdx.z, g = h / (a.H / a.G);
+  const int t0 = (int)(gridDim.y - 1 - blockIdx.y) * WP_TILE;
   unsigned char *base = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   const uint32_t q_sm = smem_u32(base), k_sm = q_sm + KT, v_sm = k_sm + KT;
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
@@ -146,6 +148,8 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
   const int dvp = (a.dv + 15) / 16 * 16;
   const uint32_t idesc_o = mma_idesc(WP_TILE, dvp, false, true);
   const int k_steps = (a.dk + 15) / 16;
+  const uint64_t q_desc = desc_k_major(q_sm, WP_TILE, 0), k_desc = desc_k_major(k_sm, WP_TILE, 0);
+  const uint64_t v_desc = desc_mn_major(v_sm, WP_TILE, 0);
   bool dead = false;  // a wait ran out: wait no more, finish and report
   __syncthreads();
   tmem_fence_after();
@@ -165,16 +169,17 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
     __syncthreads();
     if (tid == 0) {
       tmem_fence_after();
-      for (int k = 0; k < k_steps; ++k)
-        mma_ss(tm_s, desc_k_major(q_sm, WP_TILE, k), desc_k_major(k_sm, WP_TILE, k), idesc_s, k > 0);
+#pragma unroll
+      for (int k = 0; k < KB * 4; ++k) {
+        const uint32_t step = (k / 4) * (WP_TILE * 128 / 16) + (k % 4) * 2;  // descriptor units of 16 bytes
+        if (k < k_steps) mma_ss(tm_s, q_desc + step, k_desc + step, idesc_s, k > 0);
+      }
       mma_commit(&bar_s);
     }
     load(v_sm, j0, vr, a.dv, v_new, vb);
     if (!dead) dead = !mbar_wait(&bar_s, i & 1);
     __syncwarp();
     tmem_fence_after();
-    if (i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, kb);
-
     __syncwarp();
     uint32_t s[2][32];
 #pragma unroll
@@ -266,20 +271,20 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
     }
     tmem_wait_st();
     tmem_fence_before();
-    if (i + 1 < tiles)
-      cp_async_wait<1>();  // V is there; K of the next tile may still be on its way
-    else
-      cp_async_wait<0>();
+    cp_async_wait<0>();  // V
     fence_proxy_async_smem();
     __syncthreads();
     if (tid == 0) {
       tmem_fence_after();
+#pragma unroll
       for (int k = 0; k < WP_TILE / 16; ++k)
-        mma_ts(tm_o, tm_s + k * 8, desc_mn_major(v_sm, WP_TILE, k), idesc_o, i > 0 || k > 0);
+        mma_ts(tm_o, tm_s + k * 8, v_desc + (uint64_t)(k * 128), idesc_o, i > 0 || k > 0);
+#pragma unroll
       for (int k = 0; k < WP_TILE / 16; ++k)
-        mma_ts(tm_o, tm_s + 64 + k * 8, desc_mn_major(v_sm, WP_TILE, k), idesc_o, true);
+        mma_ts(tm_o, tm_s + 64 + k * 8, v_desc + (uint64_t)(k * 128), idesc_o, true);
       mma_commit(&bar_o);
     }
+    if (i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, kb);  // behind the values' products
   }
   if (!dead) dead = !mbar_wait(&bar_o, (tiles - 1) & 1);
   __syncwarp();
@@ -321,7 +326,7 @@ static int launch_window_prefill(const WindowArgs &a, cudaStream_t st) {
   const size_t least = (VB > 2 ? 120 : 80) * 1024;
   if (smem < least) smem = least;
   cudaFuncSetAttribute(window_prefill_kernel<KB, VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  djv::launch_kernel(window_prefill_kernel<KB, VB>, dim3(ceil_div(a.n, WP_TILE), a.H, a.B), dim3(WP_THREADS), smem, st,
+  djv::launch_kernel(window_prefill_kernel<KB, VB>, dim3(a.H, ceil_div(a.n, WP_TILE), a.B), dim3(WP_THREADS), smem, st,
                      a);
   count_launch();
   return check_launch("window_attn");
