@@ -116,25 +116,29 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_state_scan_kernel(GlaArgs a) 
   float *U = a.contrib + bh * a.nc * per + e;
   const float *D = a.decay + bh * a.nc * a.dk + e / a.dv;
   constexpr int CH = 8;  // chunks whose loads are in flight together
-  for (int c0 = 0; c0 < a.nc; c0 += CH, U += (size_t)CH * per, D += CH * a.dk) {
-    const int cn = min(CH, a.nc - c0);
+  int c0 = 0;
+  for (; c0 + CH <= a.nc; c0 += CH, U += (size_t)CH * per, D += CH * a.dk) {
     float u[CH][V], d[CH];
 #pragma unroll
     for (int c = 0; c < CH; ++c) {
-      if (c < cn) {
-        get(U + (size_t)c * per, u[c]);
-        d[c] = D[c * a.dk];
-      }
+      get(U + (size_t)c * per, u[c]);
+      d[c] = D[c * a.dk];
     }
 #pragma unroll
     for (int c = 0; c < CH; ++c) {
-      if (c < cn) {
-        put(U + (size_t)c * per, s);
-        const float f = expf(d[c]);
+      put(U + (size_t)c * per, s);
+      const float f = expf(d[c]);
 #pragma unroll
-        for (int v = 0; v < V; ++v) s[v] = fmaf(f, s[v], u[c][v]);
-      }
+      for (int v = 0; v < V; ++v) s[v] = fmaf(f, s[v], u[c][v]);
     }
+  }
+  for (; c0 < a.nc; ++c0, U += per, D += a.dk) {
+    float u[V];
+    get(U, u);
+    put(U, s);
+    const float f = expf(*D);
+#pragma unroll
+    for (int v = 0; v < V; ++v) s[v] = fmaf(f, s[v], u[v]);
   }
   put(a.state + bh * per + e, s);
 }

@@ -200,6 +200,9 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_out_kernel(GlaAr
   // the incoming state is needed last: have it in L2 by then
   const float *S = a.contrib + (((size_t)b * a.H + h) * a.nc + ci) * (size_t)dk * dv;
   for (int i = tid * 32; i < dk * dv; i += GLA_THREADS * 32) prefetch_l2(S + i);
+  const int gate_lines = (dv + 63) / 64;  // and the gates
+  for (int i = tid; i < cl * gate_lines; i += GLA_THREADS)
+    prefetch_l2(rows + (size_t)(i / gate_lines) * a.ld + goff + i % gate_lines * 64);
   stage_rows(qs, kp, rows + qoff, a.ld, cl, dk, dkp);
   stage_rows(ks, kp, rows + koff, a.ld, cl, dk, dkp);
   stage_rows(vs, vp, rows + voff, a.ld, cl, dv, dvp);
@@ -379,7 +382,17 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_out_kernel(GlaAr
       }
     }
   }
-  // norm over the head's values, gate
+  // norm over the head's values, gate (whose loads are in flight while the sums meet)
+  uint32_t gates[GC / 16][2][NT];
+#pragma unroll
+  for (int m = 0; m < GC / 16; ++m)
+#pragma unroll
+    for (int e = 0; e < 2; ++e)
+#pragma unroll
+      for (int x = 0; x < NT; ++x) {
+        const int t = m * 16 + g + e * 8, j = n0 + x * 8 + t4 * 2;
+        gates[m][e][x] = (t < cl && j < dv) ? *reinterpret_cast<const uint32_t *>(rows + (size_t)t * a.ld + goff + j) : 0;
+      }
 #pragma unroll
   for (int m = 0; m < GC / 16; ++m)
 #pragma unroll
@@ -405,13 +418,12 @@ __global__ void __launch_bounds__(GLA_THREADS, 2) gla_mma_chunk_out_kernel(GlaAr
 #pragma unroll
       for (int w = 0; w < GW; ++w) tot += ssq[w][t];
       const float rn = 1.f / sqrtf(tot / (float)dv + a.eps);
-      const bf16 *gate = rows + (size_t)t * a.ld + goff;
       bf16 *out = static_cast<bf16 *>(a.out) + (((size_t)b * a.n + t0 + t) * a.H + h) * dv;
 #pragma unroll
       for (int x = 0; x < NT; ++x) {
         const int j = n0 + x * 8 + t4 * 2;
         if (j < dv) {
-          const float2 gt = b2f(*reinterpret_cast<const uint32_t *>(gate + j));
+          const float2 gt = b2f(gates[m][e][x]);
           const float2 w = *reinterpret_cast<const float2 *>(a.norm + j);
           *reinterpret_cast<uint32_t *>(out + j) =
               pack_bf16(acc[m][x][2 * e] * rn * w.x * silu_fast(gt.x), acc[m][x][2 * e + 1] * rn * w.y * silu_fast(gt.y));
