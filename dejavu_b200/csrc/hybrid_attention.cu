@@ -8,6 +8,7 @@
 // that the portion's first tokens can still see. The decode step has one token, the slot it takes is the one that has
 // just left the window, so it rotates, stores and attends in one kernel.
 #include <cooperative_groups.h>
+#include <math.h>
 
 #include "../../include/dejavu_b200_hybrid.h"
 #include "hybrid_attention.cuh"
@@ -472,12 +473,25 @@ static int dispatch_decode(const DecodeArgs &d, int nsplit, bool vec, cudaStream
 }
 
 template <typename T>
-static int dispatch_decode(const DecodeArgs &d, int nsplit, bool vec, cudaStream_t st) {
-  // query heads per block: few while the blocks of all of them still fit the device at once (K and V then come from L2
-  // for the second and later blocks of a kv head), all of a kv head's otherwise
-  const int rep = d.w.H / d.w.G;
-  int rt = 1;
-  while (rt < 8 && rt < rep && (long long)d.w.G * ceil_div(rep, rt) * d.w.B * nsplit > sm_count()) rt *= 2;
+static int dispatch_decode(const DecodeArgs &d, int max_split, bool vec, cudaStream_t st) {
+  // Query heads per block (rt) and splits of the window: waves of blocks times passes of a block times a pass's work,
+  // which is a part for the K and V loads and one per query head. Blocks of one or two heads fit a multiprocessor
+  // twice; clusters of 8 leave some multiprocessors unused (120 of 148 hold one).
+  const int rep = d.w.H / d.w.G, tile = sizeof(T) == 2 ? 128 : 64;
+  int rt = 8, nsplit = max_split;
+  double best = 1e30;
+  for (int ns = max_split; ns >= 1; ns /= 2) {
+    for (int r = 1; r <= 8 && (r == 1 || r / 2 < rep); r *= 2) {
+      const double room = (r <= 2 ? 2.0 : 1.0) * sm_count() * (ns == 8 ? 0.81 : (ns > 1 ? 0.89 : 1.0));
+      const double waves = ceil((double)d.w.G * ceil_div(rep, r) * d.w.B * ns / room);
+      const double cost = waves * ceil_div(ceil_div(d.w.window, ns), tile) * (2 + r);
+      if (cost < best) {
+        best = cost;
+        rt = r;
+        nsplit = ns;
+      }
+    }
+  }
   if (rt == 1) return dispatch_decode<T, 1>(d, nsplit, vec, st);
   if (rt == 2) return dispatch_decode<T, 2>(d, nsplit, vec, st);
   if (rt == 4) return dispatch_decode<T, 4>(d, nsplit, vec, st);
