@@ -1,5 +1,5 @@
-"""ctypes binding of libdejavu_b200.so (declared in include/dejavu_b200.h) and libdejavu_b200_hybrid.so
-(include/dejavu_b200_hybrid.h).
+"""ctypes binding of libdejavu_b200.so (declared in include/dejavu_b200.h), libdejavu_b200_hybrid.so
+(include/dejavu_b200_hybrid.h) and libdejavu_b200_routed.so (include/dejavu_b200_routed.h).
 
 The libraries are the only compute path of this package: if one is missing the import of any operator
 raises, there is no PyTorch or CPU fallback.
@@ -12,9 +12,10 @@ from pathlib import Path
 PKG = Path(__file__).resolve().parent
 LIB_PATH = PKG / "libdejavu_b200.so"
 HYBRID_LIB_PATH = PKG / "libdejavu_b200_hybrid.so"
+ROUTED_LIB_PATH = PKG / "libdejavu_b200_routed.so"
 
 OK, ERR_INVALID, ERR_UNSUPPORTED, ERR_CUDA, ERR_SCRATCH, ERR_TIMEOUT = 0, -1, -2, -3, -4, -5
-ACT = {"id": 0, "relu": 1, "gelu": 2, "gelu_approx": 3, "squared_relu": 4, "softcap": 5, "clamped_glu": 6}
+ACT = {"id": 0, "relu": 1, "gelu": 2, "gelu_approx": 3, "squared_relu": 4, "softcap": 5, "clamped_glu": 6, "silu_glu": 7}
 DTYPE_F16, DTYPE_BF16, DTYPE_F32 = 0, 1, 2
 MAX_BATCH = 32
 KV_WINDOW = 16
@@ -96,9 +97,10 @@ _PLUMBING = ("djv_version", "djv_last_error", "djv_status_string", "djv_launch_c
 HYBRID_SIGNATURES = {
     "djv_hyper_step": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _i, _i, _i, _i, _vp]),
     "djv_dense_gemv": (_i, [_i, _i, _vp, _vp, _vp, _i, _i, _i, _ll, _i, _f, _vp]),
-    "djv_clamped_glu": (_i, [_i, _vp, _vp, _ll, _i, _f, _vp]),
+    "djv_residual_step": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _f, _f, _vp, _vp, _vp, _i, _i, _i, _vp]),
+    "djv_glu": (_i, [_i, _vp, _vp, _ll, _i, _i, _f, _vp]),
     "djv_softcap": (_i, [_vp, _ll, _f, _vp]),
-    "djv_rotary": (_i, [_i, _vp, _ll, _vp, _f, _vp, _i, _i, _i, _i, _i, _vp]),
+    "djv_rotary": (_i, [_i, _vp, _ll, _vp, _f, _vp, _i, _i, _i, _i, _i, _i, _vp]),
     "djv_window_attn": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp]),
     "djv_window_store": (_i, [_i, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "djv_window_attn_decode": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _f, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _f,
@@ -110,8 +112,32 @@ HYBRID_SIGNATURES = {
     "djv_gla_decode": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _i, _f, _vp, _f, _f, _vp, _vp, _i, _i, _i, _i, _vp]),
 }
 
+# mirrors include/dejavu_b200_routed.h one to one
+ROUTED_SIGNATURES = {
+    "djv_mlstm_state_floats": (_i, [_i, _i]),
+    "djv_mlstm_scratch_bytes": (_sz, [_i, _i, _i, _i, _i, _i]),
+    "djv_mlstm_prefill": (_i, [_i, _vp, _vp, _ll, _vp, _ll, _vp, _vp, _f, _vp, _f, _f, _vp, _vp, _i, _i, _i, _i, _i, _vp,
+                               _sz, _vp]),
+    "djv_mlstm_decode": (_i, [_i, _vp, _vp, _ll, _vp, _ll, _vp, _vp, _f, _vp, _f, _f, _vp, _vp, _i, _i, _i, _i, _vp]),
+    "djv_mlstm_timeouts": (C.c_uint, []),
+    "djv_latent_rows": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
+    "djv_latent_attn": (_i, [_i, _vp, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f,
+                             _vp]),
+    "djv_latent_decode": (_i, [_i, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _i,
+                               _i, _i, _i, _f, _i, _vp]),
+    "djv_moe_route": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp]),
+    "djv_moe_grouped": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp]),
+    "djv_moe_decode": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]),
+    "djv_moe_timeouts": (C.c_uint, []),
+}
+
+# functions of the hybrid header that the routed library has as well
+SHARED = ("djv_hyper_step", "djv_residual_step", "djv_dense_gemv", "djv_glu", "djv_softcap", "djv_rotary",
+          "djv_window_timeouts")
+
 _lib = None
 _hybrid = None
+_routed = None
 
 
 def _open(path, signatures) -> C.CDLL:
@@ -144,6 +170,23 @@ def load_hybrid() -> C.CDLL:
     return _hybrid
 
 
+def load_routed() -> C.CDLL:
+    """Loads the shared library of the routed decoders (once). Raises if it has not been built."""
+    global _routed
+    if _routed is None:
+        own = {**ROUTED_SIGNATURES, **{n: HYBRID_SIGNATURES[n] for n in SHARED}}
+        _routed = _open(ROUTED_LIB_PATH, {**own, **{n: SIGNATURES[n] for n in _PLUMBING}})
+    return _routed
+
+
+def _library_of(fn_name: str) -> C.CDLL:
+    if fn_name in ROUTED_SIGNATURES:
+        return load_routed()
+    if fn_name in SHARED and _hybrid is None and (_routed is not None or not HYBRID_LIB_PATH.exists()):
+        return load_routed()
+    return load_hybrid() if fn_name in HYBRID_SIGNATURES else load()
+
+
 def check(fn_name: str, status: int, lib=None) -> None:
     if status != OK:
         msg = (lib or load()).djv_last_error().decode(errors="replace")
@@ -151,10 +194,10 @@ def check(fn_name: str, status: int, lib=None) -> None:
 
 
 def call(fn_name: str, *args) -> None:
-    lib = load_hybrid() if fn_name in HYBRID_SIGNATURES else load()
+    lib = _library_of(fn_name)
     check(fn_name, getattr(lib, fn_name)(*args), lib)
 
 
 def launch_count() -> int:
     """Kernels launched by the loaded libraries since load."""
-    return sum(int(lib.djv_launch_count()) for lib in (_lib, _hybrid) if lib is not None)
+    return sum(int(lib.djv_launch_count()) for lib in (_lib, _hybrid, _routed) if lib is not None)

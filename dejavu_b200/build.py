@@ -1,9 +1,10 @@
 """Builds the C-ABI libraries of sm_100a kernels in-tree with nvcc.
 
-    python -m dejavu_b200.build [--force] [--verbose] [--lib sparse|hybrid]
+    python -m dejavu_b200.build [--force] [--verbose] [--lib sparse|hybrid|routed]
 
   sparse  libdejavu_b200.so         the contextual-sparse OPT decode path
   hybrid  libdejavu_b200_hybrid.so  gated linear attention, sliding-window attention, hyper-connected streams
+  routed  libdejavu_b200_routed.so  matrix memories, latent attention, routed feed-forwards
 
 Each .cu file is compiled to an object in parallel, then linked into the shared libraries that sit next to this file.
 Nothing is cached outside the package directory. A library can be built alone, so that a program that serves one kind
@@ -24,7 +25,14 @@ CSRC = PKG / "csrc"
 OBJ = PKG / "build"
 LIB = PKG / "libdejavu_b200.so"
 HYBRID_LIB = PKG / "libdejavu_b200_hybrid.so"
-LIBS = {"sparse": LIB, "hybrid": HYBRID_LIB}
+ROUTED_LIB = PKG / "libdejavu_b200_routed.so"
+LIBS = {"sparse": LIB, "hybrid": HYBRID_LIB, "routed": ROUTED_LIB}
+
+# translation units of the hybrid decoders' libraries; those both use are compiled once and linked into both
+_BOTH = ("api", "hybrid_gemv", "hybrid_residual", "hybrid_rotary", "hybrid_window_simple", "hybrid_window_prefill")
+_UNITS = {"hybrid": _BOTH + ("hybrid_attention", "hybrid_gla", "hybrid_gla_mma"),
+          "routed": _BOTH + ("hybrid_mlstm", "hybrid_mlstm_prefill", "hybrid_latent", "hybrid_latent_decode", "hybrid_moe",
+                             "hybrid_moe_gemm")}
 
 NVCC_FLAGS = [
     "-O3",
@@ -45,11 +53,13 @@ def _nvcc() -> str:
 
 
 def sources(lib: str | None = None) -> list[Path]:
-    """Translation units of a library (of all, without a name). api.cu, the plumbing, is part of both."""
+    """Translation units of a library (of all, without a name). api.cu, the plumbing, is part of each."""
     out = sorted(CSRC.glob("*.cu"))
     if lib is None:
         return out
-    return [p for p in out if p.stem == "api" or p.stem.startswith("hybrid_") == (lib == "hybrid")]
+    if lib in _UNITS:
+        return [p for p in out if p.stem in _UNITS[lib]]
+    return [p for p in out if not p.stem.startswith("hybrid_")]
 
 
 def _stale(target: Path, deps: list[Path]) -> bool:
@@ -59,7 +69,7 @@ def _stale(target: Path, deps: list[Path]) -> bool:
     return any(d.stat().st_mtime > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False, libs: tuple[str, ...] = ("sparse", "hybrid")) -> Path:
+def build(force: bool = False, verbose: bool = False, libs: tuple[str, ...] = tuple(LIBS)) -> Path:
     """Compiles what is stale of the named libraries and returns the path of the first one. DJV_NVCC_FLAGS in the
     environment adds flags (e.g. -DDJV_RING_TRACE for the phase stamps of the one-pass MLP kernel; use --force, the
     flag is not part of the staleness check)."""
@@ -107,7 +117,7 @@ if __name__ == "__main__":
     ap.add_argument("--verbose", action="store_true", help="print ptxas register / shared-memory usage")
     ap.add_argument("--lib", choices=sorted(LIBS), help="build this library only")
     a = ap.parse_args()
-    names = (a.lib,) if a.lib else ("sparse", "hybrid")
+    names = (a.lib,) if a.lib else tuple(LIBS)
     build(force=a.force, verbose=a.verbose, libs=names)
     for name in names:
         print(LIBS[name])

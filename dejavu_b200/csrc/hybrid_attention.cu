@@ -18,113 +18,6 @@ namespace djv {
 
 namespace cg = cooperative_groups;
 
-// ---- rotary positions ------------------------------------------------------------------------------------------
-// One block per row; the angles of the row's position are shared by its heads.
-template <typename T, bool VEC>
-__global__ void rotary_kernel(T *__restrict__ buf, long long ld, const float *__restrict__ freqs, float amp,
-                              const long long *__restrict__ pos, int n, int heads, int dim, int half) {
-  extern __shared__ float cs[];  // cos[half], sin[half]
-  pdl_prologue();
-  const long long row = blockIdx.x;
-  const int b = (int)(row / n), t = (int)(row % n);
-  const float p = (float)(pos[b] + t);
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    float s, c;
-    sincosf(p * freqs[i], &s, &c);
-    cs[i] = c * amp;
-    cs[half + i] = s * amp;
-  }
-  __syncthreads();
-  T *x = buf + row * ld;
-  if (VEC) {  // half is a multiple of the 16-byte chunk
-    constexpr int N = Chunk<T>::N;
-    const int per = half / N;
-    for (int k = threadIdx.x; k < heads * per; k += blockDim.x) {
-      const int h = k / per, i = (k - h * per) * N;
-      uint4 *pu = reinterpret_cast<uint4 *>(x + (size_t)h * dim + i);
-      uint4 *pv = reinterpret_cast<uint4 *>(x + (size_t)h * dim + half + i);
-      float u[N], v[N];
-      T ru[N], rv[N];
-      unpack_chunk<T>(*pu, u);
-      unpack_chunk<T>(*pv, v);
-#pragma unroll
-      for (int e = 0; e < N; ++e) {
-        const float c = cs[i + e], s = cs[half + i + e];
-        ru[e] = from_f<T>(u[e] * c - v[e] * s);
-        rv[e] = from_f<T>(v[e] * c + u[e] * s);
-      }
-      *pu = *reinterpret_cast<uint4 *>(ru);
-      *pv = *reinterpret_cast<uint4 *>(rv);
-    }
-    return;
-  }
-  for (int k = threadIdx.x; k < heads * half; k += blockDim.x) {
-    const int h = k / half, i = k % half;
-    T *e = x + (size_t)h * dim + i;
-    const float u = to_f(e[0]), v = to_f(e[half]);
-    e[0] = from_f<T>(u * cs[i] - v * cs[half + i]);
-    e[half] = from_f<T>(v * cs[i] + u * cs[half + i]);
-  }
-}
-
-// ---- a portion of new tokens, any element type -----------------------------------------------------------------
-// A warp per (query, head): lanes take 32 keys at a time for the scores, then dv / 32 value columns each.
-constexpr int WA_WARPS = 8;
-
-template <typename T, int E>  // E * 32 >= dv
-__global__ void __launch_bounds__(WA_WARPS * WARP) window_attn_simple_kernel(WindowArgs a) {
-  extern __shared__ float q_sm[];  // WA_WARPS * dk
-  pdl_prologue();
-  const int warp = threadIdx.x / WARP, lane = threadIdx.x % WARP;
-  const int t = blockIdx.x * WA_WARPS + warp, h = blockIdx.y, b = blockIdx.z;
-  if (t >= a.n) return;
-  const int g = h / (a.H / a.G);
-  const long long p0 = a.pos[b], p = p0 + t;
-  const T *rows = static_cast<const T *>(a.qkv) + (size_t)b * a.n * a.ld;
-  float *q = q_sm + warp * a.dk;
-  for (int i = lane; i < a.dk; i += WARP) q[i] = to_f(rows[(size_t)t * a.ld + (size_t)h * a.dk + i]);
-  __syncwarp();
-  const T *kr = static_cast<const T *>(a.k_ring) + ((size_t)b * a.G + g) * a.cap * a.dk;
-  const T *vr = static_cast<const T *>(a.v_ring) + ((size_t)b * a.G + g) * a.cap * a.dv;
-  const T *kn = rows + (size_t)(a.H + g) * a.dk;
-  const T *vn = rows + (size_t)(a.H + a.G) * a.dk + (size_t)g * a.dv;
-  float m = a.sink ? a.sink[h] : -INFINITY, l = a.sink ? 1.f : 0.f, o[E];
-#pragma unroll
-  for (int e = 0; e < E; ++e) o[e] = 0.f;
-  long long lo = p - a.window + 1;
-  if (lo < 0) lo = 0;
-  for (long long j0 = lo; j0 <= p; j0 += WARP) {
-    const long long j = j0 + lane;
-    float s = -INFINITY;
-    if (j <= p) {
-      const T *k = j < p0 ? kr + (size_t)(j % a.cap) * a.dk : kn + (size_t)(j - p0) * a.ld;
-      s = 0.f;
-      for (int i = 0; i < a.dk; ++i) s = fmaf(q[i], to_f(k[i]), s);
-      s *= a.scale;
-    }
-    const float m_new = fmaxf(m, warp_max(s));
-    const float corr = m == -INFINITY ? 0.f : expf(m - m_new);
-    const float w = j <= p ? expf(s - m_new) : 0.f;
-    l = l * corr + warp_sum(w);
-    m = m_new;
-#pragma unroll
-    for (int e = 0; e < E; ++e) o[e] *= corr;
-    const int cnt = (int)min((long long)WARP, p - j0 + 1);
-    for (int c = 0; c < cnt; ++c) {
-      const float wc = __shfl_sync(0xffffffffu, w, c);
-      const long long jj = j0 + c;
-      const T *v = jj < p0 ? vr + (size_t)(jj % a.cap) * a.dv : vn + (size_t)(jj - p0) * a.ld;
-#pragma unroll
-      for (int e = 0; e < E; ++e)
-        if (e * WARP + lane < a.dv) o[e] = fmaf(wc, to_f(v[e * WARP + lane]), o[e]);
-    }
-  }
-  T *out = static_cast<T *>(a.out) + (((size_t)b * a.n + t) * a.H + h) * a.dv;
-#pragma unroll
-  for (int e = 0; e < E; ++e)
-    if (e * WARP + lane < a.dv) out[e * WARP + lane] = from_f<T>(o[e] / l);
-}
-
 // ---- the new tokens enter the rings ----------------------------------------------------------------------------
 template <typename T>
 __global__ void window_store_kernel(T *__restrict__ k_ring, T *__restrict__ v_ring, const T *__restrict__ qkv,
@@ -195,7 +88,7 @@ __global__ void __launch_bounds__(WD_THREADS) window_decode_kernel(DecodeArgs d)
   const int g = blockIdx.x / d.subs, sub = blockIdx.x % d.subs, b = blockIdx.y, sp = blockIdx.z;
   const int rep = a.H / a.G, r0 = sub * RT, nr = min(RT, rep - r0), h0 = g * rep + r0;
   const long long p = a.pos[b];
-  const T *row = static_cast<const T *>(a.qkv) + (size_t)b * a.ld;
+  const T *row = static_cast<const T *>(a.q) + (size_t)b * a.ldq;
   const T *k_new = row + (size_t)(a.H + g) * dk;
   const T *v_new = row + (size_t)(a.H + a.G) * dk + (size_t)g * dv;
   T *kr = static_cast<T *>(d.k_ring) + ((size_t)b * a.G + g) * a.cap * dk;
@@ -498,20 +391,6 @@ static int dispatch_decode(const DecodeArgs &d, int max_split, bool vec, cudaStr
   return dispatch_decode<T, 8>(d, nsplit, vec, st);
 }
 
-template <typename T>
-static int launch_simple(const WindowArgs &a, cudaStream_t st) {
-  const dim3 grid(ceil_div(a.n, WA_WARPS), a.H, a.B);
-  const size_t smem = (size_t)WA_WARPS * a.dk * 4;
-#define DJV_WA(E_) djv::launch_kernel(window_attn_simple_kernel<T, E_>, grid, dim3(WA_WARPS * WARP), smem, st, a)
-  if (a.dv <= 64) DJV_WA(2);
-  else if (a.dv <= 128) DJV_WA(4);
-  else if (a.dv <= 256) DJV_WA(8);
-  else DJV_WA(16);
-#undef DJV_WA
-  count_launch();
-  return check_launch("window_attn");
-}
-
 }  // namespace djv
 
 using namespace djv;
@@ -528,31 +407,14 @@ static int check_window(const char *op, int dtype, const void *qkv, const void *
   return DJV_OK;
 }
 
-extern "C" int djv_rotary(int dtype, void *buf, long long ld, const float *freqs, float amp, const long long *pos, int B,
-                          int n, int heads, int dim, int half, void *stream) {
-  DJV_REQUIRE(dtype == DJV_DTYPE_BF16 || dtype == DJV_DTYPE_F32, "rotary: dtype %d", dtype);
-  DJV_REQUIRE(buf && freqs && pos, "rotary: null pointer");
-  DJV_REQUIRE(B >= 1 && n >= 1 && heads >= 1 && half >= 1 && 2 * half <= dim && half <= 4096 &&
-                  ld >= (long long)heads * dim && (long long)B * n < (1ll << 31),
-              "rotary: B=%d n=%d heads=%d dim=%d half=%d", B, n, heads, dim, half);
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const int chunk = 16 / (int)dtype_bytes(dtype);
-  const bool vec = half % chunk == 0 && dim % chunk == 0 && ld % chunk == 0 && aligned16(buf);
-  int threads = ceil_div(vec ? heads * half / chunk : ceil_div(heads * half, 4), WARP) * WARP;
-  threads = threads > 512 ? 512 : threads;
-#define DJV_ROT(T_, VEC_)                                                                                             \
-  djv::launch_kernel(rotary_kernel<T_, VEC_>, B * n, threads, half * 8, st, static_cast<T_ *>(buf), ld, freqs, amp, pos, \
-                     n, heads, dim, half)
-  if (dtype == DJV_DTYPE_BF16) {
-    if (vec) DJV_ROT(bf16, true);
-    else DJV_ROT(bf16, false);
-  } else {
-    if (vec) DJV_ROT(float, true);
-    else DJV_ROT(float, false);
-  }
-#undef DJV_ROT
-  count_launch();
-  return check_launch("rotary");
+// q, k and v side by side in the rows of one projection, earlier tokens in the rings
+static WindowArgs fused_args(int dtype, void *out, const void *qkv, long long ld, const void *k_ring, const void *v_ring,
+                             const float *sink, const long long *pos, int B, int n, int H, int G, int dk, int dv, int cap,
+                             int window, float scale) {
+  const char *k = static_cast<const char *>(qkv) + (size_t)H * dk * dtype_bytes(dtype);
+  const char *v = k + (size_t)G * dk * dtype_bytes(dtype);
+  return WindowArgs{out, qkv, ld, k, ld, v, ld, nullptr, 0, 0, nullptr, 0, k_ring, v_ring, sink, pos, B, n, H, G, dk, dv,
+                    cap, 0, window, scale};
 }
 
 extern "C" int djv_window_attn(int dtype, void *out, const void *qkv, long long ld, const void *k_ring,
@@ -562,10 +424,8 @@ extern "C" int djv_window_attn(int dtype, void *out, const void *qkv, long long 
   if (rc) return rc;
   DJV_REQUIRE(out, "window_attn: null output");
   if (window > cap) window = cap;  // a ring that is shorter than the window holds the longest sequence
-  const WindowArgs a{out, qkv, ld, k_ring, v_ring, sink, pos, B, n, H, G, dk, dv, cap, window, scale};
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dtype == DJV_DTYPE_BF16) return window_prefill_supported(a) ? window_prefill(a, st) : launch_simple<bf16>(a, st);
-  return launch_simple<float>(a, st);
+  const WindowArgs a = fused_args(dtype, out, qkv, ld, k_ring, v_ring, sink, pos, B, n, H, G, dk, dv, cap, window, scale);
+  return window_attn_portion(dtype, a, static_cast<cudaStream_t>(stream));
 }
 
 extern "C" int djv_window_store(int dtype, void *k_ring, void *v_ring, const void *qkv, long long ld,
@@ -599,7 +459,7 @@ extern "C" int djv_window_attn_decode(int dtype, void *out, const void *qkv, lon
   DJV_REQUIRE(half >= 0 && 2 * half <= dk, "window_attn_decode: %d rotary pairs in %d dimensions", half, dk);
   if (window > cap) window = cap;
   DecodeArgs d = {};
-  d.w = WindowArgs{out, qkv, ld, k_ring, v_ring, sink, pos, B, 1, H, G, dk, dv, cap, window, scale};
+  d.w = fused_args(dtype, out, qkv, ld, k_ring, v_ring, sink, pos, B, 1, H, G, dk, dv, cap, window, scale);
   d.k_ring = k_ring;
   d.v_ring = v_ring;
   d.freqs = freqs;

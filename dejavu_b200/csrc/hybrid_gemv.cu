@@ -14,7 +14,7 @@ rowdot_any_kernel(TO *__restrict__ Y, const T *__restrict__ W, const T *__restri
   pdl_prologue();
   const int lane = threadIdx.x % WARP, b = blockIdx.y;
   const int o = blockIdx.x * 8 + threadIdx.x / WARP;
-  const int rows = act == DJV_ACT_CLAMPED_GLU ? 2 : 1;
+  const int rows = is_glu(act) ? 2 : 1;
   const int M_out = M / rows;
   if (o >= M_out) return;
   float s[2] = {0.f, 0.f};
@@ -26,6 +26,7 @@ rowdot_any_kernel(TO *__restrict__ Y, const T *__restrict__ W, const T *__restri
   if (lane) return;
   float v = s[0];
   if (act == DJV_ACT_CLAMPED_GLU) v = clamped_glu(s[0], s[1], p);
+  if (act == DJV_ACT_SILU_GLU) v = silu_glu(s[0], s[1]);
   if (act == DJV_ACT_SOFTCAP) v = apply_act_param<DJV_ACT_SOFTCAP>(v, p);
   Y[(size_t)b * M_out + o] = from_f<TO>(v);
 }
@@ -33,7 +34,7 @@ rowdot_any_kernel(TO *__restrict__ Y, const T *__restrict__ W, const T *__restri
 template <typename T, typename TO, int B, int ACT>
 static void launch_rowdot_dense(TO *Y, const T *W, const T *X, int M, int N, long long ldw, float param,
                                 cudaStream_t st) {
-  constexpr int R = (B <= 2 || ACT == DJV_ACT_CLAMPED_GLU) ? 2 : 1;
+  constexpr int R = (B <= 2 || is_glu(ACT)) ? 2 : 1;
   const RowdotPlan p = plan_rowdot(M, N / Chunk<T>::N, B, R);
 #define DJV_RD(WPR_)                                                                                            \
   djv::launch_kernel(rowdot_kernel<T, TO, B, ACT, WPR_, R, 4>, p.grid, RD_THREADS, 0, st, Y, W, X,              \
@@ -87,7 +88,7 @@ static bool try_mma(TO *, const float *, const float *, int, int, int, long long
 
 template <typename T, typename TO, int ACT>
 static int dense(TO *Y, const T *W, const T *X, int B, int M, int N, long long ldw, float param, cudaStream_t st) {
-  const int M_out = ACT == DJV_ACT_CLAMPED_GLU ? M / 2 : M;
+  const int M_out = is_glu(ACT) ? M / 2 : M;
   if (N % Chunk<T>::N != 0 || ldw % Chunk<T>::N != 0 || !aligned16(W) || !aligned16(X)) {
     djv::launch_kernel(rowdot_any_kernel<T, TO>, dim3(ceil_div(M_out, 8), B), dim3(256), 0, st, Y, W, X, M, N, ldw, ACT,
                        param);
@@ -119,7 +120,7 @@ extern "C" int djv_dense_gemv(int dtype, int out_dtype, void *y, const void *w, 
   DJV_REQUIRE(out_dtype == dtype || out_dtype == DJV_DTYPE_F32, "dense_gemv: output type %d", out_dtype);
   DJV_REQUIRE(B >= 1 && B <= DJV_MAX_BATCH, "dense_gemv: batch %d outside [1,%d]", B, DJV_MAX_BATCH);
   DJV_REQUIRE(N >= 1 && M >= 1 && ldw >= N, "dense_gemv: N=%d M=%d ldw=%lld", N, M, ldw);
-  DJV_REQUIRE(act != DJV_ACT_CLAMPED_GLU || M % 2 == 0, "dense_gemv: a gated unit needs an even number of rows");
+  DJV_REQUIRE(!is_glu(act) || M % 2 == 0, "dense_gemv: a gated unit needs an even number of rows");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   int rc = DJV_OK;
 #define DJV_DENSE(T_, TO_, ACT_)                                                                                   \
@@ -136,6 +137,9 @@ extern "C" int djv_dense_gemv(int dtype, int out_dtype, void *y, const void *w, 
   } else if (act == DJV_ACT_CLAMPED_GLU && out_dtype == dtype) {
     if (b16) DJV_DENSE(bf16, bf16, DJV_ACT_CLAMPED_GLU);
     else DJV_DENSE(float, float, DJV_ACT_CLAMPED_GLU);
+  } else if (act == DJV_ACT_SILU_GLU && out_dtype == dtype) {
+    if (b16) DJV_DENSE(bf16, bf16, DJV_ACT_SILU_GLU);
+    else DJV_DENSE(float, float, DJV_ACT_SILU_GLU);
   } else {
     set_error("dense_gemv: activation %d with output type %d is not compiled", act, out_dtype);
     return DJV_ERR_UNSUPPORTED;

@@ -5,10 +5,11 @@
 //   P goes back to TMEM over S as two bf16 terms, p = hi + lo, so that the weights keep their fp32 value to 2^-17;
 //   O (TMEM, 128 x dv fp32) += P_hi V + P_lo V.
 // O is only rescaled when a row's maximum grows by more than 2^8 (the final division by the sum makes up for the rest).
-// Keys come from the ring (tokens before the portion) or from the projection's output (the portion's own), row by row,
-// with 16-byte asynchronous copies into the swizzled operand layout. Two blocks share a multiprocessor: one computes
-// its softmax while the other's products run. V of a tile loads behind its scores, K of the next one behind the
-// values' products.
+// Keys come from the ring (tokens before the portion) or from the projection's output (the portion's own), or, where the
+// caller has put earlier tokens before the portion's, from rows on both sides; the last dimensions of a key may come from
+// rows that all heads share. They are fetched row by row, with 16-byte asynchronous copies into the swizzled operand
+// layout. Two blocks share a multiprocessor: one computes its softmax while the other's products run. V of a tile loads
+// behind its scores, K of the next one behind the values' products.
 #include "../../include/dejavu_b200_hybrid.h"
 #include "hybrid_attention.cuh"
 #include "tcgen05.cuh"
@@ -79,66 +80,78 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
   __syncwarp();
   if (warp == 0) tmem_alloc(&tmem_slot, COLS);
 
-  const bf16 *rows = static_cast<const bf16 *>(a.qkv) + (size_t)b * a.n * a.ld;
-  const bf16 *kr = static_cast<const bf16 *>(a.k_ring) + ((size_t)b * a.G + g) * a.cap * a.dk;
-  const bf16 *vr = static_cast<const bf16 *>(a.v_ring) + ((size_t)b * a.G + g) * a.cap * a.dv;
+  const size_t first = (size_t)b * (a.past + a.n) + a.past;  // row of the portion's first token among the keys
+  const int own = a.dk - a.rot, rot = a.rot;  // key dimensions of the head itself, and those all heads share
+  const bf16 *q_rows = static_cast<const bf16 *>(a.q) + (size_t)b * a.n * a.ldq + (size_t)h * a.dk;
+  const bf16 *k_new = static_cast<const bf16 *>(a.k) + first * a.ldk + (size_t)g * own;
+  const bf16 *v_new = static_cast<const bf16 *>(a.v) + first * a.ldv + (size_t)g * a.dv;
+  const bf16 *t_new = rot ? static_cast<const bf16 *>(a.tail) + first * a.ldt : k_new;
+  const bool ring = a.k_ring != nullptr;  // where the tokens before the portion are: rings, or the rows before the portion's
+  const bf16 *kr = ring ? static_cast<const bf16 *>(a.k_ring) + ((size_t)b * a.G + g) * a.cap * a.dk : k_new;
+  const bf16 *vr = ring ? static_cast<const bf16 *>(a.v_ring) + ((size_t)b * a.G + g) * a.cap * a.dv : v_new;
   const long long p0 = a.pos[b];
   const int last = min(t0 + WP_TILE, a.n) - 1;
   // everything below is relative to the portion: key j of the portion is token j, the ring holds j < 0
-  const long long reach = p0 < (long long)a.window - 1 ? p0 : (long long)a.window - 1;  // ring tokens the portion can see
+  long long reach = p0 < (long long)a.window - 1 ? p0 : (long long)a.window - 1;  // earlier tokens the portion can see
+  if (!ring && reach > a.past) reach = a.past;
   int lo = t0 - (a.window - 1);
   if (lo < -(int)reach) lo = -(int)reach;
   const int tiles = (last - lo) / WP_TILE + 1;
   const int ring_slot0 = (int)((p0 - reach) % a.cap);  // slot of token -reach
 
   // One tile of keys or values. The chunk a thread copies is the same in every row, so a tile of the portion's own
-  // tokens is a pointer that advances by a fixed number of rows.
-  auto load = [&](uint32_t dst, int j0, const bf16 *ring, int dim, const bf16 *fresh, auto blocks) {
-    constexpr int PER_ROW = decltype(blocks)::value * 8, STEP = WP_THREADS / PER_ROW, ROUNDS = WP_TILE / STEP;
-    const int ch = tid & (PER_ROW - 1), r0 = tid / PER_ROW;
-    const bool inside = ch * 8 < dim;
-    if (j0 >= 0 && j0 + WP_TILE - 1 <= last) {
-      const bf16 *src = fresh + (size_t)(j0 + r0) * a.ld + ch * 8;
-      const size_t step = (size_t)STEP * a.ld;
-      if (!inside) src = fresh;  // (not read)
+  // tokens (or of rows before them) is a pointer that advances by a fixed number of rows. Three blocks of 64 elements go
+  // one by one, so that a row's chunks are a power of two.
+  auto load = [&](uint32_t dst, int j0, const bf16 *ring_rows, int dim, const bf16 *fresh, long long ld, int head_dim,
+                  auto blocks) {
+    constexpr int NB = decltype(blocks)::value, PASSES = NB == 3 ? 3 : 1;
+    constexpr int PER_ROW = NB / PASSES * 8, STEP = WP_THREADS / PER_ROW, ROUNDS = WP_TILE / STEP;
+    const int r0 = tid / PER_ROW;
 #pragma unroll
-      for (int it = 0; it < ROUNDS; ++it) {
-        cp_async16_zfill(dst + sw128_offset(WP_TILE, r0 + it * STEP, ch), src, inside ? 16 : 0);
-        if (inside) src += step;
-      }
-    } else {
-      for (int x = r0; x < WP_TILE; x += STEP) {
-        const int j = j0 + x;
-        const bf16 *src = fresh;
-        const bool ok = inside && j <= last;
-        if (ok) {
-          if (j >= 0) {
-            src = fresh + (size_t)j * a.ld + ch * 8;
-          } else {
-            int slot = ring_slot0 + (j + (int)reach);
-            if (slot >= a.cap) slot -= a.cap;
-            src = ring + (size_t)slot * dim + ch * 8;
-          }
+    for (int ps = 0; ps < PASSES; ++ps) {
+      const int ch = ps * 8 + (tid & (PER_ROW - 1));
+      const bool inside = ch * 8 < dim, shared = ch * 8 >= head_dim;
+      const bf16 *col = shared ? t_new + (ch * 8 - head_dim) : fresh + ch * 8;
+      const long long step1 = shared ? a.ldt : ld;
+      if ((!ring || j0 >= 0) && j0 + WP_TILE - 1 <= last) {
+        const bf16 *src = inside ? col + (long long)(j0 + r0) * step1 : fresh;  // (not read outside)
+        const long long step = (long long)STEP * step1;
+#pragma unroll
+        for (int it = 0; it < ROUNDS; ++it) {
+          cp_async16_zfill(dst + sw128_offset(WP_TILE, r0 + it * STEP, ch), src, inside ? 16 : 0);
+          if (inside) src += step;
         }
-        cp_async16_zfill(dst + sw128_offset(WP_TILE, x, ch), src, ok ? 16 : 0);
+      } else {
+        for (int x = r0; x < WP_TILE; x += STEP) {
+          const int j = j0 + x;
+          const bf16 *src = fresh;
+          const bool ok = inside && j <= last;
+          if (ok) {
+            if (!ring || j >= 0) {
+              src = col + (long long)j * step1;
+            } else {
+              int slot = ring_slot0 + (j + (int)reach);
+              if (slot >= a.cap) slot -= a.cap;
+              src = ring_rows + (size_t)slot * dim + ch * 8;
+            }
+          }
+          cp_async16_zfill(dst + sw128_offset(WP_TILE, x, ch), src, ok ? 16 : 0);
+        }
       }
     }
     cp_async_commit();
   };
   const std::integral_constant<int, KB> kb;
   const std::integral_constant<int, VB> vb;
-  const bf16 *k_new = rows + (size_t)(a.H + g) * a.dk;
-  const bf16 *v_new = rows + (size_t)(a.H + a.G) * a.dk + (size_t)g * a.dv;
   {  // queries
-    constexpr int PER_ROW = KB * 8;
-    const int ch = tid & (PER_ROW - 1);
-    for (int x = tid / PER_ROW; x < WP_TILE; x += WP_THREADS / PER_ROW) {
+    for (int i = tid; i < WP_TILE * KB * 8; i += WP_THREADS) {
+      const int x = i / (KB * 8), ch = i - x * (KB * 8);
       const bool ok = ch * 8 < a.dk && t0 + x <= last;
-      cp_async16_zfill(q_sm + sw128_offset(WP_TILE, x, ch),
-                       ok ? rows + (size_t)(t0 + x) * a.ld + (size_t)h * a.dk + ch * 8 : rows, ok ? 16 : 0);
+      cp_async16_zfill(q_sm + sw128_offset(WP_TILE, x, ch), ok ? q_rows + (size_t)(t0 + x) * a.ldq + ch * 8 : q_rows,
+                       ok ? 16 : 0);
     }
   }
-  load(k_sm, lo, kr, a.dk, k_new, kb);
+  load(k_sm, lo, kr, a.dk, k_new, a.ldk, own, kb);
 
   const float sink = a.sink ? a.sink[h] * 1.4426950408889634f : 0.f;
   const float c = a.scale * 1.4426950408889634f;  // scores in units of log 2
@@ -176,7 +189,7 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
       }
       mma_commit(&bar_s);
     }
-    load(v_sm, j0, vr, a.dv, v_new, vb);
+    load(v_sm, j0, vr, a.dv, v_new, a.ldv, a.dv, vb);
     if (!dead) dead = !mbar_wait(&bar_s, i & 1);
     __syncwarp();
     tmem_fence_after();
@@ -284,7 +297,7 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
         mma_ts(tm_o, tm_s + 64 + k * 8, v_desc + (uint64_t)(k * 128), idesc_o, true);
       mma_commit(&bar_o);
     }
-    if (i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, kb);  // behind the values' products
+    if (i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, a.ldk, own, kb);  // behind the values' products
   }
   if (!dead) dead = !mbar_wait(&bar_o, (tiles - 1) & 1);
   __syncwarp();
@@ -294,6 +307,7 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
   __syncthreads();
   const float inv = 1.f / (l + exch[half ^ 1][r]);
   bf16 *out = static_cast<bf16 *>(a.out) + (((size_t)b * a.n + row) * a.H + h) * a.dv;
+  const bf16 *gate = a.gate ? static_cast<const bf16 *>(a.gate) + ((size_t)b * a.n + row) * a.ldg + (size_t)h * a.dv : nullptr;
   for (int q = half * 16; q < dvp; q += 32) {
     uint32_t o[16];
     tmem_ld16(o, tm_o + lane_base + q);
@@ -302,11 +316,20 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
 #pragma unroll
       for (int e = 0; e < 16; e += 8) {
         if (q + e < a.dv) {  // dv % 8 == 0
+          float f[8];
+#pragma unroll
+          for (int x = 0; x < 8; ++x) f[x] = __uint_as_float(o[e + x]) * inv;
+          if (gate) {
+            float z[8];
+            unpack_chunk<bf16>(*reinterpret_cast<const uint4 *>(gate + q + e), z);
+#pragma unroll
+            for (int x = 0; x < 8; ++x) f[x] *= sigmoid_f(z[x]);
+          }
           uint4 v;
-          v.x = pack_bf16(__uint_as_float(o[e]) * inv, __uint_as_float(o[e + 1]) * inv);
-          v.y = pack_bf16(__uint_as_float(o[e + 2]) * inv, __uint_as_float(o[e + 3]) * inv);
-          v.z = pack_bf16(__uint_as_float(o[e + 4]) * inv, __uint_as_float(o[e + 5]) * inv);
-          v.w = pack_bf16(__uint_as_float(o[e + 6]) * inv, __uint_as_float(o[e + 7]) * inv);
+          v.x = pack_bf16(f[0], f[1]);
+          v.y = pack_bf16(f[2], f[3]);
+          v.z = pack_bf16(f[4], f[5]);
+          v.w = pack_bf16(f[6], f[7]);
           *reinterpret_cast<uint4 *>(out + q + e) = v;
         }
       }
@@ -333,12 +356,15 @@ static int launch_window_prefill(const WindowArgs &a, cudaStream_t st) {
 }
 
 bool window_prefill_supported(const WindowArgs &a) {
-  return a.dk % 8 == 0 && a.dv % 8 == 0 && a.dk <= 256 && a.dv <= 256 && a.ld % 8 == 0 && aligned16(a.qkv) &&
-         aligned16(a.k_ring) && aligned16(a.v_ring) && aligned16(a.out);
+  if (!(aligned16(a.k_ring) && aligned16(a.v_ring))) return false;
+  if (a.rot && !(a.rot % 8 == 0 && a.ldt % 8 == 0 && aligned16(a.tail))) return false;
+  if (a.gate && !(a.ldg % 8 == 0 && aligned16(a.gate))) return false;
+  return a.dk % 8 == 0 && a.dv % 8 == 0 && a.dk <= 256 && a.dv <= 256 && a.ldq % 8 == 0 && a.ldk % 8 == 0 &&
+         a.ldv % 8 == 0 && aligned16(a.q) && aligned16(a.k) && aligned16(a.v) && aligned16(a.out);
 }
 
 int window_prefill(const WindowArgs &a, cudaStream_t st) {
-  const int kb = a.dk <= 64 ? 1 : (a.dk <= 128 ? 2 : 4), vb = a.dv <= 64 ? 1 : (a.dv <= 128 ? 2 : 4);
+  const int kb = a.dk <= 64 ? 1 : (a.dk <= 128 ? 2 : (a.dk <= 192 ? 3 : 4)), vb = a.dv <= 64 ? 1 : (a.dv <= 128 ? 2 : 4);
 #define DJV_WP(K_, V_) \
   if (kb == K_ && vb == V_) return launch_window_prefill<K_, V_>(a, st)
   DJV_WP(1, 1);
@@ -347,6 +373,9 @@ int window_prefill(const WindowArgs &a, cudaStream_t st) {
   DJV_WP(2, 1);
   DJV_WP(2, 2);
   DJV_WP(2, 4);
+  DJV_WP(3, 1);
+  DJV_WP(3, 2);
+  DJV_WP(3, 4);
   DJV_WP(4, 1);
   DJV_WP(4, 2);
   return launch_window_prefill<4, 4>(a, st);

@@ -12,6 +12,15 @@ __device__ __forceinline__ float clamped_glu(float gate, float up, float limit) 
   return g * sigmoid_f(1.702f * g) * (u + 1.f);
 }
 
+__device__ __forceinline__ float silu_glu(float gate, float up) { return gate * sigmoid_f(gate) * up; }
+
+// gated units: two rows of the matrix make one output
+__host__ __device__ constexpr bool is_glu(int act) { return act == DJV_ACT_CLAMPED_GLU || act == DJV_ACT_SILU_GLU; }
+template <int ACT>
+__device__ __forceinline__ float apply_glu(float gate, float up, float p) {
+  return ACT == DJV_ACT_CLAMPED_GLU ? clamped_glu(gate, up, p) : silu_glu(gate, up);
+}
+
 // activations that take a constant, next to those that do not
 template <int ACT>
 __device__ __forceinline__ float apply_act_param(float v, float p) {
@@ -33,7 +42,7 @@ __global__ void __launch_bounds__(RD_THREADS)
 rowdot_kernel(TO *__restrict__ Y, const T *__restrict__ W, const T *__restrict__ X,
               const void *__restrict__ idx, const T *__restrict__ bias, int M, int N,
               long long ldw, int idx64, int early, float act_param) {
-  static_assert(ACT != DJV_ACT_CLAMPED_GLU || ROWS % 2 == 0, "a group owns whole (gate, up) pairs of rows");
+  static_assert(!is_glu(ACT) || ROWS % 2 == 0, "a group owns whole (gate, up) pairs of rows");
   constexpr int GROUPS = RD_WARPS / WPR;
   constexpr int GLANES = WARP * WPR;
   __shared__ float red[WPR > 1 ? RD_WARPS * ROWS * B : 1];
@@ -137,7 +146,7 @@ rowdot_kernel(TO *__restrict__ Y, const T *__restrict__ W, const T *__restrict__
       }
     }
     if (wig == 0 && lane == 0) {
-      if (ACT == DJV_ACT_CLAMPED_GLU) {
+      if (is_glu(ACT)) {
         // rows 2i, 2i + 1 of the matrix are the gate and up rows of output i
 #pragma unroll
         for (int j = 0; j + 1 < ROWS; j += 2) {
@@ -146,7 +155,7 @@ rowdot_kernel(TO *__restrict__ Y, const T *__restrict__ W, const T *__restrict__
 #pragma unroll
             for (int b = 0; b < B; ++b)
               Y[(size_t)b * (M / 2) + m / 2] =
-                  from_f<TO>(clamped_glu(acc[j][b] + bv[j], acc[j + 1][b] + bv[j + 1], act_param));
+                  from_f<TO>(apply_glu<ACT>(acc[j][b] + bv[j], acc[j + 1][b] + bv[j + 1], act_param));
           }
         }
       } else {

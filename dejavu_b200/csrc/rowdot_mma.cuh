@@ -125,10 +125,10 @@ rowdot_mma_kernel(TO *__restrict__ Y, const T *__restrict__ W, const T *__restri
           }
           return s;
         };
-        if (ACT == DJV_ACT_CLAMPED_GLU) {
+        if (is_glu(ACT)) {
           // rows 2i, 2i + 1 are the gate and up rows of output i (no bias in this form)
           if (row % 2 == 0 && m + 1 < M)
-            Y[(size_t)tok * (M / 2) + m / 2] = from_f<TO>(clamped_glu(total(o), total(o + 8), act_param));
+            Y[(size_t)tok * (M / 2) + m / 2] = from_f<TO>(apply_glu<ACT>(total(o), total(o + 8), act_param));
         } else {
           float s = total(o);
           if (bias != nullptr) s += to_f(bias[load_index(idx, m, idx64)]);

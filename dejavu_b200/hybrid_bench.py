@@ -187,7 +187,7 @@ def kernel_table(hyb, opt, opt_cfg, size, n, kernel_timing, gbs, tflops, dev) ->
     # flops of the recurrence itself: state update and read-out
     rec("prefill.gla", us, n * GH * (2 * gk + 3 * gv) * 2, 4.0 * n * GH * gk * gv)
     rows = [rand(n, 2 * size["ff"]) for _ in range(3)]
-    us = kernel_timing([lambda r=r: ops.clamped_glu(r, 7.0) for r in rows])
+    us = kernel_timing([lambda r=r: ops.glu(r, "clamped_glu", 7.0) for r in rows])
     rec("prefill.clamped_glu", us, n * size["ff"] * 6)
     import torch.nn.functional as F
 

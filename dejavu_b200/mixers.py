@@ -1,16 +1,16 @@
-"""Building blocks of hybrid decoders: linear layers, rotary positions, sliding-window attention with sinks, gated
-linear attention, clamped gated MLP, hyper-connected residual streams. bf16 (activations and products, fp32 where a
-comment says so) or fp32 throughout.
+"""Building blocks of hybrid decoders: linear layers, rotary positions, sliding-window attention with sinks, windowed
+latent attention, gated linear attention, matrix memories (mLSTM), gated MLPs, mixtures of experts, hyper-connected
+residual streams. bf16 (activations and products, fp32 where a comment says so) or fp32 throughout.
 
 Each block takes its sizes and constants as arguments and works on rows (B * n, features), B sequences of n new tokens
 each, with their first positions in a device tensor `pos` (B,). n == 1 is a decode step and runs the fused decode
 kernels; larger n is a portion of a prompt. A mixer owns no state: `new_cache` says what a sequence needs, the forward
-call gets it back.
+call gets it back. `past`, where a mixer takes it, is a bound the host knows on every sequence's position.
 """
 from __future__ import annotations
 
 import math
-from typing import Optional
+from typing import NamedTuple, Optional
 
 import torch
 import torch.nn as nn
@@ -37,6 +37,11 @@ class Linear(nn.Module):
         if out_dtype in (None, x.dtype):
             return torch.mm(x, self.weight.t())
         return torch.mm(x, self.weight.t(), out_dtype=out_dtype)
+
+    def part(self, x, first: int, last: int, out_dtype=None):
+        """Rows first .. last - 1 of the weight only."""
+        w = self.weight[first:last].t()
+        return torch.mm(x, w) if out_dtype in (None, x.dtype) else torch.mm(x, w, out_dtype=out_dtype)
 
     def rows(self, x, decode: bool, out_dtype=None):
         if decode and x.shape[0] <= _lib.MAX_BATCH:
@@ -100,7 +105,7 @@ class WindowAttention(nn.Module):
         return (torch.zeros(batch, self.kv_heads, cap, self.dim, device=device, dtype=dtype),
                 torch.zeros(batch, self.kv_heads, cap, self.vdim, device=device, dtype=dtype))
 
-    def forward(self, h, cache, pos, n: int):
+    def forward(self, h, cache, pos, n: int, past: int = 0):
         k_ring, v_ring = cache
         qkv = self.qkv.rows(h, n == 1)
         rot = self.rotary
@@ -133,33 +138,186 @@ class GatedLinearAttention(nn.Module):
         self.norm = _empty(vdim, device=device, dtype=torch.float32)
         self.o = Linear(heads * vdim, width, device, dtype)
 
+    def zero_padding(self):
+        self.proj.weight[sum(self.sizes):].zero_()
+
     def new_cache(self, batch: int, max_seqlen: int, device, dtype):
         """The recurrent state, fp32, whatever the model's type."""
         return (torch.zeros(batch, self.heads, self.dim, self.vdim, device=device, dtype=torch.float32),)
 
-    def forward(self, h, cache, pos, n: int):
+    def forward(self, h, cache, pos, n: int, past: int = 0):
         proj = self.proj.rows(h, n == 1)
         ctx = ops.gated_linear_attention(proj, self.a2, self.a2_bias, self.tau, self.norm, self.eps, self.scale,
                                          cache[0], pos, n)
         return self.o.rows(ctx, n == 1, torch.float32)
 
 
-class ClampedGatedMLP(nn.Module):
-    """down(min(gate, limit) * sigmoid(1.702 .) * (clamp(up, limit) + 1)); gate and up rows are interleaved in one
-    weight, so that a decode row's two products meet in one warp."""
+class MatrixMemory(nn.Module):
+    """mLSTM: a (dim, vdim) state per head with scalar exponential gates, kept in range by a running maximum, a normaliser
+    beside it, per-head RMS norm and a sigmoid gate. The state, the gates (from their projections on) and everything made
+    of them are fp32."""
 
-    def __init__(self, width: int, ff: int, limit: float, device=None, dtype=None):
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, gate_cap: float, eps: float, device=None, dtype=None):
         super().__init__()
-        self.ff, self.limit = ff, float(limit)
+        self.heads, self.dim, self.vdim = heads, dim, vdim
+        self.gate_cap, self.eps, self.scale = float(gate_cap), float(eps), dim ** -0.5
+        self.sizes = (heads * dim, heads * dim, heads * vdim, heads * vdim)  # q, k, v, output gate
+        # rows are padded so that every row of the product starts on a 16-byte boundary; the gates' rows come after them
+        self.main = -(-sum(self.sizes) // 8) * 8
+        self.proj = Linear(width, self.main + 2 * heads, device, dtype)
+        f32 = {"device": device, "dtype": torch.float32}
+        self.i_bias, self.f_bias, self.norm = _empty(heads, **f32), _empty(heads, **f32), _empty(heads * vdim, **f32)
+        self.o = Linear(heads * vdim, width, device, dtype)
+
+    def zero_padding(self):
+        self.proj.weight[sum(self.sizes):self.main].zero_()
+
+    def checkpoint_slots(self):
+        w, m, H = self.proj.weight, self.main, self.heads
+        return {**dict(zip("qkvg", w[:sum(self.sizes)].split(self.sizes))), "i": w[m:m + H], "f": w[m + H:],
+                "i.b": self.i_bias, "f.b": self.f_bias, "norm": self.norm, "o": self.o.weight}
+
+    def new_cache(self, batch: int, max_seqlen: int, device, dtype):
+        """The recurrent state, fp32, whatever the model's type."""
+        return (ops.mlstm_state(batch, self.heads, self.dim, self.vdim, device),)
+
+    def forward(self, h, cache, pos, n: int, past: int = 0):
+        if n == 1:  # one product for all projections, in fp32
+            proj = self.proj.rows(h, True, torch.float32)
+            gates = proj[:, self.main:]
+        else:
+            proj = self.proj.part(h, 0, self.main)
+            gates = self.proj.part(h, self.main, self.main + 2 * self.heads, torch.float32)
+        ctx = ops.mlstm(proj, gates, self.i_bias, self.f_bias, self.gate_cap, self.norm, self.eps, self.scale, cache[0],
+                        pos, n, self.dim, self.vdim, h.dtype)
+        return self.o.rows(ctx, n == 1, torch.float32)
+
+
+class LatentAttention(nn.Module):
+    """Causal attention over the last `window` tokens (None: all) whose keys and values are projections of one latent per
+    token, with a rotated key part that all heads share and a sigmoid gate on the output. Only latents and rotated parts
+    are cached. A prompt portion expands the latents in sight into keys and values; a decode step works on the latents
+    themselves. Scores and softmax are fp32."""
+
+    def __init__(self, width: int, heads: int, dim: int, rot_dim: int, vdim: int, rank: int, scale: float,
+                 window: Optional[int], rot: dict, eps: float, device=None, dtype=None):
+        super().__init__()
+        self.heads, self.dim, self.rot_dim, self.vdim, self.rank = heads, dim, rot_dim, vdim, rank
+        self.scale, self.window, self.eps = float(scale), window, float(eps)
+        self.sizes = (heads * (dim + rot_dim), rank + rot_dim, heads * vdim)  # q, latent and key part, output gate
+        self.proj = Linear(width, -(-sum(self.sizes) // 8) * 8, device, dtype)
+        self.norm = _empty(rank, device=device, dtype=torch.float32)
+        self.ukv = Linear(rank, heads * (dim + vdim), device, dtype)
+        self.o = Linear(heads * vdim, width, device, dtype)
+        self.rotary = RotaryTable(rot, device)
+        if self.rotary.dims != rot_dim:
+            raise ValueError(f"{self.rotary.dims} rotary dims in a rotated part of {rot_dim}")
+
+    def zero_padding(self):
+        self.proj.weight[sum(self.sizes):].zero_()
+
+    def checkpoint_slots(self):
+        q, d, g = self.proj.weight[:sum(self.sizes)].split(self.sizes)
+        uk, uv = self.ukv.weight.split((self.heads * self.dim, self.heads * self.vdim))
+        return {"q": q, "dkv": d, "g": g, "dkv.norm": self.norm, "uk": uk, "uv": uv, "o": self.o.weight}
+
+    def new_cache(self, batch: int, max_seqlen: int, device, dtype):
+        """A ring of the window's length: (batch, tokens, latent | rotated key part)."""
+        cap = max_seqlen if self.window is None else min(self.window, max_seqlen)
+        return (torch.zeros(batch, cap, self.rank + self.rot_dim, device=device, dtype=dtype),)
+
+    def forward(self, h, cache, pos, n: int, past: int = 0):
+        ring, = cache
+        H, dim, rot, rank = self.heads, self.dim, self.rot_dim, self.rank
+        window = self.window if self.window is not None else 2 ** 30
+        proj = self.proj.rows(h, n == 1)
+        a, b = self.sizes[0], self.sizes[0] + self.sizes[1]
+        gate = proj[:, b:b + self.sizes[2]]
+        if n == 1:
+            uk, uv = self.ukv.weight[:H * dim], self.ukv.weight[H * dim:]
+            ctx = ops.latent_attention_decode(proj, uk, uv, self.norm, self.eps, self.rotary.freqs, ring, gate, pos, H,
+                                              window, self.scale)
+            return self.o.rows(ctx, True, torch.float32)
+        past = min(past, window - 1, ring.shape[1])
+        ops.rotary_(proj[:, dim:], self.rotary.freqs, self.rotary.amp, pos, n, H, dim + rot, interleaved=True)
+        rows = ops.latent_rows(proj[:, a:b], ring, self.norm, self.eps, self.rotary.freqs, pos, n, past, rank)
+        kv = self.ukv(rows[:, :rank])
+        ctx = ops.latent_attention(proj[:, :a], kv, rows[:, rank:], gate, pos, n, past, H, dim, rot, window, self.scale)
+        ops.latent_store(rows, ring, self.norm, self.rotary.freqs, pos, n, past, rank)
+        return self.o(ctx, torch.float32)
+
+
+class GatedMLP(nn.Module):
+    """down(unit(gate, up)); the unit is "silu_glu" (silu(gate) * up) or "clamped_glu" (min(gate, limit) * sigmoid(1.702 .) *
+    (clamp(up, limit) + 1)). Gate and up rows are interleaved in one weight, so that a decode row's two products meet in one
+    warp."""
+
+    def __init__(self, width: int, ff: int, activation: str, limit: float = 0.0, device=None, dtype=None):
+        super().__init__()
+        self.ff, self.activation, self.limit = ff, activation, float(limit)
         self.gate_up = Linear(width, 2 * ff, device, dtype)
         self.down = Linear(ff, width, device, dtype)
 
+    def checkpoint_slots(self):
+        gu = self.gate_up.weight.view(self.ff, 2, -1)
+        return {"gate": gu[:, 0], "up": gu[:, 1], "down": self.down.weight}
+
     def forward(self, h, n: int):
         if n == 1 and h.shape[0] <= _lib.MAX_BATCH:
-            a = self.gate_up.decode(h, activation="clamped_glu", param=self.limit)
+            a = self.gate_up.decode(h, activation=self.activation, param=self.limit)
         else:
-            a = ops.clamped_glu(self.gate_up(h), self.limit)
+            a = ops.glu(self.gate_up(h), self.activation, self.limit)
         return self.down.rows(a, n == 1, torch.float32)
+
+
+class SplitSum(NamedTuple):
+    """A sublayer's output that the next boundary adds up: y (rows, width) fp32 or None, plus, for every row, the rows
+    `places` (rows, k) of `parts`."""
+
+    y: Optional[torch.Tensor]
+    parts: torch.Tensor
+    places: torch.Tensor
+
+
+class MixtureOfExperts(nn.Module):
+    """Every token goes through the `top` experts (silu gated units) with the largest scores sigmoid(router logits); the
+    scores multiply the experts' inputs and are not renormalised. A shared expert of its own size, if any, takes every
+    token. Router logits and scores are fp32.
+
+    A prompt portion is sorted by expert and runs as grouped products (SplitSum); a decode step reads the chosen experts'
+    weights only."""
+
+    def __init__(self, width: int, ff: int, experts: int, top: int, shared_ff: Optional[int] = None, device=None, dtype=None):
+        super().__init__()
+        if not 1 <= top <= experts:
+            raise ValueError(f"{top} of {experts} experts")
+        self.ff, self.experts, self.top = ff, experts, top
+        self.router = Linear(width, experts, device, dtype)
+        self.gate_up = _empty(experts, 2 * ff, width, device=device, dtype=dtype)
+        self.down = _empty(experts, width, ff, device=device, dtype=dtype)
+        self.shared = GatedMLP(width, shared_ff, "silu_glu", device=device, dtype=dtype) if shared_ff else None
+
+    def checkpoint_slots(self):
+        out = {"router": self.router.weight}
+        gu = self.gate_up.view(self.experts, self.ff, 2, -1)
+        for e in range(self.experts):
+            out.update({f"e{e}.gate": gu[e, :, 0], f"e{e}.up": gu[e, :, 1], f"e{e}.down": self.down[e]})
+        if self.shared is not None:
+            out.update({f"shared.{k}": v for k, v in self.shared.checkpoint_slots().items()})
+        return out
+
+    def forward(self, h, n: int):
+        z = self.router.rows(h, n == 1, torch.float32)
+        if n == 1 and h.shape[0] <= _lib.MAX_BATCH:
+            if self.shared is None:
+                return ops.moe_decode(h, z, self.gate_up, self.down, self.top)
+            if h.shape[0] <= 4:  # the shared expert runs beside the others; for more rows its products share their weights
+                return ops.moe_decode(h, z, self.gate_up, self.down, self.top, self.shared.gate_up.weight,
+                                      self.shared.down.weight)
+            return ops.moe_decode(h, z, self.gate_up, self.down, self.top, init=self.shared(h, n))
+        xs, ws, offsets, places = ops.moe_route(h, z, self.top)
+        a = ops.moe_grouped(xs, self.gate_up, offsets, ws, glu=True)
+        return SplitSum(None if self.shared is None else self.shared(h, n), ops.moe_grouped(a, self.down, offsets), places)
 
 
 class HyperConnection(nn.Module):

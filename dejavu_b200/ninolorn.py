@@ -15,10 +15,9 @@ from typing import Optional
 import torch
 import torch.nn as nn
 
-from . import ops
-from .generation import GenerationMixin, InferenceParams
-from .gpt import CausalLMOutput, _randn_big, _stable_hash
-from .mixers import ClampedGatedMLP, GatedLinearAttention, HyperConnection, Linear, WindowAttention, _empty
+from . import _lib, ops
+from .hybrid import HybridDecoder
+from .mixers import GatedLinearAttention, GatedMLP, HyperConnection, WindowAttention, _empty
 
 ARCHITECTURE = "Ninolorn"
 
@@ -57,7 +56,7 @@ class HybridLayer(nn.Module):
                                          dtype)
         self.norm1, self.hc1 = _empty(D, device=device, dtype=torch.float32), HyperConnection(cfg.streams, device)
         mlp = spec.get("mlp")
-        self.mlp = None if mlp is None else ClampedGatedMLP(D, mlp["ff"], mlp["limit"], device, dtype)
+        self.mlp = None if mlp is None else GatedMLP(D, mlp["ff"], "clamped_glu", mlp["limit"], device, dtype)
         if self.mlp is not None:
             self.norm2, self.hc2 = _empty(D, device=device, dtype=torch.float32), HyperConnection(cfg.streams, device)
 
@@ -74,8 +73,7 @@ class HybridLayer(nn.Module):
         parts["o"] = m.o.weight
         out = {f"mix.{k}": v for k, v in parts.items()}
         if self.mlp is not None:
-            gu = self.mlp.gate_up.weight.view(self.mlp.ff, 2, -1)
-            out.update({"mlp.gate": gu[:, 0], "mlp.up": gu[:, 1], "mlp.down": self.mlp.down.weight})
+            out.update({f"mlp.{k}": v for k, v in self.mlp.checkpoint_slots().items()})
         for q in ("1", "2") if self.mlp is not None else ("1",):
             hc = getattr(self, "hc" + q)
             out.update({"norm" + q: getattr(self, "norm" + q), f"hc{q}.in": hc.w_in, f"hc{q}.out": hc.w_out,
@@ -83,123 +81,41 @@ class HybridLayer(nn.Module):
         return out
 
 
-class NinolornForCausalLM(nn.Module, GenerationMixin):
-    """Same calls as the other models: forward(input_ids, position_ids, inference_params).logits, generate(...)."""
-
-    selects_logit_rows = True  # forward(logit_rows=...) computes logits at those tokens only
-    takes_portions = True      # a prompt may arrive in portions of any size
+class NinolornForCausalLM(HybridDecoder):
+    """The residual is `streams` parallel streams; `collect` receives their sum."""
 
     def __init__(self, config: dict, tensor_shapes: Optional[dict] = None, gla_rank: int = 16, device=None,
                  dtype=torch.bfloat16):
         """`config` is the parsed config.json. The rank of the decay projection and the presence of sinks follow
         `tensor_shapes` (name -> shape) when given, else `gla_rank` and True."""
-        super().__init__()
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError(f"this model runs in bfloat16 or float32, not {dtype}")
-        self.config = cfg = parse_config(config)
-        self.dtype = dtype
-        f = {"device": device, "dtype": dtype}
-        self.embed = _empty(cfg.vocab_size, cfg.hidden_size, **f)
-        self.layers = nn.ModuleList()
+        cfg = parse_config(config)
+        super().__init__(cfg, device, dtype)
         for i, spec in enumerate(cfg.layers):
             rank, sink = gla_rank, True
             if tensor_shapes is not None:
                 rank = tensor_shapes.get(f"l{i}.mix.a1", (gla_rank,))[0]
                 sink = f"l{i}.mix.sink" in tensor_shapes
-            self.layers.append(HybridLayer(cfg, spec, rank, sink, **f))
-        self.final_norm = _empty(cfg.hidden_size, device=device, dtype=torch.float32)
-        self.lm_head = Linear(cfg.hidden_size, cfg.vocab_size, **f)
+            self.layers.append(HybridLayer(cfg, spec, rank, sink, device=device, dtype=dtype))
         start, stop, times = cfg.loop
-        # layer number of every layer run; each run has a cache of its own
         self.runs = [*range(start), *(list(range(start, stop)) * times), *range(stop, len(cfg.layers))]
-        # bf16 products accumulate in fp32 to the end, fp32 products are true fp32
-        torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
-        if dtype == torch.float32:
-            torch.backends.cuda.matmul.allow_tf32 = False
 
-    # ---- weights ------------------------------------------------------------------------------------------
-    def checkpoint_slots(self) -> dict:
-        """Checkpoint tensor name -> the parameter (or slice of a fused one) that holds it."""
-        out = {"embed": self.embed, "final.norm": self.final_norm, "head": self.lm_head.weight}
-        for i, layer in enumerate(self.layers):
-            out.update({f"l{i}.{k}": v for k, v in layer.checkpoint_slots().items()})
-        return out
+    def init_constant(self, name: str):
+        """Norms 1, streams that pass through (identity mix, mean in, unit out), mild decays."""
+        leaf, S = name.rsplit(".", 1)[-1], self.config.streams
+        if "norm" in leaf or leaf == "out":
+            return 1.0
+        if leaf == "in":
+            return 1.0 / S
+        if name.endswith((".hc1.mix", ".hc2.mix")):
+            return torch.eye(S)
+        return 1.0 if leaf in ("sink", "b") else None
 
-    def _zero_padding(self):
-        for layer in self.layers:
-            if isinstance(layer.mixer, GatedLinearAttention):
-                layer.mixer.proj.weight[sum(layer.mixer.sizes):].zero_()
-
-    @torch.no_grad()
-    def load_tensors(self, tensors: dict):
-        """Fills the model from checkpoint tensors; a missing, unknown or misshapen one is an error."""
-        slots = self.checkpoint_slots()
-        missing, unknown = sorted(set(slots) - set(tensors)), sorted(set(tensors) - set(slots))
-        if missing or unknown:
-            raise ValueError(f"checkpoint does not fit the configuration: missing {missing}, unknown {unknown}")
-        for name, dst in slots.items():
-            src = tensors[name]
-            if tuple(src.shape) != tuple(dst.shape):
-                raise ValueError(f"{name}: shape {tuple(src.shape)}, expected {tuple(dst.shape)}")
-            dst.copy_(src)
-        self._zero_padding()
-        return self
-
-    @torch.no_grad()
-    def init_random(self, seed: int = 0, std: float = 0.02):
-        """Random weights from seeds derived from tensor names: N(0, std) matrices, norms 1, streams that pass
-        through (identity mix, mean in, unit out), mild decays."""
-        gen = torch.Generator(device=self.embed.device)
-        S = self.config.streams
-        for name, dst in self.checkpoint_slots().items():
-            leaf = name.rsplit(".", 1)[-1]
-            if "norm" in leaf or leaf == "out":
-                dst.fill_(1.0)
-            elif leaf == "in":
-                dst.fill_(1.0 / S)
-            elif name.endswith((".hc1.mix", ".hc2.mix")):
-                dst.copy_(torch.eye(S))
-            elif leaf in ("sink", "b"):
-                dst.fill_(1.0)
-            else:
-                gen.manual_seed((seed * 1000003 + _stable_hash(name)) % (2 ** 63))
-                dst.copy_(_randn_big(tuple(dst.shape), gen, dst.device, std, dst.dtype))
-        self._zero_padding()
-        return self
-
-    # ---- caches -------------------------------------------------------------------------------------------
-    def allocate_cache(self, batch_size: int, max_seqlen: int, device) -> dict:
-        """Per layer run: the window's K/V rings or the recurrent state. Nothing needs clearing between requests: a
-        sequence that starts at position 0 reads neither."""
-        return {r: self.layers[i].mixer.new_cache(batch_size, max_seqlen, device, self.dtype)
-                for r, i in enumerate(self.runs)}
-
-    def reset_decode_state(self, prompt_len: int, device, max_seqlen: int, batch: int = 1):
-        """All decode state is in the caches and in the positions."""
-
-    # ---- forward ------------------------------------------------------------------------------------------
-    def forward(self, input_ids, position_ids=None, inference_params=None, logit_rows=None, collect=None):
-        """input_ids (B, n): the next n tokens of every sequence; the caches of `inference_params` hold what came
-        before. position_ids (B, n) or (B, 1): only the first column is read; without it the position is the caches'
-        offset. logit_rows: places among the n tokens whose logits are wanted (default all). collect: a list that
-        receives the sum of the streams after every layer run (for inspection). -> logits (B, len(logit_rows), vocab)
-        fp32."""
-        cfg = self.config
-        B, n = input_ids.shape
-        dev = input_ids.device
-        if inference_params is None:
-            inference_params = InferenceParams(max_sequence_len=n, max_batch_size=B,
-                                               key_value_memory_dict=self.allocate_cache(B, n, dev))
-        if position_ids is None:
-            pos = torch.full((B,), inference_params.sequence_len_offset, dtype=torch.int64, device=dev)
-        else:
-            pos = position_ids[:, 0].contiguous()
-        caches = inference_params.key_value_memory_dict
-        ids = input_ids.reshape(-1).contiguous()
+    def hidden(self, ids, caches, pos, n, past, rows, collect):
+        cfg, dev = self.config, ids.device
         S, eps = cfg.streams, cfg.eps
         first = {"ids": ids, "embed": self.embed, "streams": S}
         x = None  # the streams; while None they are all the embedding
-        new_x = torch.empty(B * n, S, cfg.hidden_size, dtype=torch.float32, device=dev)
+        new_x = torch.empty(ids.numel(), S, cfg.hidden_size, dtype=torch.float32, device=dev)
         y, hc = None, None  # the last sublayer's output and its hyper-connection
 
         def boundary(w_in, gamma, rows=None, keep=True):
@@ -215,7 +131,7 @@ class NinolornForCausalLM(nn.Module, GenerationMixin):
         for r, i in enumerate(self.runs):
             layer = self.layers[i]
             h = boundary(layer.hc1.w_in, layer.norm1)
-            y, hc = layer.mixer(h, caches[r], pos, n), layer.hc1
+            y, hc = layer.mixer(h, caches[r], pos, n, past), layer.hc1
             if layer.mlp is not None:
                 h = boundary(layer.hc2.w_in, layer.norm2)
                 y, hc = layer.mlp(h, n), layer.hc2
@@ -223,18 +139,11 @@ class NinolornForCausalLM(nn.Module, GenerationMixin):
                 boundary(None, None)
                 y = None
                 collect.append(x.sum(dim=1))
-        if logit_rows is None or list(logit_rows) == list(range(n)):
-            rows, R = None, n
-        else:
-            R = len(logit_rows)
-            rows = torch.tensor([b * n + t for b in range(B) for t in logit_rows], dtype=torch.int32, device=dev)
-        if R == 0:
-            return CausalLMOutput(logits=torch.empty(B, 0, cfg.vocab_size, device=dev))
-        h = boundary(None, self.final_norm, rows, keep=False)
-        if n == 1 and B <= 32:
-            logits = self.lm_head.decode(h, torch.float32, "softcap" if cfg.softcap else "id", cfg.softcap or 0.0)
-        else:
-            logits = self.lm_head(h, torch.float32)
-            if cfg.softcap:
-                ops.softcap_(logits, cfg.softcap)
-        return CausalLMOutput(logits=logits.view(B, R, cfg.vocab_size))
+        return boundary(None, self.final_norm, rows, keep=False)
+
+    def head(self, h, decode: bool):
+        cap = self.config.softcap
+        if decode and h.shape[0] <= _lib.MAX_BATCH:
+            return self.lm_head.decode(h, torch.float32, "softcap" if cap else "id", cap or 0.0)
+        logits = self.lm_head(h, torch.float32)
+        return ops.softcap_(logits, cap) if cap else logits

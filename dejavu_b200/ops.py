@@ -518,7 +518,8 @@ def hyper_step(x, y, mix, w_out, w_in, gamma, eps: float, dtype, *, x_out=None, 
 def linear_gemv(x: torch.Tensor, weight: torch.Tensor, out_dtype=None, activation: str = "id",
                 param: float = 0.0) -> torch.Tensor:
     """y = activation(x @ weight.T) for a few rows of x (decode), bf16 or fp32 weights, result in their type or fp32.
-    activation "softcap" (param * tanh(v / param)) or "clamped_glu" (weight rows 2i, 2i+1 are gate and up of output i)."""
+    activation "softcap" (param * tanh(v / param)), "clamped_glu" or "silu_glu" (weight rows 2i, 2i+1 are gate and up of
+    output i)."""
     M, N = weight.shape
     B = x.shape[0]
     assert x.shape == (B, N) and 1 <= B <= _lib.MAX_BATCH and x.dtype == weight.dtype
@@ -526,19 +527,20 @@ def linear_gemv(x: torch.Tensor, weight: torch.Tensor, out_dtype=None, activatio
     _require_cuda(x, weight)
     x = x.contiguous()
     out_dtype = out_dtype or x.dtype
-    y = torch.empty(B, M // 2 if activation == "clamped_glu" else M, dtype=out_dtype, device=x.device)
+    y = torch.empty(B, M // 2 if activation.endswith("_glu") else M, dtype=out_dtype, device=x.device)
     call("djv_dense_gemv", _dtype_code(x), _dtype_code(y), y.data_ptr(), weight.data_ptr(), x.data_ptr(), B, N, M,
          weight.stride(0), _lib.ACT[activation], float(param), _stream())
     return y
 
 
-def clamped_glu(gu: torch.Tensor, limit: float) -> torch.Tensor:
-    """(R, 2F) with gate and up interleaved -> (R, F): min(g, limit) * sigmoid(1.702 .) * (clamp(u) + 1)."""
+def glu(gu: torch.Tensor, activation: str, param: float = 0.0) -> torch.Tensor:
+    """(R, 2F) with gate and up interleaved -> (R, F). "clamped_glu": min(g, param) * sigmoid(1.702 .) * (clamp(u, param)
+    + 1); "silu_glu": g * sigmoid(g) * u."""
     R, F2 = gu.shape
     _require_cuda(gu)
     assert gu.is_contiguous()
     y = torch.empty(R, F2 // 2, dtype=gu.dtype, device=gu.device)
-    call("djv_clamped_glu", _dtype_code(gu), y.data_ptr(), gu.data_ptr(), R, F2 // 2, float(limit), _stream())
+    call("djv_glu", _dtype_code(gu), y.data_ptr(), gu.data_ptr(), R, F2 // 2, _lib.ACT[activation], float(param), _stream())
     return y
 
 
@@ -549,13 +551,14 @@ def softcap_(y: torch.Tensor, cap: float) -> torch.Tensor:
     return y
 
 
-def rotary_(buf: torch.Tensor, freqs: torch.Tensor, amp: float, pos: torch.Tensor, n: int, heads: int, dim: int):
-    """Rotates the first `heads` heads of `dim` elements of every row of buf (B*n, ld) in place; pos (B,) int64 is the
-    position of each sequence's first row."""
+def rotary_(buf: torch.Tensor, freqs: torch.Tensor, amp: float, pos: torch.Tensor, n: int, heads: int, dim: int,
+            interleaved: bool = False):
+    """Rotates the first `heads` heads, `dim` elements apart, of every row of buf (B*n, ld) in place; pos (B,) int64 is the
+    position of each sequence's first row. Pairs (i, i + half), or (2i, 2i + 1) if interleaved."""
     _require_cuda(buf, freqs, pos)
     assert buf.stride(1) == 1 and pos.dtype == torch.int64 and buf.shape[0] == pos.numel() * n
     call("djv_rotary", _dtype_code(buf), buf.data_ptr(), buf.stride(0), freqs.data_ptr(), float(amp), pos.data_ptr(),
-         pos.numel(), n, heads, dim, freqs.numel(), _stream())
+         pos.numel(), n, heads, dim, freqs.numel(), int(interleaved), _stream())
 
 
 def _window_shapes(qkv, k_ring, v_ring, pos, n, heads):
@@ -614,3 +617,179 @@ def gated_linear_attention(proj, a2, a2_bias, tau: float, norm, eps: float, scal
         scratch = torch.empty(max(need, 256), dtype=torch.uint8, device=proj.device)
         call("djv_gla_prefill", *args, n, H, dk, dv, scratch.data_ptr(), scratch.numel(), _stream())
     return out
+
+
+# ---- routed decoders: matrix memories, latent attention, routed feed-forwards (bf16 or fp32) --------------------------
+
+def residual_step(x, y, gamma_y, gamma, eps: float, dtype, *, base: float = 0.0, x_out=None, parts=None, part_rows=None,
+                  rows=None, ids=None, embed=None):
+    """Boundary between two sublayers of a decoder with one residual and norms on both sides (djv_residual_step):
+        s = y + sum of the row's parts;  new = x + norm(s; base + gamma_y);  h = norm(new; base + gamma)
+    x (rows, D) fp32, or None: embed[ids]. y None: 0. parts (any, D) of `dtype` with part_rows (rows, k) int32. gamma_y
+    None: no norm of s. gamma None: only the update. x_out (may be x) receives new. rows (int32) selects rows. Returns
+    h (R, D) in `dtype`."""
+    src = x if x is not None else ids
+    _require_cuda(src, y, embed, parts)
+    _f32(x, y, gamma_y, gamma, x_out)
+    if x is not None:
+        n, D = x.shape
+    else:
+        n, D = ids.numel(), embed.shape[1]
+        assert ids.dtype == torch.int64 and ids.is_contiguous() and embed.is_contiguous() and embed.dtype == dtype
+    if parts is not None:
+        assert parts.is_contiguous() and parts.dtype == dtype and parts.shape[1] == D
+        assert part_rows.shape[0] == n and part_rows.dtype == torch.int32 and part_rows.is_contiguous()
+    R = n if rows is None else rows.numel()
+    h = None if gamma is None else torch.empty(R, D, dtype=dtype, device=src.device)
+    code = _lib.DTYPE_BF16 if dtype == torch.bfloat16 else _lib.DTYPE_F32
+    call("djv_residual_step", code, _ptr(h), _ptr(x_out), _ptr(x), _ptr(y), _ptr(parts),
+         None if parts is None else part_rows.data_ptr(), 0 if parts is None else part_rows.shape[1], _ptr(gamma_y),
+         _ptr(gamma), float(base), float(eps), _ptr(rows), None if x is not None else ids.data_ptr(),
+         None if x is not None else embed.data_ptr(), R, D, 0 if x is not None else embed.shape[0], _stream())
+    return h
+
+
+def mlstm_state(batch: int, heads: int, dk: int, dv: int, device) -> torch.Tensor:
+    """State of a matrix memory: S (dk, dv), n (dk) and m of every head, one fp32 row each."""
+    return torch.zeros(batch, heads, _lib.load_routed().djv_mlstm_state_floats(dk, dv), dtype=torch.float32, device=device)
+
+
+def mlstm(proj, gates, bias_i, bias_f, cap: float, norm, eps: float, scale: float, state, pos, n: int, dk: int, dv: int,
+          dtype):
+    """proj (B*n, q | k | v | output gate), gates (B*n, input | forget) fp32 -> (B*n, H*dv) of `dtype`, normed and gated;
+    state (B, H, ...) is advanced in place (a sequence at position 0 starts from zero). n == 1: a decode step, proj is
+    fp32; else proj is of `dtype`."""
+    H, b = state.shape[1], pos.numel()
+    assert proj.shape[0] == gates.shape[0] == b * n and proj.stride(1) == 1 and gates.stride(1) == 1
+    assert proj.shape[1] >= 2 * H * (dk + dv) and gates.shape[1] >= 2 * H and gates.dtype == torch.float32
+    assert proj.dtype == (torch.float32 if n == 1 else dtype) and b <= state.shape[0] and pos.dtype == torch.int64
+    _require_cuda(proj, gates, state, pos)
+    _f32(bias_i, bias_f, norm, state)
+    out = torch.empty(b * n, H * dv, dtype=dtype, device=proj.device)
+    code = _dtype_code(out)
+    args = (code, out.data_ptr(), proj.data_ptr(), proj.stride(0), gates.data_ptr(), gates.stride(0), bias_i.data_ptr(),
+            bias_f.data_ptr(), float(cap), norm.data_ptr(), float(eps), float(scale), state.data_ptr(), pos.data_ptr(), b)
+    if n == 1:
+        call("djv_mlstm_decode", *args, H, dk, dv, _stream())
+    else:
+        need = _lib.load_routed().djv_mlstm_scratch_bytes(code, b, n, H, dk, dv)
+        scratch = torch.empty(max(need, 256), dtype=torch.uint8, device=proj.device)
+        call("djv_mlstm_prefill", *args, n, H, dk, dv, scratch.data_ptr(), scratch.numel(), _stream())
+    return out
+
+
+def latent_rows(proj, ring, norm, eps: float, freqs, pos, n: int, past: int, rank: int):
+    """Cache rows (latent | shared key part) of `past` earlier tokens per sequence, from the ring, and of n new ones, from
+    proj (B*n, rank + rot), a view with any row stride: (B * (past + n), rank + rot)."""
+    B, cap, width = ring.shape
+    b = pos.numel()
+    assert b <= B and proj.shape == (b * n, width) and proj.stride(1) == 1 and proj.dtype == ring.dtype
+    assert ring.is_contiguous() and 0 <= past <= cap and pos.dtype == torch.int64 and freqs.numel() * 2 == width - rank
+    _require_cuda(proj, ring, pos)
+    _f32(norm, freqs)
+    rows = torch.empty(b * (past + n), width, dtype=ring.dtype, device=ring.device)
+    call("djv_latent_rows", _dtype_code(ring), rows.data_ptr(), proj.data_ptr(), proj.stride(0), ring.data_ptr(),
+         norm.data_ptr(), float(eps), freqs.data_ptr(), pos.data_ptr(), b, n, past, rank, width - rank, cap, 0, _stream())
+    return rows
+
+
+def latent_store(rows, ring, norm, freqs, pos, n: int, past: int, rank: int):
+    """The new rows of latent_rows enter the ring; afterwards, because they may take the slots of earlier ones."""
+    cap, width = ring.shape[1:]
+    call("djv_latent_rows", _dtype_code(ring), rows.data_ptr(), rows.data_ptr(), width, ring.data_ptr(), norm.data_ptr(),
+         0.0, freqs.data_ptr(), pos.data_ptr(), pos.numel(), n, past, rank, width - rank, cap, 1, _stream())
+
+
+def latent_attention(q, kv, tail, gate, pos, n: int, past: int, heads: int, dim: int, rot: int, window: int, scale: float):
+    """n new tokens per sequence over `past` earlier ones and themselves. q (B*n, H*(dim+rot)) rotated, kv
+    (B*(past+n), H*dim | H*dv), tail (B*(past+n), rot) and gate (B*n, H*dv) or None: views with any row stride. Returns
+    (B*n, H*dv), times sigmoid(gate)."""
+    b = pos.numel()
+    dv = kv.shape[1] // heads - dim
+    assert q.shape == (b * n, heads * (dim + rot)) and kv.shape == (b * (past + n), heads * (dim + dv))
+    assert tail.shape == (b * (past + n), rot) and (gate is None or gate.shape == (b * n, heads * dv))
+    assert q.dtype == kv.dtype == tail.dtype and pos.dtype == torch.int64
+    assert all(t is None or t.stride(1) == 1 for t in (q, kv, tail, gate))
+    _require_cuda(q, kv, tail, gate, pos)
+    out = torch.empty(b * n, heads * dv, dtype=q.dtype, device=q.device)
+    call("djv_latent_attn", _dtype_code(q), out.data_ptr(), q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0),
+         tail.data_ptr(), tail.stride(0), _ptr(gate), 0 if gate is None else gate.stride(0), pos.data_ptr(), b, n, past,
+         heads, dim, rot, dv, window, float(scale), _stream())
+    return out
+
+
+def latent_attention_decode(proj, uk, uv, norm, eps: float, freqs, ring, gate, pos, heads: int, window: int, scale: float,
+                            stages: int = 7, scratch=None):
+    """One token per sequence on the ring itself: proj (B, q | latent | key part, ...) neither normed nor rotated, uk
+    (H*dim, rank), uv (H*dv, rank), gate (B, H*dv) or None. Returns (B, H*dv). stages (1 queries and cache row, 2
+    attention, 4 values) and scratch (qc, ctx) are for timing the kernels one by one."""
+    B, cap, width = ring.shape
+    b, rank = pos.numel(), uk.shape[1]
+    dim, dv, rot = uk.shape[0] // heads, uv.shape[0] // heads, width - rank
+    assert b <= B and proj.shape[0] == b and proj.shape[1] >= heads * (dim + rot) + width and proj.stride(1) == 1
+    assert uk.is_contiguous() and uv.is_contiguous() and uv.shape[1] == rank and freqs.numel() * 2 == rot
+    assert proj.dtype == ring.dtype == uk.dtype == uv.dtype and pos.dtype == torch.int64
+    _require_cuda(proj, uk, uv, ring, pos, gate)
+    _f32(norm, freqs)
+    dev = ring.device
+    qc, ctx = scratch or (torch.empty(b, heads, width, dtype=ring.dtype, device=dev),
+                          torch.empty(b, heads, rank, dtype=torch.float32, device=dev))
+    out = torch.empty(b, heads * dv, dtype=ring.dtype, device=dev)
+    call("djv_latent_decode", _dtype_code(ring), out.data_ptr(), qc.data_ptr(), ctx.data_ptr(), proj.data_ptr(),
+         proj.stride(0), uk.data_ptr(), uv.data_ptr(), norm.data_ptr(), float(eps), freqs.data_ptr(), ring.data_ptr(),
+         _ptr(gate), 0 if gate is None else gate.stride(0), pos.data_ptr(), b, heads, dim, rot, dv, rank, cap, window,
+         float(scale), stages, _stream())
+    return out
+
+
+def moe_route(x, z, top: int):
+    """Sorts the choices of n tokens (router logits z (n, E) fp32) by expert. Returns (xs (n*top, D), ws (n*top,) fp32,
+    offsets (E+1,) int32, place (n, top) int32: the row of each choice)."""
+    n, E = z.shape
+    D, dev = x.shape[1], x.device
+    assert x.shape[0] == n and x.is_contiguous()
+    _require_cuda(x, z)
+    _f32(z)
+    i32 = {"dtype": torch.int32, "device": dev}
+    xs = torch.empty(n * top, D, dtype=x.dtype, device=dev)
+    expert, place, count, offsets = torch.empty(n, top, **i32), torch.empty(n, top, **i32), torch.empty(E, **i32), torch.empty(E + 1, **i32)
+    weight, ws = torch.empty(n, top, device=dev), torch.empty(n * top, device=dev)
+    call("djv_moe_route", _dtype_code(x), xs.data_ptr(), x.data_ptr(), z.data_ptr(), expert.data_ptr(), place.data_ptr(),
+         weight.data_ptr(), ws.data_ptr(), count.data_ptr(), offsets.data_ptr(), n, E, top, D, _stream())
+    return xs, ws, offsets, place
+
+
+def moe_grouped(x, w, offsets, scale=None, glu: bool = False):
+    """Rows offsets[e] .. offsets[e+1]-1 of x (R, K), times scale (R,), by w[e] (E, N, K): (R, N), or the gated units
+    (R, N/2) of interleaved gate and up rows."""
+    R, K = x.shape
+    E, N, _ = w.shape
+    assert w.shape[2] == K and x.is_contiguous() and w.is_contiguous() and x.dtype == w.dtype
+    assert offsets.dtype == torch.int32 and offsets.numel() == E + 1
+    _require_cuda(x, w, offsets)
+    _f32(scale)
+    y = torch.empty(R, N // 2 if glu else N, dtype=x.dtype, device=x.device)
+    call("djv_moe_grouped", _dtype_code(x), y.data_ptr(), x.data_ptr(), w.data_ptr(), _ptr(scale), offsets.data_ptr(), R, E,
+         N, K, int(glu), _stream())
+    return y
+
+
+def moe_decode(x, z, w_gu, w_down, top: int, shared_gu=None, shared_down=None, init=None, stages: int = 3, scratch=None):
+    """Routed feed-forward of B rows: x (B, D), router logits z (B, E) fp32, w_gu (E, 2F, D), w_down (E, D, F), optionally a
+    shared expert (2F', D), (D, F') and a summand init (B, D) fp32. Returns (B, D) fp32. stages (1 gated units, 2 down
+    products) and scratch (act, chosen) are for timing the kernels one by one."""
+    B, D = x.shape
+    E, F = w_gu.shape[0], w_gu.shape[1] // 2
+    Fs = 0 if shared_gu is None else shared_gu.shape[0] // 2
+    assert z.shape == (B, E) and w_gu.shape == (E, 2 * F, D) and w_down.shape == (E, D, F)
+    assert all(t is None or (t.is_contiguous() and t.dtype == x.dtype) for t in (x, w_gu, w_down, shared_gu, shared_down))
+    _require_cuda(x, z, w_gu, w_down, shared_gu, shared_down, init)
+    _f32(z, init)
+    ld = -(-max(F, Fs) // 8) * 8
+    act, chosen = scratch or (torch.empty(B, top + (Fs > 0), ld, dtype=x.dtype, device=x.device),
+                              torch.empty(B, top, dtype=torch.int32, device=x.device))
+    y = torch.empty(B, D, dtype=torch.float32, device=x.device)
+    call("djv_moe_decode", _dtype_code(x), y.data_ptr(), act.data_ptr(), chosen.data_ptr(), x.data_ptr(), z.data_ptr(),
+         w_gu.data_ptr(), w_down.data_ptr(), _ptr(shared_gu), _ptr(shared_down), _ptr(init), B, E, top, D, F, Fs, ld, stages,
+         _stream())
+    return y

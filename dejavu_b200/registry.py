@@ -30,6 +30,12 @@ def _build_ninolorn(raw, tensors, device, dtype):
     return NinolornForCausalLM(raw, shapes, device=device, dtype=dtype).load_tensors(tensors)
 
 
+def _build_tifosun(raw, tensors, device, dtype):
+    from .tifosun import TifosunForCausalLM
+
+    return TifosunForCausalLM(raw, device=device, dtype=dtype).load_tensors(tensors)
+
+
 def opt_config_from_json(raw):
     """Hugging Face OPT config.json -> this package's OPT configuration (dense: every head and neuron)."""
     from .gpt import opt_config
@@ -57,6 +63,7 @@ def _build_opt(raw, tensors, device, dtype):
 
 MODELS = {
     "Ninolorn": Entry(_build_ninolorn, (torch.bfloat16, torch.float32), "hybrid"),
+    "Tifosun": Entry(_build_tifosun, (torch.bfloat16, torch.float32), "routed"),
     "OPTForCausalLM": Entry(_build_opt, (torch.float16,), "sparse"),
 }
 

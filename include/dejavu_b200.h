@@ -40,6 +40,7 @@ extern "C" {
 #define DJV_ACT_SOFTCAP 5     /* c * tanh(v / c)                                                          */
 #define DJV_ACT_CLAMPED_GLU 6 /* rows 2i, 2i+1 = gate, up: g = min(gate, c), u = clamp(up, -c, c),        */
                               /* g * sigmoid(1.702 g) * (u + 1)                                           */
+#define DJV_ACT_SILU_GLU 7    /* rows 2i, 2i+1 = gate, up: g * sigmoid(g) * u (no constant)               */
 
 /* element types of the entry points that are compiled for several */
 #define DJV_DTYPE_F16 0

@@ -1,6 +1,8 @@
 /*
  * dejavu_b200_hybrid.h — C ABI of the kernels for decoders that mix gated linear attention, sliding-window attention
- * with sinks, clamped gated MLPs and hyper-connected residual streams (libdejavu_b200_hybrid.so).
+ * with sinks, gated MLPs and hyper-connected residual streams (libdejavu_b200_hybrid.so).
+ *
+ * Functions marked (both) are also in libdejavu_b200_routed.so (dejavu_b200_routed.h).
  *
  * Same conventions as dejavu_b200.h: raw device pointers, sizes, a CUDA stream as void*; work is only enqueued, never
  * allocated; DJV_OK or a negative DJV_ERR_* with a message in djv_last_error() (each library has its own). `dtype` is
@@ -20,7 +22,7 @@
 extern "C" {
 #endif
 
-/* One boundary between sublayers of a decoder whose residual is S parallel streams (1 <= S <= 8), in one pass:
+/* (both) One boundary between sublayers of a decoder whose residual is S parallel streams (1 <= S <= 8), in one pass:
  *   new_t = sum_s mix[s*S + t] * x_s + w_out[t] * y        (y = NULL: new = x)
  *   u     = sum_t w_in[t] * new_t                          (w_in = NULL: plain sum)
  *   h     = u / sqrt(mean(u^2) + eps) * gamma              (gamma = NULL: h is not written)
@@ -31,21 +33,33 @@ int djv_hyper_step(int dtype, void *h, float *x_out, const float *x_in, const fl
                    const float *w_out, const float *w_in, const float *gamma, float eps, const int32_t *row_list,
                    const long long *ids, const void *embed, int R, int S, int D, int vocab, void *stream);
 
-/* y[b, m] = act(w[m, :] . x[b, :]) for B <= DJV_MAX_BATCH rows of x: the decode step's matrix products. out_dtype: T or
- * DJV_DTYPE_F32. act: DJV_ACT_ID, DJV_ACT_SOFTCAP, DJV_ACT_CLAMPED_GLU (y then has M/2 columns). */
+/* (both) The boundary of a decoder with one residual and norms on both sides of a sublayer, in one pass:
+ *   s = y + sum_k parts[part_rows[row * n_parts + k]]      (y = NULL: 0; parts = NULL: none)
+ *   new = x + s / sqrt(mean(s^2) + eps) * (base + gamma_y) (gamma_y = NULL: new = x + s)
+ *   h = new / sqrt(mean(new^2) + eps) * (base + gamma)     (gamma = NULL: h is not written)
+ * parts: rows of D elements of T, part_rows (rows, n_parts) int32. The rest as in djv_hyper_step with S = 1. */
+int djv_residual_step(int dtype, void *h, float *x_out, const float *x_in, const float *y, const void *parts,
+                      const int32_t *part_rows, int n_parts, const float *gamma_y, const float *gamma, float base,
+                      float eps, const int32_t *row_list, const long long *ids, const void *embed, int R, int D,
+                      int vocab, void *stream);
+
+/* (both) y[b, m] = act(w[m, :] . x[b, :]) for B <= DJV_MAX_BATCH rows of x: the decode step's matrix products. out_dtype:
+ * T or DJV_DTYPE_F32. act: DJV_ACT_ID, DJV_ACT_SOFTCAP, DJV_ACT_CLAMPED_GLU, DJV_ACT_SILU_GLU (gated units: y has M/2
+ * columns). */
 int djv_dense_gemv(int dtype, int out_dtype, void *y, const void *w, const void *x, int B, int N, int M,
                    long long ldw, int act, float act_param, void *stream);
 
-/* y (R, F) = clamped gated unit of gu (R, 2F), gate and up interleaved (see DJV_ACT_CLAMPED_GLU). */
-int djv_clamped_glu(int dtype, void *y, const void *gu, long long R, int F, float limit, void *stream);
+/* (both) y (R, F) = gated unit of gu (R, 2F), gate and up interleaved; act: DJV_ACT_CLAMPED_GLU or DJV_ACT_SILU_GLU. */
+int djv_glu(int dtype, void *y, const void *gu, long long R, int F, int act, float limit, void *stream);
 
-/* y <- cap * tanh(y / cap), fp32, in place */
+/* (both) y <- cap * tanh(y / cap), fp32, in place */
 int djv_softcap(float *y, long long n, float cap, void *stream);
 
-/* Rotary positions in place on the first `heads` heads (dim each) of every row of buf (B*n rows, ld elements apart):
- * dimension i < half is paired with i + half, angle = position * freqs[i], cos and sin times amp. */
+/* (both) Rotary positions in place on the first `heads` heads (dim elements apart) of every row of buf (B*n rows, ld
+ * elements apart): pair i < half is dimensions (i, i + half), or (2i, 2i + 1) if interleaved; angle = position * freqs[i],
+ * cos and sin times amp. */
 int djv_rotary(int dtype, void *buf, long long ld, const float *freqs, float amp, const long long *pos, int B, int n,
-               int heads, int dim, int half, void *stream);
+               int heads, int dim, int half, int interleaved, void *stream);
 
 /* Causal attention of n new tokens per sequence over themselves and the tokens the cache holds. qkv rows hold
  * q (H, dk) | k (G, dk) | v (G, dv), already rotated; H % G == 0. The caches are rings of `cap` tokens per
@@ -57,7 +71,7 @@ int djv_window_attn(int dtype, void *out, const void *qkv, long long ld, const v
                     int window, float scale, void *stream);
 int djv_window_store(int dtype, void *k_ring, void *v_ring, const void *qkv, long long ld, const long long *pos, int B,
                      int n, int H, int G, int dk, int dv, int cap, void *stream);
-/* Waits of the tensor-core kernels on their own products that ran out since load (0 in a healthy process; synchronises). */
+/* (both) Waits of the tensor-core kernels on their own products that ran out since load (0 in a healthy process; synchronises). */
 unsigned djv_window_timeouts(void);
 /* The decode step of the same in one kernel: rotates q and k of one token per sequence, stores k and v into the rings
  * and attends. qkv rows are not rotated yet; freqs NULL: no rotation. */

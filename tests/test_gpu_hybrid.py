@@ -104,7 +104,7 @@ def test_elementwise(dtype, R, F):
     from dejavu_b200 import ops
 
     gu = rnd(gen(F), R, 2 * F, dtype=dtype, scale=2.0)
-    close(ops.clamped_glu(dev(gu, dtype), 0.7), O.clamped_glu(gu[:, 0::2], gu[:, 1::2], 0.7), dtype, 1e-6 if dtype == torch.float32 else 5e-3)
+    close(ops.glu(dev(gu, dtype), "clamped_glu", 0.7), O.clamped_glu(gu[:, 0::2], gu[:, 1::2], 0.7), dtype, 1e-6 if dtype == torch.float32 else 5e-3)
     y = rnd(gen(R), R, F, scale=10.0)
     close(ops.softcap_(dev(y), 6.0), O.softcap(y, 6.0), torch.float32, 1e-6)
 
