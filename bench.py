@@ -16,7 +16,8 @@ uniform-random prompt) after a dense prompt pass. Prints one JSON line:
   cpu_baseline   the reference's torch formulation on the host cores (bounded sample, N=1 only)
 `--impl reference` times only that CPU formulation (all host threads) and prints it in the same format.
 `--hybrid 1b,7b` instead times the Ninolorn design beside the dense OPT decoder at those sizes (one GPU; see
-dejavu_b200/hybrid_bench.py) and prints one JSON line of its own.
+dejavu_b200/hybrid_bench.py) and prints one JSON line of its own; `--routed 1b,7b` does the same for the Tifosun design
+beside Ninolorn (dejavu_b200/routed_bench.py).
 """
 from __future__ import annotations
 
@@ -327,16 +328,17 @@ def run_reference(args, cfg, mlp_K, att_K, world, rank):
 
 
 def run_hybrid(args):
-    """Throughput and kernels of the hybrid design beside dense OPT, one JSON line."""
-    from dejavu_b200 import _lib, hybrid_bench
+    """Throughput and kernels of a hybrid design beside its comparator, one JSON line."""
+    from dejavu_b200 import _lib, hybrid_bench, routed_bench
 
-    _lib.load(), _lib.load_hybrid()  # fail loudly if a CUDA library is missing
+    _lib.load(), _lib.load_hybrid(), _lib.load_routed()  # fail loudly if a CUDA library is missing
+    bench, names = (hybrid_bench, args.hybrid) if args.hybrid else (routed_bench, args.routed)
     peak, kind = measured_peaks()
     p = ROOT / "MEASURED_PEAKS.json"
     tflops = float(json.loads(p.read_text())["bf16_tflops"]) if p.exists() else 1590.0
     with ClockSampler(0) as clocks:
-        res = hybrid_bench.run(args.hybrid.split(","), kernel_timing, peak, tflops, prompt=args.promptlen or 4096)
-    emit({"metric": "hybrid_decoder_throughput", "peak_gbs": peak, "peak_tflops": tflops, "peak_kind": kind,
+        res = bench.run(names.split(","), kernel_timing, peak, tflops, prompt=args.promptlen or 4096)
+    emit({"metric": f"{'hybrid' if args.hybrid else 'routed'}_decoder_throughput", "peak_gbs": peak, "peak_tflops": tflops, "peak_kind": kind,
           "data": "synthetic", "sizes": res, "clocks": clocks.summary()})
 
 
@@ -400,9 +402,10 @@ def main():
     ap.add_argument("--no-cpu", action="store_true")
     ap.add_argument("--fused-allreduce", type=int, default=1)
     ap.add_argument("--hybrid", default=None, help="comma-separated sizes (1b, 7b, 30b): time the hybrid design beside dense OPT")
+    ap.add_argument("--routed", default=None, help="comma-separated sizes (1b, 7b, 30b): time the routed design beside the hybrid one")
     args = ap.parse_args()
 
-    if args.hybrid:
+    if args.hybrid or args.routed:
         run_hybrid(args)
         return
     if args.model_name:

@@ -123,8 +123,9 @@ ROUTED_SIGNATURES = {
     "djv_latent_rows": (_i, [_i, _vp, _vp, _ll, _vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "djv_latent_attn": (_i, [_i, _vp, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f,
                              _vp]),
-    "djv_latent_decode": (_i, [_i, _vp, _vp, _vp, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _i,
-                               _i, _i, _i, _f, _i, _vp]),
+    "djv_latent_scratch_floats": (_sz, [_i, _i, _i, _i]),
+    "djv_latent_decode": (_i, [_i, _vp, _vp, _vp, _sz, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i,
+                               _i, _i, _i, _i, _f, _i, _vp]),
     "djv_moe_route": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp]),
     "djv_moe_grouped": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp]),
     "djv_moe_decode": (_i, [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]),

@@ -5,7 +5,6 @@
 // A portion of tokens expands the latents it can see into keys and values with one matrix product and runs the windowed
 // attention kernels on them. A decode step leaves the latents as they are: the key projection is applied to the query
 // and the value projection to the weighted sum of latents, so that every head reads the same rows.
-#include <cooperative_groups.h>
 #include <math.h>
 
 #include "../../include/dejavu_b200_routed.h"
@@ -13,6 +12,9 @@
 #include "hybrid_latent.cuh"
 
 namespace djv {
+
+// blocks among which the sequences of a decode step are dealt out, per block of weights
+constexpr int LATENT_GROUPS = 8;
 
 // one row: RMS norm of the latent, rotation of the shared key part, by a whole block
 template <typename T>
@@ -60,6 +62,64 @@ __global__ void latent_rows_kernel(T *__restrict__ rows, const T *__restrict__ s
   for (int i = threadIdx.x; i < w; i += blockDim.x) dst[i] = old ? old[i] : from_f<T>(0.f);
 }
 
+// the same with 16-byte accesses, a warp per row of at most LR_U * 32 latent chunks; with `store` (only where no earlier
+// rows are read) the new rows also enter the ring
+constexpr int LR_WARPS = 4, LR_U = 4;
+template <typename T>
+__global__ void __launch_bounds__(LR_WARPS * WARP)
+latent_rows_warp_kernel(T *__restrict__ rows, const T *__restrict__ src, long long ld, T *__restrict__ ring,
+                        const float *__restrict__ norm, float eps, const float *__restrict__ freqs,
+                        const long long *__restrict__ pos, int n, int past, int rank, int rot, int cap, int store) {
+  pdl_prologue();
+  constexpr int N = Chunk<T>::N;
+  const int lane = threadIdx.x % WARP, row = blockIdx.x * LR_WARPS + threadIdx.x / WARP, b = blockIdx.y;
+  if (row >= past + n) return;
+  const int j = row - past, w = rank + rot, nch = rank / N;
+  T *dst = rows + ((size_t)b * (past + n) + row) * w;
+  const long long p = pos[b] + j;
+  if (j < 0) {
+    const uint4 *old = p >= 0 ? reinterpret_cast<const uint4 *>(ring + ((size_t)b * cap + (size_t)(p % cap)) * w) : nullptr;
+    for (int c = lane; c < w / N; c += WARP) reinterpret_cast<uint4 *>(dst)[c] = old ? old[c] : make_uint4(0, 0, 0, 0);
+    return;
+  }
+  T *slot = store && j >= n - cap ? ring + ((size_t)b * cap + (size_t)(p % cap)) * w : nullptr;
+  const T *s = src + ((size_t)b * n + j) * ld;
+  float f[LR_U][N], ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < LR_U; ++u) {
+    const int c = lane + u * WARP;
+    const uint4 v = c < nch ? reinterpret_cast<const uint4 *>(s)[c] : make_uint4(0, 0, 0, 0);
+    unpack_chunk<T>(v, f[u]);
+  }
+#pragma unroll
+  for (int u = 0; u < LR_U; ++u)
+#pragma unroll
+    for (int e = 0; e < N; ++e) ss = fmaf(f[u][e], f[u][e], ss);
+  const float r = 1.f / sqrtf(warp_sum(ss) / (float)rank + eps);
+#pragma unroll
+  for (int u = 0; u < LR_U; ++u) {
+    const int c = lane + u * WARP;
+    if (c >= nch) continue;
+    T o[N];
+#pragma unroll
+    for (int e = 0; e < N; ++e) o[e] = from_f<T>(f[u][e] * r * norm[c * N + e]);
+    reinterpret_cast<uint4 *>(dst)[c] = *reinterpret_cast<uint4 *>(o);
+    if (slot) reinterpret_cast<uint4 *>(slot)[c] = *reinterpret_cast<uint4 *>(o);
+  }
+  for (int i = lane; i < rot / 2; i += WARP) {
+    float sn, cs;
+    sincosf((float)p * freqs[i], &sn, &cs);
+    const float u = to_f(s[rank + 2 * i]), v = to_f(s[rank + 2 * i + 1]);
+    const T x = from_f<T>(u * cs - v * sn), y = from_f<T>(v * cs + u * sn);
+    dst[rank + 2 * i] = x;
+    dst[rank + 2 * i + 1] = y;
+    if (slot) {
+      slot[rank + 2 * i] = x;
+      slot[rank + 2 * i + 1] = y;
+    }
+  }
+}
+
 // the new rows enter the ring (after latent_rows_kernel has read the old ones): the last min(n, cap) tokens
 template <typename T>
 __global__ void latent_store_kernel(T *__restrict__ ring, const T *__restrict__ rows, const long long *__restrict__ pos,
@@ -74,18 +134,20 @@ __global__ void latent_store_kernel(T *__restrict__ ring, const T *__restrict__ 
 // ---- decode: queries ------------------------------------------------------------------------------------------------
 // Blocks 0 .. H * cbs - 1: query of head h against columns of its key projection, for all sequences,
 //   out[b, h, r] = sum_d q[b, h, d] uk[h * dim + d, r];  the first column block of a head also rotates its query part.
-// The B blocks after them: a sequence's new latent row goes straight into its ring slot.
+// The blocks after them: a sequence's new latent row goes straight into its ring slot.
 // V columns per thread; with REG the weights (at most LQ_REG rows per thread) are fetched before the kernel waits for its
-// predecessor and stay in registers for all sequences.
+// predecessor and stay in registers for the block's `per` sequences.
 template <typename T, int V, bool REG>
-__global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(LatentDecodeArgs a, int cbs) {
+__global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(LatentDecodeArgs a, int cbs, int per) {
   extern __shared__ float sm[];
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   constexpr int CT = LQ_COLS / V, RG = LQ_THREADS / CT;  // threads along the columns, row groups
   const int tid = threadIdx.x, w = a.rank + a.rot, qd = a.dim + a.rot;
+  const int b0 = blockIdx.y * per, b1 = min(a.B, b0 + per);
   if ((int)blockIdx.x >= a.H * cbs) {
     asm volatile("griddepcontrol.wait;" ::: "memory");
-    const int b = blockIdx.x - a.H * cbs;
+    const int b = b0 + blockIdx.x - a.H * cbs;
+    if (b >= b1) return;
     const long long p = a.pos[b];
     make_latent_row<T>(static_cast<const T *>(a.proj) + (size_t)b * a.ld + (size_t)a.H * qd,
                        static_cast<T *>(a.ring) + ((size_t)b * a.cap + (size_t)(p % a.cap)) * w, a.norm, a.eps, a.freqs, p,
@@ -106,7 +168,7 @@ __global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(LatentDecodeAr
   }
   asm volatile("griddepcontrol.wait;" ::: "memory");
   float *q = sm, *red = q + ((a.dim + 3) & ~3);  // [RG][LQ_COLS]
-  for (int b = 0; b < a.B; ++b) {
+  for (int b = b0; b < b1; ++b) {
     const T *row = static_cast<const T *>(a.proj) + (size_t)b * a.ld + (size_t)h * qd;
     T *out = static_cast<T *>(a.qc) + ((size_t)b * a.H + h) * w;
     for (int i = tid; i < a.dim; i += LQ_THREADS) q[i] = to_f(row[i]);
@@ -211,23 +273,27 @@ __global__ void __launch_bounds__(LS_THREADS) latent_attend_simple_kernel(Latent
     }
     __syncthreads();
   }
-  float *out = a.ctx + ((size_t)b * a.H + h) * a.rank;
-  for (int i = tid; i < a.rank; i += LS_THREADS) out[i] = o[i] / l_run;
+  float *out = a.part_o + ((size_t)b * a.H + h) * a.splits * a.rank, *ml = a.part_ml + ((size_t)b * a.H + h) * a.splits * 2;
+  for (int i = tid; i < a.rank; i += LS_THREADS) out[i] = o[i];
+  for (int s = tid; s < a.splits; s += LS_THREADS) {  // one part has it all
+    ml[2 * s] = s ? -INFINITY : m_run;
+    ml[2 * s + 1] = s ? 0.f : l_run;
+  }
 }
 
 // ---- decode: values -------------------------------------------------------------------------------------------------
-// out[b, h, j] = (uv[h * dv + j, :] . ctx[b, h, :]) * sigmoid(gate[b, h, j]); a warp takes LO_ROWS rows of one head, all
-// of whose weights are fetched before the kernel waits (VEC; U 16-byte chunks per lane and row).
-constexpr int LO_THREADS = 256, LO_ROWS = 4;
+// out[b, h, j] = (uv[h * dv + j, :] . ctx[b, h, :]) * sigmoid(gate[b, h, j]), ctx the window's parts put together. A block
+// takes LO_ROWS rows per warp of one head and `per` sequences; the weights are fetched before the kernel waits (U 16-byte chunks per lane and
+// row).
+constexpr int LO_THREADS = 256, LO_WARPS = LO_THREADS / WARP, LO_ROWS = 4;
 template <typename T, int U>  // U == 0: any rank and alignment
-__global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(LatentDecodeArgs a) {
+__global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(LatentDecodeArgs a, int per) {
+  extern __shared__ __align__(16) float ctx[];  // rank
+  __shared__ float factor[LD_MAX_SPLITS];
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  const int lane = threadIdx.x % WARP, warp = threadIdx.x / WARP;
-  const int per = (a.dv + LO_ROWS - 1) / LO_ROWS, task = blockIdx.x * (LO_THREADS / WARP) + warp;
-  const bool any = task < a.H * per;
-  const int h = any ? task / per : 0, r0 = any ? task % per * LO_ROWS : 0;
+  const int tid = threadIdx.x, lane = tid % WARP, warp = tid / WARP, h = blockIdx.y;
+  const int r0 = (blockIdx.x * LO_WARPS + warp) * LO_ROWS, rows = max(0, min(LO_ROWS, a.dv - r0));
   const T *W = static_cast<const T *>(a.uv) + ((size_t)h * a.dv + r0) * a.rank;
-  const int rows = any ? min(LO_ROWS, a.dv - r0) : 0;
   constexpr int N = Chunk<T>::N;
   const int nch = a.rank / N;
   uint4 w[LO_ROWS][U > 0 ? U : 1];
@@ -241,8 +307,38 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(LatentDecodeArgs
       }
   }
   asm volatile("griddepcontrol.wait;" ::: "memory");
-  for (int b = 0; b < a.B; ++b) {
-    const float *x = a.ctx + ((size_t)b * a.H + h) * a.rank;
+  const int b1 = min(a.B, ((int)blockIdx.z + 1) * per);
+  for (int b = blockIdx.z * per; b < b1; ++b) {
+    const size_t bh = (size_t)b * a.H + h;
+    if (warp == 0) {  // (at most a part per lane)
+      const float m = lane < a.splits ? a.part_ml[(bh * a.splits + lane) * 2] : -INFINITY;
+      const float l = lane < a.splits ? a.part_ml[(bh * a.splits + lane) * 2 + 1] : 0.f;
+      const float top = warp_max(m), f = m == -INFINITY ? 0.f : expf(m - top);
+      factor[lane] = f / warp_sum(f * l);
+    }
+    __syncthreads();
+    const float *part = a.part_o + bh * a.splits * a.rank;
+    if (U > 0) {
+      for (int c = tid * 2; c < a.rank; c += LO_THREADS * 2) {
+        float2 o = make_float2(0.f, 0.f);
+#pragma unroll 16
+        for (int s = 0; s < a.splits; ++s) {
+          const float f = factor[s];  // (0: an empty part, whose sums may be anything)
+          const float2 v = f != 0.f ? *reinterpret_cast<const float2 *>(part + (size_t)s * a.rank + c) : make_float2(0.f, 0.f);
+          o.x = fmaf(f, v.x, o.x);
+          o.y = fmaf(f, v.y, o.y);
+        }
+        *reinterpret_cast<float2 *>(ctx + c) = o;
+      }
+    } else {
+      for (int c = tid; c < a.rank; c += LO_THREADS) {
+        float o = 0.f;
+        for (int s = 0; s < a.splits; ++s)
+          if (factor[s] != 0.f) o = fmaf(factor[s], part[(size_t)s * a.rank + c], o);
+        ctx[c] = o;
+      }
+    }
+    __syncthreads();
     float acc[LO_ROWS];
 #pragma unroll
     for (int r = 0; r < LO_ROWS; ++r) acc[r] = 0.f;
@@ -253,7 +349,7 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(LatentDecodeArgs
         if (c < nch) {
           float xv[N];
 #pragma unroll
-          for (int e = 0; e < N; e += 4) *reinterpret_cast<float4 *>(xv + e) = *reinterpret_cast<const float4 *>(x + c * N + e);
+          for (int e = 0; e < N; e += 4) *reinterpret_cast<float4 *>(xv + e) = *reinterpret_cast<const float4 *>(ctx + c * N + e);
 #pragma unroll
           for (int r = 0; r < LO_ROWS; ++r) {
             float f[N];
@@ -265,7 +361,7 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(LatentDecodeArgs
       }
     } else {
       for (int c = lane; c < a.rank; c += WARP)
-        for (int r = 0; r < rows; ++r) acc[r] = fmaf(to_f(W[(size_t)r * a.rank + c]), x[c], acc[r]);
+        for (int r = 0; r < rows; ++r) acc[r] = fmaf(to_f(W[(size_t)r * a.rank + c]), ctx[c], acc[r]);
     }
 #pragma unroll
     for (int r = 0; r < LO_ROWS; ++r) acc[r] = warp_sum(acc[r]);
@@ -278,6 +374,7 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(LatentDecodeArgs
       if (a.gate) v *= sigmoid_f(to_f(static_cast<const T *>(a.gate)[(size_t)b * a.ldg + col]));
       static_cast<T *>(a.out)[(size_t)b * a.H * a.dv + col] = from_f<T>(v);
     }
+    if (b + 1 < b1) __syncthreads();  // ctx is reused
   }
 }
 
@@ -286,12 +383,13 @@ static int launch_query(const LatentDecodeArgs &a, cudaStream_t st) {
   constexpr int N = Chunk<T>::N;
   const int cbs = ceil_div(a.rank, LQ_COLS);
   const bool vec = a.rank % N == 0 && aligned16(a.uk);
-  const dim3 grid(a.H * cbs + a.B);
+  const int per = ceil_div(a.B, LATENT_GROUPS);
+  const dim3 grid(a.H * cbs + per, ceil_div(a.B, per));
   auto smem = [&](int v) { return 4 * ((size_t)((a.dim + 3) & ~3) + (size_t)(LQ_THREADS / (LQ_COLS / v)) * LQ_COLS); };
   if (vec && a.dim <= LQ_REG * (LQ_THREADS / (LQ_COLS / N)))
-    djv::launch_kernel(latent_query_kernel<T, N, true>, grid, dim3(LQ_THREADS), smem(N), st, a, cbs);
+    djv::launch_kernel(latent_query_kernel<T, N, true>, grid, dim3(LQ_THREADS), smem(N), st, a, cbs, per);
   else
-    djv::launch_kernel(latent_query_kernel<T, 1, false>, grid, dim3(LQ_THREADS), smem(1), st, a, cbs);
+    djv::launch_kernel(latent_query_kernel<T, 1, false>, grid, dim3(LQ_THREADS), smem(1), st, a, cbs, per);
   count_launch();
   return check_launch("latent_decode");
 }
@@ -310,12 +408,14 @@ static int launch_attend(const LatentDecodeArgs &a, cudaStream_t st) {
 template <typename T>
 static int launch_out(const LatentDecodeArgs &a, cudaStream_t st) {
   constexpr int N = Chunk<T>::N;
-  const int tasks = a.H * ceil_div(a.dv, LO_ROWS), grid = ceil_div(tasks, LO_THREADS / WARP);
-  const int u = a.rank % N == 0 && aligned16(a.uv) ? ceil_div(a.rank / N, WARP) : 0;
-  if (u == 1) djv::launch_kernel(latent_out_kernel<T, 1>, dim3(grid), dim3(LO_THREADS), 0, st, a);
-  else if (u == 2) djv::launch_kernel(latent_out_kernel<T, 2>, dim3(grid), dim3(LO_THREADS), 0, st, a);
-  else if (u == 3 || u == 4) djv::launch_kernel(latent_out_kernel<T, 4>, dim3(grid), dim3(LO_THREADS), 0, st, a);
-  else djv::launch_kernel(latent_out_kernel<T, 0>, dim3(grid), dim3(LO_THREADS), 0, st, a);
+  const int per = ceil_div(a.B, LATENT_GROUPS);
+  const dim3 grid(ceil_div(a.dv, LO_WARPS * LO_ROWS), a.H, ceil_div(a.B, per));
+  const size_t smem = (size_t)a.rank * 4;
+  const int u = a.rank % N == 0 && aligned16(a.uv) && aligned16(a.part_o) ? ceil_div(a.rank / N, WARP) : 0;
+  if (u == 1) djv::launch_kernel(latent_out_kernel<T, 1>, grid, dim3(LO_THREADS), smem, st, a, per);
+  else if (u == 2) djv::launch_kernel(latent_out_kernel<T, 2>, grid, dim3(LO_THREADS), smem, st, a, per);
+  else if (u == 3 || u == 4) djv::launch_kernel(latent_out_kernel<T, 4>, grid, dim3(LO_THREADS), smem, st, a, per);
+  else djv::launch_kernel(latent_out_kernel<T, 0>, grid, dim3(LO_THREADS), smem, st, a, per);
   count_launch();
   return check_launch("latent_decode");
 }
@@ -339,23 +439,28 @@ extern "C" int djv_latent_rows(int dtype, void *rows, const void *proj, long lon
   if (rc) return rc;
   DJV_REQUIRE(rows && proj && ring && norm && pos && (freqs || rot == 0), "latent_rows: null pointer");
   DJV_REQUIRE(past >= 0 && past <= cap && ld >= rank + rot, "latent_rows: past=%d cap=%d row stride %lld", past, cap, ld);
-  const int cnt = n < cap ? n : cap;
+  DJV_REQUIRE(store >= 0 && store <= 2 && (store != 2 || past == 0), "latent_rows: store=%d past=%d", store, past);
+  const int cnt = n < cap ? n : cap, chunk = 16 / (int)dtype_bytes(dtype);
+  const bool vec = rank % chunk == 0 && rot % chunk == 0 && rank / chunk <= LR_U * WARP && ld % chunk == 0 &&
+                   aligned16(rows) && aligned16(proj) && aligned16(ring);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
 #define DJV_GO(T_)                                                                                                       \
-  if (!store)                                                                                                            \
-    djv::launch_kernel(latent_rows_kernel<T_>, dim3(past + n, B), dim3(128), 0, st, static_cast<T_ *>(rows),             \
-                       static_cast<const T_ *>(proj), ld, static_cast<const T_ *>(ring), norm, eps, freqs, pos, n, past, \
-                       rank, rot, cap);                                                                                  \
-  else                                                                                                                   \
-    djv::launch_kernel(latent_store_kernel<T_>, dim3(cnt, B), dim3(128), 0, st, static_cast<T_ *>(ring),                 \
-                       static_cast<const T_ *>(rows), pos, n, past, rank + rot, cap, n - cnt)
-  if (dtype == DJV_DTYPE_BF16) {
-    DJV_GO(bf16);
-  } else {
-    DJV_GO(float);
+  {                                                                                                                      \
+    T_ *r = static_cast<T_ *>(rows), *g = static_cast<T_ *>(ring);                                                       \
+    const T_ *p = static_cast<const T_ *>(proj);                                                                         \
+    if (store != 1 && vec)                                                                                               \
+      djv::launch_kernel(latent_rows_warp_kernel<T_>, dim3(ceil_div(past + n, LR_WARPS), B), dim3(LR_WARPS * WARP), 0,   \
+                         st, r, p, ld, g, norm, eps, freqs, pos, n, past, rank, rot, cap, store);                        \
+    else if (store != 1)                                                                                                 \
+      djv::launch_kernel(latent_rows_kernel<T_>, dim3(past + n, B), dim3(128), 0, st, r, p, ld, g, norm, eps, freqs,     \
+                         pos, n, past, rank, rot, cap);                                                                  \
+    if (store == 1 || (store == 2 && !vec))                                                                              \
+      djv::launch_kernel(latent_store_kernel<T_>, dim3(cnt, B), dim3(128), 0, st, g, r, pos, n, past, rank + rot, cap,   \
+                         n - cnt);                                                                                       \
   }
+  if (dtype == DJV_DTYPE_BF16) DJV_GO(bf16) else DJV_GO(float)
 #undef DJV_GO
-  count_launch();
+  count_launch(store == 2 && !vec ? 2 : 1);
   return check_launch("latent_rows");
 }
 
@@ -378,21 +483,32 @@ extern "C" int djv_latent_attn(int dtype, void *out, const void *q, long long ld
   return window_attn_portion(dtype, a, static_cast<cudaStream_t>(stream));
 }
 
-extern "C" int djv_latent_decode(int dtype, void *out, void *qc, float *ctx, const void *proj, long long ld, const void *uk,
-                                 const void *uv, const float *norm, float eps, const float *freqs, void *ring,
-                                 const void *gate, long long ldg, const long long *pos, int B, int H, int dim, int rot,
-                                 int dv, int rank, int cap, int window, float scale, int stages, void *stream) {
+extern "C" size_t djv_latent_scratch_floats(int B, int H, int rank, int window) {
+  if (B < 1 || H < 1 || rank < 1 || window < 1) return 0;
+  return (size_t)B * H * latent_splits(B, H, window) * (rank + 2);
+}
+
+extern "C" int djv_latent_decode(int dtype, void *out, void *qc, float *scratch, size_t scratch_floats, const void *proj,
+                                 long long ld, const void *uk, const void *uv, const float *norm, float eps,
+                                 const float *freqs, void *ring, const void *gate, long long ldg, const long long *pos,
+                                 int B, int H, int dim, int rot, int dv, int rank, int cap, int window, float scale,
+                                 int stages, void *stream) {
   int rc = check_latent("latent_decode", dtype, B, 1, rank, rot, cap);
   if (rc) return rc;
-  DJV_REQUIRE(out && qc && ctx && proj && uk && uv && norm && ring && pos && (freqs || rot == 0),
-              "latent_decode: null pointer");
+  DJV_REQUIRE(out && qc && proj && uk && uv && norm && ring && pos && (freqs || rot == 0), "latent_decode: null pointer");
   DJV_REQUIRE(H >= 1 && H <= 65535 && dim >= 1 && dim <= 1024 && dv >= 1 && window >= 1,
               "latent_decode: H=%d head sizes %d / %d window=%d", H, dim, dv, window);
   DJV_REQUIRE(ld >= (long long)H * (dim + rot) + rank + rot && (!gate || ldg >= (long long)H * dv),
               "latent_decode: a row stride is too small");
   if (window > cap) window = cap;  // a ring that is shorter than the window holds the longest sequence
-  const LatentDecodeArgs a{out, qc, ctx, proj, ld, uk, uv, norm, eps, freqs, ring, gate, ldg, pos, B, H, dim, rot, dv, rank,
-                           cap, window, scale};
+  const int splits = latent_splits(B, H, window);
+  const size_t sums = (size_t)B * H * splits * rank, need = sums + (size_t)B * H * splits * 2;
+  if (!scratch || scratch_floats < need) {
+    set_error("latent_decode: scratch needs %zu floats (got %zu)", need, scratch_floats);
+    return DJV_ERR_SCRATCH;
+  }
+  const LatentDecodeArgs a{out, qc, scratch, scratch + sums, proj, ld, uk, uv, norm, eps, freqs, ring, gate, ldg, pos, B, H,
+                           dim, rot, dv, rank, cap, window, splits, scale};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const bool b16 = dtype == DJV_DTYPE_BF16;
   if (stages & 1) rc = b16 ? launch_query<bf16>(a, st) : launch_query<float>(a, st);

@@ -1,13 +1,12 @@
 // Decode attention over latents on the tensor cores (bf16): all heads of a sequence read the same rows, so 16 heads at a
 // time are the rows of mma.sync tiles (a decode step has too few rows for the TMEM path's 128).
 //
-// A block takes 16 heads and a part of the window, 64 tokens per pass:
-//   scores: a warp per 8 tokens, over the whole row (latent and shared key part);
+// A block takes 16 heads and a part of the window, 32 tokens per pass:
+//   scores: a warp per 8 tokens and half of the row (latent and shared key part);
 //   weights: fp32 softmax, two heads per warp, kept as two bf16 terms (hi + lo);
 //   sums: a warp takes every 8th group of 16 latent columns of all heads.
-// The next pass's rows load while this one computes. The parts of a window are a cluster; each of its blocks combines a share
-// of the columns from all of them.
-#include <cooperative_groups.h>
+// In long parts the next pass's rows load while this one computes. The parts' sums are put together by the kernel that applies the value
+// projection.
 #include <math.h>
 
 #include "../../include/dejavu_b200_routed.h"
@@ -16,10 +15,8 @@
 
 namespace djv {
 
-namespace cg = cooperative_groups;
-
 constexpr int LM_THREADS = 256, LM_WARPS = LM_THREADS / WARP;
-constexpr int LM_HEADS = 16, LM_TILE = 64, LM_MAX_SPLITS = 8;
+constexpr int LM_HEADS = 16, LM_TILE = 32;
 constexpr int LM_PP = LM_TILE + 8;  // row pitch of the weights
 
 __host__ __device__ __forceinline__ int lm_pitch(int width) { return ((width + 15) & ~15) + 8; }
@@ -27,44 +24,44 @@ __host__ __device__ __forceinline__ int lm_pitch(int width) { return ((width + 1
 template <int NG>  // groups of 16 latent columns per warp
 __global__ void __launch_bounds__(LM_THREADS) latent_attend_mma_kernel(LatentDecodeArgs a, int nbuf) {
   extern __shared__ __align__(16) unsigned char sm_raw[];
-  __shared__ __align__(16) float sc[LM_HEADS][LM_TILE + 4], part_m[LM_MAX_SPLITS][LM_HEADS], part_l[LM_MAX_SPLITS][LM_HEADS];
-  __shared__ float m_run[LM_HEADS], l_run[LM_HEADS], corr[LM_HEADS];
+  __shared__ float sc[2][LM_HEADS][LM_TILE + 4], m_run[LM_HEADS], l_run[LM_HEADS], corr[LM_HEADS];
   __shared__ __align__(16) bf16 p_hi[LM_HEADS * LM_PP], p_lo[LM_HEADS * LM_PP];
-  cg::cluster_group cluster = cg::this_cluster();
-  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  const int nsplit = gridDim.z;
-  if (nsplit > 1) cluster.barrier_arrive();  // (waited for before the first access to another block's memory)
-  asm volatile("griddepcontrol.wait;" ::: "memory");
+  pdl_prologue();
   const int tid = threadIdx.x, lane = tid % WARP, warp = tid / WARP;
   const int h0 = blockIdx.x * LM_HEADS, nh = min(LM_HEADS, a.H - h0), b = blockIdx.y, sp = blockIdx.z;
   const int w = a.rank + a.rot, wp = (w + 15) & ~15, pitch = lm_pitch(w), nch = w / 8;
   bf16 *q = reinterpret_cast<bf16 *>(sm_raw), *tiles = q + LM_HEADS * pitch;
+  const bf16 *qr = static_cast<const bf16 *>(a.qc) + ((size_t)b * a.H + h0) * w;
+  for (int r = warp; r < LM_HEADS; r += LM_WARPS)
+#pragma unroll 3
+    for (int c = lane; c < wp / 8; c += WARP) {
+      const bool ok = r < nh && c < nch;
+      cp_async16_zfill(smem_addr(q + r * pitch + c * 8), ok ? qr + (size_t)r * w + c * 8 : qr, ok ? 16 : 0);
+    }
   const long long p = a.pos[b];
   long long lo = p - a.window + 1;
   if (lo < 0) lo = 0;
-  const int len = (int)(p - lo + 1), part = (len + nsplit - 1) / nsplit;
+  const int len = (int)(p - lo + 1), part = (len + a.splits - 1) / a.splits;
   const int t_begin = min(len, sp * part), t_end = min(len, t_begin + part);
   const int slot0 = (int)(lo % a.cap);
   const bf16 *ring = static_cast<const bf16 *>(a.ring) + (size_t)b * a.cap * w;
 
   auto fetch = [&](int t0, int buf) {
     bf16 *dst = tiles + (size_t)buf * LM_TILE * pitch;
-    for (int i = tid; i < LM_TILE * nch; i += LM_THREADS) {
-      const int r = i / nch, c = i - r * nch, t = t0 + r;
+#pragma unroll
+    for (int x = 0; x < LM_TILE / LM_WARPS; ++x) {  // a warp per row
+      const int r = warp + x * LM_WARPS, t = t0 + r;
       const bool ok = t < t_end;
       int slot = slot0 + t;
       if (slot >= a.cap) slot -= a.cap;
-      cp_async16_zfill(smem_addr(dst + r * pitch + c * 8), ok ? ring + (size_t)slot * w + c * 8 : ring, ok ? 16 : 0);
+      const bf16 *src = ok ? ring + (size_t)slot * w : ring;
+      const uint32_t to = smem_addr(dst + r * pitch);
+#pragma unroll 3
+      for (int c = lane; c < nch; c += WARP) cp_async16_zfill(to + c * 16, ok ? src + c * 8 : src, ok ? 16 : 0);
     }
     cp_async_commit();
   };
   fetch(t_begin, 0);
-  const bf16 *qr = static_cast<const bf16 *>(a.qc) + ((size_t)b * a.H + h0) * w;
-  for (int i = tid; i < LM_HEADS * wp / 8; i += LM_THREADS) {
-    const int r = i / (wp / 8), c = i - r * (wp / 8);
-    *reinterpret_cast<uint4 *>(q + r * pitch + c * 8) =
-        r < nh && c < nch ? *reinterpret_cast<const uint4 *>(qr + (size_t)r * w + c * 8) : make_uint4(0, 0, 0, 0);
-  }
   if (nch * 8 < wp)  // the columns that pad a row to whole tiles
     for (int i = tid; i < nbuf * LM_TILE; i += LM_THREADS)
       *reinterpret_cast<uint4 *>(tiles + (size_t)i * pitch + nch * 8) = make_uint4(0, 0, 0, 0);
@@ -82,6 +79,8 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attend_mma_kernel(LatentDec
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[x][y][e] = 0.f;
 
+  const int nt = warp % 4, kh = warp / 4, mid = (wp / 32 + 1) / 2 * 32;  // tokens and part of the row of this warp's scores
+  const int k_begin = kh ? min(mid, wp) : 0, k_end = kh ? wp : min(mid, wp);
   int buf = 0;
   for (int t0 = t_begin; t0 < t_end; t0 += LM_TILE) {
     const bool more = t0 + LM_TILE < t_end;
@@ -90,37 +89,42 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attend_mma_kernel(LatentDec
     else cp_async_wait<0>();
     __syncthreads();
     const bf16 *tile = tiles + (size_t)buf * LM_TILE * pitch;
-    {  // scores of 16 heads against this warp's 8 tokens
-      float s[2][4] = {};
-      const uint32_t qa = smem_addr(q + lrow * pitch + lcol), ka = smem_addr(tile + (warp * 8 + lm) * pitch + lq * 8);
-      for (int k = 0; k < wp; k += 32) {
+    {  // scores of 16 heads against 8 tokens
+      float s[4][4] = {};  // independent chains
+      const uint32_t qa = smem_addr(q + lrow * pitch + lcol), ka = smem_addr(tile + (nt * 8 + lm) * pitch + lq * 8);
+      int k = k_begin;
+#pragma unroll 2
+      for (; k + 64 <= k_end; k += 64) {
+        uint32_t kb[2][4], qf[4][4];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) ldmatrix_x4(kb[x], ka + k * 2 + x * 64);
+#pragma unroll
+        for (int x = 0; x < 4; ++x) ldmatrix_x4(qf[x], qa + k * 2 + x * 32);
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+          mma_m16n8k16_t<bf16>(s[x], qf[x][0], qf[x][1], qf[x][2], qf[x][3], kb[x / 2][x % 2 * 2], kb[x / 2][x % 2 * 2 + 1]);
+      }
+      for (; k < k_end; k += 16) {
         uint32_t kb[4], qf[4];
-        ldmatrix_x4(kb, ka + k * 2);  // k .. k+31 (the second half may be past the row: the pitch's pad, not used)
+        ldmatrix_x4(kb, ka + k * 2);  // (only the first 16 columns are used: the rest may lie past the row)
         ldmatrix_x4(qf, qa + k * 2);
         mma_m16n8k16_t<bf16>(s[0], qf[0], qf[1], qf[2], qf[3], kb[0], kb[1]);
-        if (k + 16 < wp) {
-          ldmatrix_x4(qf, qa + k * 2 + 32);
-          mma_m16n8k16_t<bf16>(s[1], qf[0], qf[1], qf[2], qf[3], kb[2], kb[3]);
-        }
       }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int t = warp * 8 + t4 * 2 + e % 2;
-        sc[g + (e / 2) * 8][t] = t0 + t < t_end ? (s[0][e] + s[1][e]) * a.scale : -INFINITY;
-      }
+      for (int e = 0; e < 4; ++e)
+        sc[kh][g + (e / 2) * 8][nt * 8 + t4 * 2 + e % 2] = (s[0][e] + s[1][e]) + (s[2][e] + s[3][e]);
     }
     __syncthreads();
 #pragma unroll
     for (int x = 0; x < LM_HEADS / LM_WARPS; ++x) {
       const int r = warp * (LM_HEADS / LM_WARPS) + x;
-      const float2 v = *reinterpret_cast<const float2 *>(&sc[r][lane * 2]);
-      const float mx = fmaxf(m_run[r], warp_max(fmaxf(v.x, v.y)));
-      const float e0 = expf(v.x - mx), e1 = expf(v.y - mx);  // 0 past the end
-      const uint32_t hi = pack_bf16(e0, e1);
-      const float2 top = b2f(hi);
-      *reinterpret_cast<uint32_t *>(p_hi + r * LM_PP + lane * 2) = hi;
-      *reinterpret_cast<uint32_t *>(p_lo + r * LM_PP + lane * 2) = pack_bf16(e0 - top.x, e1 - top.y);
-      const float sum = warp_sum(e0 + e1);
+      const float v = t0 + lane < t_end ? (sc[0][r][lane] + sc[1][r][lane]) * a.scale : -INFINITY;
+      const float mx = fmaxf(m_run[r], warp_max(v));
+      const float e = expf(v - mx);  // 0 past the end
+      const bf16 hi = from_f<bf16>(e);
+      p_hi[r * LM_PP + lane] = hi;
+      p_lo[r * LM_PP + lane] = from_f<bf16>(e - to_f(hi));
+      const float sum = warp_sum(e);
       __syncwarp();
       if (lane == 0) {
         corr[r] = m_run[r] == -INFINITY ? 0.f : expf(m_run[r] - mx);
@@ -151,8 +155,8 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attend_mma_kernel(LatentDec
         uint32_t v[4];  // (t 0-7, c 0-7), (t 8-15, c 0-7), (t 0-7, c 8-15), (t 8-15, c 8-15)
         ldmatrix_x4_trans(v, smem_addr(tile + (k + (lq % 2) * 8 + lm) * pitch + col + (lq / 2) * 8));
         mma_m16n8k16_t<bf16>(acc[x][0], ph[0], ph[1], ph[2], ph[3], v[0], v[1]);
-        mma_m16n8k16_t<bf16>(acc[x][0], pl[0], pl[1], pl[2], pl[3], v[0], v[1]);
         mma_m16n8k16_t<bf16>(acc[x][1], ph[0], ph[1], ph[2], ph[3], v[2], v[3]);
+        mma_m16n8k16_t<bf16>(acc[x][0], pl[0], pl[1], pl[2], pl[3], v[0], v[1]);
         mma_m16n8k16_t<bf16>(acc[x][1], pl[0], pl[1], pl[2], pl[3], v[2], v[3]);
       }
     }
@@ -162,89 +166,59 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attend_mma_kernel(LatentDec
   }
   cp_async_wait<0>();  // (of a part without tokens)
   __syncthreads();
-  float *part_o = reinterpret_cast<float *>(sm_raw);  // [heads][rank]: over the queries and tiles
-  const int op = a.rank;
+  if (tid < nh) {
+    float *ml = a.part_ml + (((size_t)b * a.H + h0 + tid) * a.splits + sp) * 2;
+    ml[0] = m_run[tid];
+    ml[1] = l_run[tid];
+  }
+  float *out = a.part_o + (((size_t)b * a.H + h0) * a.splits + sp) * a.rank;
+  const size_t step = (size_t)a.splits * a.rank;  // from head to head
 #pragma unroll
   for (int x = 0; x < NG; ++x)
 #pragma unroll
     for (int y = 0; y < 2; ++y) {
       const int col = (warp + x * LM_WARPS) * 16 + y * 8 + t4 * 2;
       if (col < a.rank) {
-        *reinterpret_cast<float2 *>(part_o + g * op + col) = make_float2(acc[x][y][0], acc[x][y][1]);
-        *reinterpret_cast<float2 *>(part_o + (g + 8) * op + col) = make_float2(acc[x][y][2], acc[x][y][3]);
+        if (g < nh) *reinterpret_cast<float2 *>(out + g * step + col) = make_float2(acc[x][y][0], acc[x][y][1]);
+        if (g + 8 < nh) *reinterpret_cast<float2 *>(out + (g + 8) * step + col) = make_float2(acc[x][y][2], acc[x][y][3]);
       }
     }
-  if (nsplit > 1) {
-    cluster.barrier_wait();
-    cluster.sync();  // every block's sums are in place
-  } else {
-    __syncthreads();
-  }
-  // factors of the parts, then this block's share of the columns
-  if (tid < nsplit * LM_HEADS) {
-    const int s = tid / LM_HEADS, r = tid % LM_HEADS;
-    part_m[s][r] = nsplit > 1 ? cluster.map_shared_rank(m_run, s)[r] : m_run[r];
-    part_l[s][r] = nsplit > 1 ? cluster.map_shared_rank(l_run, s)[r] : l_run[r];
-  }
-  __syncthreads();
-  if (tid < LM_HEADS) {
-    float m = -INFINITY, l = 0.f;
-    for (int s = 0; s < nsplit; ++s) m = fmaxf(m, part_m[s][tid]);
-    for (int s = 0; s < nsplit; ++s) {
-      const float f = part_m[s][tid] == -INFINITY ? 0.f : expf(part_m[s][tid] - m);
-      l = fmaf(f, part_l[s][tid], l);
-      part_m[s][tid] = f;
-    }
-    for (int s = 0; s < nsplit; ++s) part_m[s][tid] /= l;
-  }
-  __syncthreads();
-  const int share = ((a.rank + nsplit - 1) / nsplit + 1) & ~1, j0 = min(a.rank, sp * share), jn = min(share, a.rank - j0) / 2;
-  float *out = a.ctx + ((size_t)b * a.H + h0) * a.rank;
-  for (int i = tid; i < nh * jn; i += LM_THREADS) {
-    const int r = i / jn, j = j0 + (i - r * jn) * 2;
-    float2 v[LM_MAX_SPLITS];
-#pragma unroll
-    for (int s = 0; s < LM_MAX_SPLITS; ++s)
-      if (s < nsplit)
-        v[s] = *reinterpret_cast<const float2 *>((nsplit > 1 ? cluster.map_shared_rank(part_o, s) : part_o) + r * op + j);
-    float2 o = make_float2(0.f, 0.f);
-#pragma unroll
-    for (int s = 0; s < LM_MAX_SPLITS; ++s)
-      if (s < nsplit) {
-        o.x = fmaf(part_m[s][r], v[s].x, o.x);
-        o.y = fmaf(part_m[s][r], v[s].y, o.y);
-      }
-    *reinterpret_cast<float2 *>(out + (size_t)r * a.rank + j) = o;
-  }
-  if (nsplit > 1) cluster.sync();  // no block leaves while another may still read its sums
 }
 
 static size_t lm_smem(const LatentDecodeArgs &a, int nbuf) {
-  const size_t pitch = lm_pitch(a.rank + a.rot);
-  // (32 bytes more: the last row's second half of a 32-column step)
-  const size_t work = (LM_HEADS + (size_t)nbuf * LM_TILE) * pitch * 2 + 32, sums = (size_t)LM_HEADS * a.rank * 4;
-  return work > sums ? work : sums;
+  // (32 bytes more: a last step of 16 columns loads 32)
+  return (LM_HEADS + (size_t)nbuf * LM_TILE) * lm_pitch(a.rank + a.rot) * 2 + 32;
 }
-constexpr size_t LM_SMEM = 210 * 1024;
+constexpr size_t LM_SMEM = 200 * 1024;
+
+int latent_splits(int B, int H, int window) {
+  // at most two blocks of 16 heads per multiprocessor, a pass of tokens each
+  const long long groups = (long long)B * ceil_div(H, LM_HEADS);
+  long long s = 2 * sm_count() / groups;
+  if (s > ceil_div(window, LM_TILE)) s = ceil_div(window, LM_TILE);
+  return s < 1 ? 1 : (s > LD_MAX_SPLITS ? LD_MAX_SPLITS : (int)s);
+}
 
 bool latent_attend_mma_supported(const LatentDecodeArgs &a, bool bf16_rows) {
   return bf16_rows && a.rank % 8 == 0 && a.rot % 8 == 0 && a.rank <= 1024 && aligned16(a.ring) && aligned16(a.qc) &&
-         lm_smem(a, 1) <= LM_SMEM;
+         aligned16(a.part_o) && lm_smem(a, 1) <= LM_SMEM;
 }
 
 int latent_attend_mma(const LatentDecodeArgs &a, cudaStream_t st) {
-  const int nbuf = lm_smem(a, 2) <= LM_SMEM ? 2 : 1;
+  const int part = ceil_div(a.window, a.splits), nbuf = part > 4 * LM_TILE && lm_smem(a, 2) <= LM_SMEM ? 2 : 1;
   const size_t smem = lm_smem(a, nbuf);
-  const int hb = ceil_div(a.H, LM_HEADS);
-  // parts of the window: as long as each has a pass of its own and the blocks fit the device at once
-  int nsplit = 1;
-  while (nsplit < LM_MAX_SPLITS && a.window > LM_TILE * nsplit && (long long)hb * a.B * nsplit * 2 <= sm_count()) nsplit *= 2;
-  const dim3 grid(hb, a.B, nsplit);
+  const dim3 grid(ceil_div(a.H, LM_HEADS), a.B, a.splits);
+  // No more shared memory per multiprocessor than the blocks of this launch fill: in a chain of early launched kernels the
+  // ones that follow live with the split between shared memory and L1 they find, and they want L1 for their activations.
+  const long long blocks = (long long)grid.x * grid.y * grid.z;
+  const int per_sm = blocks <= sm_count() ? 1 : 2;
+  const int carveout = (int)((per_sm * (smem + 8 * 1024) * 100 + 228 * 1024 - 1) / (228 * 1024));
 #define DJV_GO(G_)                                                                                                       \
   {                                                                                                                      \
     cudaFuncSetAttribute(latent_attend_mma_kernel<G_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LM_SMEM);       \
-    djv::launch_kernel_cluster(latent_attend_mma_kernel<G_>, grid, dim3(LM_THREADS), smem, st, dim3(1, 1, nsplit), a,    \
-                               nbuf);                                                                                    \
+    cudaFuncSetAttribute(latent_attend_mma_kernel<G_>, cudaFuncAttributePreferredSharedMemoryCarveout,                   \
+                         carveout < 100 ? carveout : 100);                                                               \
+    djv::launch_kernel(latent_attend_mma_kernel<G_>, grid, dim3(LM_THREADS), smem, st, a, nbuf);                         \
   }
   const int ng = ceil_div(a.rank, 16 * LM_WARPS);
   if (ng == 1) DJV_GO(1)

@@ -240,10 +240,11 @@ class LatentAttention(nn.Module):
             return self.o.rows(ctx, True, torch.float32)
         past = min(past, window - 1, ring.shape[1])
         ops.rotary_(proj[:, dim:], self.rotary.freqs, self.rotary.amp, pos, n, H, dim + rot, interleaved=True)
-        rows = ops.latent_rows(proj[:, a:b], ring, self.norm, self.eps, self.rotary.freqs, pos, n, past, rank)
+        rows = ops.latent_rows(proj[:, a:b], ring, self.norm, self.eps, self.rotary.freqs, pos, n, past, rank, store=past == 0)
         kv = self.ukv(rows[:, :rank])
         ctx = ops.latent_attention(proj[:, :a], kv, rows[:, rank:], gate, pos, n, past, H, dim, rot, window, self.scale)
-        ops.latent_store(rows, ring, self.norm, self.rotary.freqs, pos, n, past, rank)
+        if past:
+            ops.latent_store(rows, ring, self.norm, self.rotary.freqs, pos, n, past, rank)
         return self.o(ctx, torch.float32)
 
 
@@ -311,10 +312,7 @@ class MixtureOfExperts(nn.Module):
         if n == 1 and h.shape[0] <= _lib.MAX_BATCH:
             if self.shared is None:
                 return ops.moe_decode(h, z, self.gate_up, self.down, self.top)
-            if h.shape[0] <= 4:  # the shared expert runs beside the others; for more rows its products share their weights
-                return ops.moe_decode(h, z, self.gate_up, self.down, self.top, self.shared.gate_up.weight,
-                                      self.shared.down.weight)
-            return ops.moe_decode(h, z, self.gate_up, self.down, self.top, init=self.shared(h, n))
+            return ops.moe_decode(h, z, self.gate_up, self.down, self.top, self.shared.gate_up.weight, self.shared.down.weight)
         xs, ws, offsets, places = ops.moe_route(h, z, self.top)
         a = ops.moe_grouped(xs, self.gate_up, offsets, ws, glu=True)
         return SplitSum(None if self.shared is None else self.shared(h, n), ops.moe_grouped(a, self.down, offsets), places)

@@ -678,9 +678,10 @@ def mlstm(proj, gates, bias_i, bias_f, cap: float, norm, eps: float, scale: floa
     return out
 
 
-def latent_rows(proj, ring, norm, eps: float, freqs, pos, n: int, past: int, rank: int):
+def latent_rows(proj, ring, norm, eps: float, freqs, pos, n: int, past: int, rank: int, store: bool = False):
     """Cache rows (latent | shared key part) of `past` earlier tokens per sequence, from the ring, and of n new ones, from
-    proj (B*n, rank + rot), a view with any row stride: (B * (past + n), rank + rot)."""
+    proj (B*n, rank + rot), a view with any row stride: (B * (past + n), rank + rot). store (with past 0 only): the new
+    rows enter the ring as well."""
     B, cap, width = ring.shape
     b = pos.numel()
     assert b <= B and proj.shape == (b * n, width) and proj.stride(1) == 1 and proj.dtype == ring.dtype
@@ -689,7 +690,8 @@ def latent_rows(proj, ring, norm, eps: float, freqs, pos, n: int, past: int, ran
     _f32(norm, freqs)
     rows = torch.empty(b * (past + n), width, dtype=ring.dtype, device=ring.device)
     call("djv_latent_rows", _dtype_code(ring), rows.data_ptr(), proj.data_ptr(), proj.stride(0), ring.data_ptr(),
-         norm.data_ptr(), float(eps), freqs.data_ptr(), pos.data_ptr(), b, n, past, rank, width - rank, cap, 0, _stream())
+         norm.data_ptr(), float(eps), freqs.data_ptr(), pos.data_ptr(), b, n, past, rank, width - rank, cap, 2 if store else 0,
+         _stream())
     return rows
 
 
@@ -722,7 +724,7 @@ def latent_attention_decode(proj, uk, uv, norm, eps: float, freqs, ring, gate, p
                             stages: int = 7, scratch=None):
     """One token per sequence on the ring itself: proj (B, q | latent | key part, ...) neither normed nor rotated, uk
     (H*dim, rank), uv (H*dv, rank), gate (B, H*dv) or None. Returns (B, H*dv). stages (1 queries and cache row, 2
-    attention, 4 values) and scratch (qc, ctx) are for timing the kernels one by one."""
+    attention, 4 values) and scratch (qc, sums) are for timing the kernels one by one."""
     B, cap, width = ring.shape
     b, rank = pos.numel(), uk.shape[1]
     dim, dv, rot = uk.shape[0] // heads, uv.shape[0] // heads, width - rank
@@ -732,11 +734,12 @@ def latent_attention_decode(proj, uk, uv, norm, eps: float, freqs, ring, gate, p
     _require_cuda(proj, uk, uv, ring, pos, gate)
     _f32(norm, freqs)
     dev = ring.device
-    qc, ctx = scratch or (torch.empty(b, heads, width, dtype=ring.dtype, device=dev),
-                          torch.empty(b, heads, rank, dtype=torch.float32, device=dev))
+    floats = _lib.load_routed().djv_latent_scratch_floats(b, heads, rank, min(window, cap))
+    qc, sums = scratch or (torch.empty(b, heads, width, dtype=ring.dtype, device=dev),
+                           torch.empty(floats, dtype=torch.float32, device=dev))
     out = torch.empty(b, heads * dv, dtype=ring.dtype, device=dev)
-    call("djv_latent_decode", _dtype_code(ring), out.data_ptr(), qc.data_ptr(), ctx.data_ptr(), proj.data_ptr(),
-         proj.stride(0), uk.data_ptr(), uv.data_ptr(), norm.data_ptr(), float(eps), freqs.data_ptr(), ring.data_ptr(),
+    call("djv_latent_decode", _dtype_code(ring), out.data_ptr(), qc.data_ptr(), sums.data_ptr(), sums.numel(),
+         proj.data_ptr(), proj.stride(0), uk.data_ptr(), uv.data_ptr(), norm.data_ptr(), float(eps), freqs.data_ptr(), ring.data_ptr(),
          _ptr(gate), 0 if gate is None else gate.stride(0), pos.data_ptr(), b, heads, dim, rot, dv, rank, cap, window,
          float(scale), stages, _stream())
     return out

@@ -3,6 +3,7 @@
     python -m dejavu_b200.profile_cases <case>
         case: qkv | out_proj | attn | topk | exchange | ring | fc1 | fc2 | fc1_b16 | fc2_b16 | ring_trace
               hybrid_window | hybrid_gla | hybrid_decode   (shapes of the 7b size of bench.py --hybrid)
+              routed_memory | routed_experts | routed_latent | routed_decode   (the same of bench.py --routed)
 
 Every case launches ONE kind of kernel a dozen times at the per-rank shapes of an OPT-175B layer under 8-way
 tensor parallelism (d 12288, 12 local heads of which 4 are active, 512 of 6144 ffn rows), rotating several weight
@@ -94,6 +95,31 @@ def main(case: str) -> None:
             freqs = torch.rand(dk // 2, device=dev)
             for r in rings: ops.window_attention_decode(row, *r, sink, freqs, 1.0, far, H, W, dk ** -0.5)
             for s in states: ops.gated_linear_attention(prow, *gla, s, far, 1)
+    elif case in ("routed_memory", "routed_experts", "routed_latent", "routed_decode"):
+        from .routed_bench import DIM, RANK, ROT, VDIM
+        H, W, GH, gk, gv, n, D, E, ff, top = 32, 1024, 16, 128, 256, 4096, 4096, 8, 3648, 2
+        def bf(*shape): return torch.randn(*shape, device=dev, generator=g).bfloat16()
+        def f32(*shape): return torch.randn(*shape, device=dev, generator=g)
+        pos, far = torch.zeros(1, dtype=torch.int64, device=dev), torch.full((1,), 5000, dtype=torch.int64, device=dev)
+        mem = (torch.zeros(GH, device=dev), torch.full((GH,), 3.0, device=dev), 15.0, torch.ones(GH * gv, device=dev), 1e-6, gk ** -0.5)
+        main, width, norm, freqs = 2 * GH * (gk + gv), RANK + ROT, torch.ones(RANK, device=dev), torch.rand(ROT // 2, device=dev)
+        if case == "routed_memory":
+            rows, gates, st = [bf(n, main) for _ in range(2)], f32(n, 2 * GH), ops.mlstm_state(1, GH, gk, gv, dev)
+            for r in rows * 2: ops.mlstm(r, gates, *mem, st, pos, n, gk, gv, torch.bfloat16)
+        elif case == "routed_experts":
+            x, z, w = bf(n, D), f32(n, E), [bf(E, 2 * ff, D) for _ in range(2)]
+            for wi in w * 2:
+                xs, ws, off, _ = ops.moe_route(x, z, top)
+                ops.moe_grouped(xs, wi, off, ws, glu=True)
+        elif case == "routed_latent":
+            q, kv, tail, gate = bf(n, H * (DIM + ROT)), bf(n, H * (DIM + VDIM)), bf(n, ROT), bf(n, H * VDIM)
+            for _ in range(4): ops.latent_attention(q, kv, tail, gate, pos, n, 0, H, DIM, ROT, W, (DIM + ROT) ** -0.5)
+        else:
+            proj, uk, uv, gate = bf(1, H * (DIM + ROT) + width), bf(H * DIM, RANK), bf(H * VDIM, RANK), bf(1, H * VDIM)
+            for r in [bf(1, W, width) for _ in range(8)]:
+                ops.latent_attention_decode(proj, uk, uv, norm, 1e-6, freqs, r, gate, far, H, W, (DIM + ROT) ** -0.5)
+            prow = f32(1, main + 2 * GH)
+            for _ in range(4): ops.mlstm(prow, prow[:, main:], *mem, ops.mlstm_state(1, GH, gk, gv, dev), far, 1, gk, gv, torch.bfloat16)
     torch.cuda.synchronize()
     if case == "ring_trace":
         lib = _lib.load()

@@ -38,7 +38,7 @@ unsigned djv_mlstm_timeouts(void);
  * that all heads share; the ring (B, cap, rank + rot) holds position p in slot p % cap, cap >= min(window, longest sequence).
  * djv_latent_rows, store = 0: rows (B, past + n, rank + rot) from the ring (positions pos - past .. pos - 1, zeros before
  * position 0) and from proj (B*n rows of latent | key part, ld apart). store = 1: the last min(n, cap) of these rows enter
- * the ring (proj is not read). `past` is no less than what a sequence can see of its earlier tokens. */
+ * the ring (proj is not read); store = 2: both, for past = 0. `past` is no less than what a sequence can see of its earlier tokens. */
 int djv_latent_rows(int dtype, void *rows, const void *proj, long long ld, void *ring, const float *norm, float eps,
                     const float *freqs, const long long *pos, int B, int n, int past, int rank, int rot, int cap,
                     int store, void *stream);
@@ -51,12 +51,14 @@ int djv_latent_attn(int dtype, void *out, const void *q, long long ldq, const vo
 /* The decode step of the same on the ring itself. proj rows hold q (H, dim + rot) | latent (rank) | key part (rot), neither
  * normed nor rotated; uk (H*dim, rank), uv (H*dv, rank). stages is a sum of
  *   1  qc (B, H, rank + rot) = (uk_h^T q_h | rotated q_h), and the token's row enters the ring
- *   2  ctx (B, H, rank) fp32 = softmax(qc . ring rows * scale) times the rows' latents
- *   4  out (B, H*dv) = uv_h ctx_h, times sigmoid(gate) */
-int djv_latent_decode(int dtype, void *out, void *qc, float *ctx, const void *proj, long long ld, const void *uk,
-                      const void *uv, const float *norm, float eps, const float *freqs, void *ring, const void *gate,
-                      long long ldg, const long long *pos, int B, int H, int dim, int rot, int dv, int rank, int cap,
-                      int window, float scale, int stages, void *stream);
+ *   2  scratch (djv_latent_scratch_floats with window <= cap) = weighted sums of the rows' latents over parts of the window,
+ *      weights from softmax(qc . ring rows * scale)
+ *   4  out (B, H*dv) = uv_h applied to the parts put together, times sigmoid(gate) */
+size_t djv_latent_scratch_floats(int B, int H, int rank, int window);
+int djv_latent_decode(int dtype, void *out, void *qc, float *scratch, size_t scratch_floats, const void *proj, long long ld,
+                      const void *uk, const void *uv, const float *norm, float eps, const float *freqs, void *ring,
+                      const void *gate, long long ldg, const long long *pos, int B, int H, int dim, int rot, int dv,
+                      int rank, int cap, int window, float scale, int stages, void *stream);
 
 /* Routed feed-forward: a token's `top` largest router logits z choose its experts, with weights sigmoid(z).
  * djv_moe_route sorts n tokens' choices by expert: xs (n*top, D) their activations, ws (n*top) their weights, offsets

@@ -125,7 +125,8 @@ def test_kernels_check_their_arguments_on_the_host():
     assert lib.djv_latent_rows(BF, p, p, 20, p, p, 1e-5, p, p, 1, 4, 0, 16, 8, 8, 0, None) == bad
     assert lib.djv_latent_rows(BF, p, p, 24, p, p, 1e-5, p, p, 1, 4, 9, 16, 8, 8, 0, None) == bad
     assert lib.djv_latent_attn(BF, p, p, 47, p, 64, p, 8, None, 0, p, 1, 4, 0, 2, 16, 8, 16, 8, 1.0, None) == bad
-    assert lib.djv_latent_decode(BF, p, p, p, p, 60, p, p, p, 1e-5, p, p, None, 0, p, 1, 2, 16, 8, 16, 16, 8, 8, 1.0, 7, None) == bad
+    assert lib.djv_latent_decode(BF, p, p, p, 1 << 20, p, 60, p, p, p, 1e-5, p, p, None, 0, p, 1, 2, 16, 8, 16, 16, 8, 8, 1.0, 7, None) == bad
+    assert lib.djv_latent_decode(BF, p, p, p, 16, p, 72, p, p, p, 1e-5, p, p, None, 0, p, 1, 2, 16, 8, 16, 16, 8, 8, 1.0, 7, None) == _lib.ERR_SCRATCH
     assert lib.djv_moe_route(BF, p, p, p, p, p, p, p, p, p, 4, 3, 4, 64, None) == bad
     assert lib.djv_moe_grouped(BF, p, p, p, None, p, 4, 3, 7, 64, 1, None) == bad
     assert lib.djv_moe_decode(BF, p, p, p, p, p, p, p, p, None, None, 1, 4, 1, 64, 32, 16, 32, 3, None) == bad
