@@ -287,8 +287,8 @@ __global__ void __launch_bounds__(LS_THREADS) latent_attend_simple_kernel(Latent
 // row).
 constexpr int LO_THREADS = 256, LO_WARPS = LO_THREADS / WARP, LO_ROWS = 4;
 template <typename T, int U>  // U == 0: any rank and alignment
-__global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(LatentDecodeArgs a, int per) {
-  extern __shared__ __align__(16) float ctx[];  // rank
+__global__ void __launch_bounds__(LO_THREADS, U > 2 ? 1 : 2) latent_out_kernel(LatentDecodeArgs a, int per) {
+  extern __shared__ __align__(16) float ctx[];  // [2][rank]: two partial sums
   __shared__ float factor[LD_MAX_SPLITS];
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   const int tid = threadIdx.x, lane = tid % WARP, warp = tid / WARP, h = blockIdx.y;
@@ -319,16 +319,21 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(LatentDecodeArgs
     __syncthreads();
     const float *part = a.part_o + bh * a.splits * a.rank;
     if (U > 0) {
-      for (int c = tid * 2; c < a.rank; c += LO_THREADS * 2) {
-        float2 o = make_float2(0.f, 0.f);
-#pragma unroll 16
-        for (int s = 0; s < a.splits; ++s) {
+      // two halves of the block take every other part, 4 columns per thread
+      constexpr int HALF = LO_THREADS / 2;
+      float *dst = ctx + tid / HALF * a.rank;
+      for (int c = tid % HALF * 4; c < a.rank; c += HALF * 4) {
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int s = tid / HALF; s < a.splits; s += 2) {
           const float f = factor[s];  // (0: an empty part, whose sums may be anything)
-          const float2 v = f != 0.f ? *reinterpret_cast<const float2 *>(part + (size_t)s * a.rank + c) : make_float2(0.f, 0.f);
+          const float4 v = f != 0.f ? *reinterpret_cast<const float4 *>(part + (size_t)s * a.rank + c) : make_float4(0.f, 0.f, 0.f, 0.f);
           o.x = fmaf(f, v.x, o.x);
           o.y = fmaf(f, v.y, o.y);
+          o.z = fmaf(f, v.z, o.z);
+          o.w = fmaf(f, v.w, o.w);
         }
-        *reinterpret_cast<float2 *>(ctx + c) = o;
+        *reinterpret_cast<float4 *>(dst + c) = o;
       }
     } else {
       for (int c = tid; c < a.rank; c += LO_THREADS) {
@@ -349,7 +354,14 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(LatentDecodeArgs
         if (c < nch) {
           float xv[N];
 #pragma unroll
-          for (int e = 0; e < N; e += 4) *reinterpret_cast<float4 *>(xv + e) = *reinterpret_cast<const float4 *>(ctx + c * N + e);
+          for (int e = 0; e < N; e += 4) {
+            const float4 u0 = *reinterpret_cast<const float4 *>(ctx + c * N + e);
+            const float4 u1 = *reinterpret_cast<const float4 *>(ctx + a.rank + c * N + e);
+            xv[e] = u0.x + u1.x;
+            xv[e + 1] = u0.y + u1.y;
+            xv[e + 2] = u0.z + u1.z;
+            xv[e + 3] = u0.w + u1.w;
+          }
 #pragma unroll
           for (int r = 0; r < LO_ROWS; ++r) {
             float f[N];
@@ -410,8 +422,9 @@ static int launch_out(const LatentDecodeArgs &a, cudaStream_t st) {
   constexpr int N = Chunk<T>::N;
   const int per = ceil_div(a.B, LATENT_GROUPS);
   const dim3 grid(ceil_div(a.dv, LO_WARPS * LO_ROWS), a.H, ceil_div(a.B, per));
-  const size_t smem = (size_t)a.rank * 4;
-  const int u = a.rank % N == 0 && aligned16(a.uv) && aligned16(a.part_o) ? ceil_div(a.rank / N, WARP) : 0;
+  int u = a.rank % N == 0 && aligned16(a.uv) && aligned16(a.part_o) ? ceil_div(a.rank / N, WARP) : 0;
+  if (u > 4) u = 0;
+  const size_t smem = (size_t)a.rank * (u ? 8 : 4);
   if (u == 1) djv::launch_kernel(latent_out_kernel<T, 1>, grid, dim3(LO_THREADS), smem, st, a, per);
   else if (u == 2) djv::launch_kernel(latent_out_kernel<T, 2>, grid, dim3(LO_THREADS), smem, st, a, per);
   else if (u == 3 || u == 4) djv::launch_kernel(latent_out_kernel<T, 4>, grid, dim3(LO_THREADS), smem, st, a, per);

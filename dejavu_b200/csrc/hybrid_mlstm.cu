@@ -437,6 +437,8 @@ static int launch_prefill(const MlstmArgs &a, bool tc, cudaStream_t st) {
   const dim3 grid(a.nc, a.H, a.B);
   int rc = DJV_OK;
   if (tc) {
+    rc = mlstm_tc_gates(a, st);
+    if (rc) return rc;
     rc = mlstm_tc_chunk_state(a, st);
     if (rc) return rc;
   } else {
@@ -519,7 +521,7 @@ extern "C" size_t djv_mlstm_scratch_bytes(int dtype, int B, int n, int H, int dk
     if (C == 0) continue;
     const size_t rows = (size_t)B * H * ceil_div(n, C);
     size_t need = al256(rows * mlstm_contrib_stride(dk, dv) * 4) + al256(rows * 3 * 8);
-    if (tc) need += 2 * al256(rows * dk * dv * 2);
+    if (tc) need += 2 * al256(rows * dk * dv * 2) + 3 * al256(rows * C * 8);
     if (need > most) most = need;
   }
   return most;
@@ -530,7 +532,7 @@ extern "C" int djv_mlstm_prefill(int dtype, void *out, const void *proj, long lo
                                  float scale, float *state, const long long *pos, int B, int n, int H, int dk, int dv,
                                  void *scratch, size_t scratch_bytes, void *stream) {
   MlstmArgs a{out, proj, ld, gates, ldg, bias_i, bias_f, cap, norm, eps, scale, state, pos, B, n, H, dk, dv, 0, 0,
-              nullptr, nullptr, nullptr, nullptr};
+              nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr};
   int rc = check_mlstm("mlstm_prefill", dtype, a);
   if (rc) return rc;
   const bool tc = use_tc(dtype, a);
@@ -555,6 +557,12 @@ extern "C" int djv_mlstm_prefill(int dtype, void *out, const void *proj, long lo
     a.s_hi = reinterpret_cast<bf16 *>(p);
     p += al256(rows * dk * dv * 2);
     a.s_lo = reinterpret_cast<bf16 *>(p);
+    p += al256(rows * dk * dv * 2);
+    a.g_a = reinterpret_cast<float2 *>(p);
+    p += al256(rows * a.C * 8);
+    a.g_run = reinterpret_cast<double *>(p);
+    p += al256(rows * a.C * 8);
+    a.g_sum = reinterpret_cast<double *>(p);
   }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return dtype == DJV_DTYPE_BF16 ? launch_prefill<bf16>(a, tc, st) : launch_prefill<float>(a, false, st);
@@ -565,7 +573,7 @@ extern "C" int djv_mlstm_decode(int dtype, void *out, const float *proj, long lo
                                 float scale, float *state, const long long *pos, int B, int H, int dk, int dv,
                                 void *stream) {
   const MlstmArgs a{out, proj, ld, gates, ldg, bias_i, bias_f, cap, norm, eps, scale, state, pos, B, 1, H, dk, dv, 0, 0,
-                    nullptr, nullptr, nullptr, nullptr};
+                    nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr};
   int rc = check_mlstm("mlstm_decode", dtype, a);
   if (rc) return rc;
   cudaStream_t st = static_cast<cudaStream_t>(stream);

@@ -23,6 +23,8 @@ struct MlstmArgs {
   float *contrib;        // (B, H, nc, dk * dv + dk): a chunk's own S and n, then the incoming ones
   double *chunk;         // (B, H, nc, 3): sum of log f, maximum of a, incoming m
   bf16 *s_hi, *s_lo;     // (B, H, nc, dk, dv): incoming S as two bf16 terms (tensor-core form)
+  float2 *g_a;           // (B, H, nc, C): a_s of every token, and (below) M_t without m_in and F_t (tensor-core form)
+  double *g_run, *g_sum;
 };
 
 // a head's state: S (dk, dv), n (dk), m
@@ -100,6 +102,7 @@ __device__ __forceinline__ void chunk_gates(const MlstmArgs &a, int b, int h, in
 // tensor-core form of the chunk kernels (bf16); chunks of MLSTM_TC_CHUNK tokens
 constexpr int MLSTM_TC_CHUNK = 128;
 bool mlstm_tc_supported(int dtype, int dk, int dv);
+int mlstm_tc_gates(const MlstmArgs &a, cudaStream_t st);
 int mlstm_tc_chunk_state(const MlstmArgs &a, cudaStream_t st);
 int mlstm_tc_chunk_out(const MlstmArgs &a, cudaStream_t st);
 

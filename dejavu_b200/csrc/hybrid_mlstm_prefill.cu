@@ -5,7 +5,7 @@
 // Outputs: S = Q K^T (TMEM); P_ts = S_ts e^(a_s - M_t) for s <= t goes back to TMEM over S, as hi + lo; O (TMEM) = Q S_in, S_in
 // in hi + lo, scaled by e^(m_in - M_t) row by row, then += P_hi V + P_lo V. The denominator takes the fp32 sums of P and
 // q . n_in. Norm and gate run on the way out. The incoming state streams through two buffers of 64 channels; V takes the one
-// that is free first. A block has 256 threads, two per row of TMEM, and up to 256 value columns; wider heads are a cluster of
+// that is free first, the output gates the other. A block has 256 threads, two per row of TMEM, and up to 256 value columns; wider heads are a cluster of
 // blocks that exchange their sums of squares.
 #include <cooperative_groups.h>
 
@@ -47,13 +47,36 @@ __device__ __forceinline__ void split_pair(float x, float y, uint32_t &hi, uint3
   lo = pack_bf16(x - __uint_as_float(__float_as_uint(x) & 0xffff0000u), y - __uint_as_float(__float_as_uint(y) & 0xffff0000u));
 }
 
+// ---- gates of all chunks, a warp each ----------------------------------------------------------------------------------
+constexpr int MG_WARPS = 4;
+__global__ void __launch_bounds__(MG_WARPS * WARP) mlstm_tc_gates_kernel(MlstmArgs a) {
+  __shared__ float2 as[MG_WARPS][MT_C];
+  __shared__ double run[MG_WARPS][MT_C], sum[MG_WARPS][MT_C];
+  pdl_prologue();
+  const int warp = threadIdx.x / WARP, lane = threadIdx.x % WARP, ci = blockIdx.x * MG_WARPS + warp;
+  const int h = blockIdx.y, b = blockIdx.z;
+  if (ci >= a.nc) return;
+  double total, top;
+  chunk_gates<MT_C / WARP>(a, b, h, ci * MT_C, min(MT_C, a.n - ci * MT_C), as[warp], run[warp], sum[warp], total, top);
+  __syncwarp();
+  const size_t at = ((size_t)b * a.H + h) * a.nc + ci;
+  for (int t = lane; t < MT_C; t += WARP) {
+    a.g_a[at * MT_C + t] = as[warp][t];
+    a.g_run[at * MT_C + t] = run[warp][t];
+    a.g_sum[at * MT_C + t] = sum[warp][t];
+  }
+  if (lane == 0) {
+    a.chunk[at * 3] = total;
+    a.chunk[at * 3 + 1] = top;
+  }
+}
+
 // ---- a chunk's own contribution to the state -----------------------------------------------------------------------
 template <int KB, int VB>  // 64-column blocks: keys (2 or 4: M comes in 128 channels), values
 __global__ void __launch_bounds__(ML_THREADS, KB > 2 ? 1 : 2) mlstm_tc_chunk_state_kernel(MlstmArgs a, int nvt) {
   extern __shared__ unsigned char smem_raw[];
   __shared__ __align__(8) uint64_t bar;
   __shared__ uint32_t tmem_slot;
-  __shared__ float2 as[MT_C];
   constexpr int PER = KB * 8, STEP = ML_THREADS / PER;  // chunks of 8 channels in a row, rows at a time
   __shared__ float wt[MT_C], nsum[STEP][KB * 64];
   constexpr uint32_t COLS = KB > 2 ? 256 : (VB > 1 ? 128 : 64);
@@ -76,19 +99,9 @@ __global__ void __launch_bounds__(ML_THREADS, KB > 2 ? 1 : 2) mlstm_tc_chunk_sta
   load_tile<VB, MT_C>(v_sm, rows + (size_t)2 * a.H * dk + (size_t)h * dv + v0, a.ld, cl, vn);
   cp_async_commit();
   const size_t at = ((size_t)b * a.H + h) * a.nc + ci;
-  if (warp == 0) {
-    __syncwarp();
-    tmem_alloc(&tmem_slot, COLS);
-    double total, top;
-    chunk_gates<MT_C / WARP>(a, b, h, t0, cl, as, nullptr, nullptr, total, top);
-    __syncwarp();
-    const float2 m = split_double(top);
-    for (int t = tid; t < MT_C; t += WARP) wt[t] = exp_diff(as[t], m);
-    if (tid == 0 && vt == 0) {
-      a.chunk[at * 3] = total;
-      a.chunk[at * 3 + 1] = top;
-    }
-  }
+  __syncwarp();
+  if (warp == 0) tmem_alloc(&tmem_slot, COLS);
+  if (tid < MT_C) wt[tid] = exp_diff(a.g_a[at * MT_C + tid], split_double(a.chunk[at * 3 + 1]));
   cp_async_wait<1>();
   __syncthreads();
   {  // weighted keys, split in place; a thread keeps its chunk of 8 channels over the rows and sums them for n
@@ -181,12 +194,11 @@ __global__ void __launch_bounds__(ML_THREADS, VB > 2 ? 1 : 2) mlstm_tc_chunk_out
   __shared__ __align__(8) uint64_t bar_s, bar_o, bar_buf[2];
   __shared__ uint32_t tmem_slot;
   __shared__ float2 as[MT_C], mt[MT_C];  // in units of log 2
-  __shared__ float w_in[MT_C], floor_s[MT_C], exch[2][MT_C], ssq[MT_MAX_TILES][MT_C], n_in[KB * 64];
-  __shared__ double run[MT_C], fs[MT_C];
+  __shared__ float w_in[MT_C], floor_s[MT_C], exch[2][MT_C], ssq[MT_MAX_TILES][MT_C], n_in[KB * 64], norm_s[VB * 64];
   constexpr uint32_t COLS = VB > 2 ? 512 : 256;
   constexpr uint32_t SLICE = 64 * 128;            // bytes of a 64-column block of 64 channels
   constexpr uint32_t BUF = 2 * VB * SLICE;        // hi and lo of 64 channels; or 128 rows of V
-  const int tid = threadIdx.x, warp = tid / WARP, lane = tid % WARP;
+  const int tid = threadIdx.x, warp = tid / WARP;
   const int half = tid / MT_C, r = tid % MT_C;
   const int vt = blockIdx.x, nvt = gridDim.x, ci = blockIdx.y, h = blockIdx.z % a.H, b = blockIdx.z / a.H;
   const int dk = a.dk, dv = a.dv, v0 = vt * VB * 64, vn = min(VB * 64, dv - v0);
@@ -205,7 +217,7 @@ __global__ void __launch_bounds__(ML_THREADS, VB > 2 ? 1 : 2) mlstm_tc_chunk_out
     mbar_fence_init();
   }
   const bf16 *rows = static_cast<const bf16 *>(a.proj) + ((size_t)b * a.n + t0) * a.ld;
-  const bf16 *v_rows = rows + (size_t)2 * a.H * dk + (size_t)h * dv + v0, *gate = v_rows + (size_t)a.H * dv + (long long)r * a.ld;
+  const bf16 *v_rows = rows + (size_t)2 * a.H * dk + (size_t)h * dv + v0, *gate = v_rows + (size_t)a.H * dv;
   const size_t at = ((size_t)b * a.H + h) * a.nc + ci;
   load_tile<KB, MT_C>(q_sm, rows + (size_t)h * dk, a.ld, cl, dk);
   load_tile<KB, MT_C>(k_sm, rows + (size_t)(a.H + h) * dk, a.ld, cl, dk);
@@ -219,27 +231,19 @@ __global__ void __launch_bounds__(ML_THREADS, VB > 2 ? 1 : 2) mlstm_tc_chunk_out
   };
   slice(0);
   if (KB > 1) slice(1);
-  if (warp == 0) {
-    __syncwarp();
-    tmem_alloc(&tmem_slot, COLS);
-    double total, top;
-    chunk_gates<MT_C / WARP>(a, b, h, t0, cl, as, run, fs, total, top);
-    __syncwarp();
-    const double m0 = a.chunk[at * 3 + 2];
-    for (int t = lane; t < MT_C; t += WARP) {
-      const double M = fmax(run[t], m0);
-      mt[t] = split_double(M * LOG2E);
-      const float2 x = as[t];
-      as[t] = split_double(((double)x.x + (double)x.y) * LOG2E);
-      w_in[t] = expf((float)(m0 - M)) * a.scale;
-      floor_s[t] = expf((float)-(fs[t] + M));
-    }
+  __syncwarp();
+  if (warp == 0) tmem_alloc(&tmem_slot, COLS);
+  if (tid < MT_C) {
+    const double m0 = a.chunk[at * 3 + 2], M = fmax(a.g_run[at * MT_C + tid], m0);
+    const float2 x = a.g_a[at * MT_C + tid];
+    mt[tid] = split_double(M * LOG2E);
+    as[tid] = split_double(((double)x.x + (double)x.y) * LOG2E);
+    w_in[tid] = expf((float)(m0 - M)) * a.scale;
+    floor_s[tid] = expf((float)-(a.g_sum[at * MT_C + tid] + M));
   } else {
     const float *N = a.contrib + at * mlstm_contrib_stride(dk, dv) + (size_t)dk * dv;
-    for (int c = tid - WARP; c < KB * 64; c += ML_THREADS - WARP) n_in[c] = c < dk ? N[c] : 0.f;
-    // the gates are needed last: have them in L2 by then
-    if (tid >= MT_C && r < cl)
-      for (int j = 0; j < vn; j += 64) prefetch_l2(gate + j);
+    for (int c = tid - MT_C; c < KB * 64; c += ML_THREADS - MT_C) n_in[c] = c < dk ? N[c] : 0.f;
+    for (int c = tid - MT_C; c < VB * 64; c += ML_THREADS - MT_C) norm_s[c] = c < vn ? a.norm[(size_t)h * dv + v0 + c] : 0.f;
   }
   cp_async_wait<(KB > 1 ? 2 : 1)>();
   fence_proxy_async_smem();
@@ -335,19 +339,28 @@ __global__ void __launch_bounds__(ML_THREADS, VB > 2 ? 1 : 2) mlstm_tc_chunk_out
   load_tile<VB, MT_C>(buf_sm + VBUF * BUF, v_rows, a.ld, cl, vn);
   cp_async_commit();
   if (!dead) dead = !mbar_wait(&bar_buf[(KB - 1) & 1], ((KB - 1) / 2) & 1);
+  // the gates take the last slice's buffer
+  load_tile<VB, MT_C>(buf_sm + (VBUF ^ 1) * BUF, gate, a.ld, cl, vn);
+  cp_async_commit();
   __syncwarp();
   tmem_fence_after();
-  for (int q = half * 16; q < np; q += 32) {
-    uint32_t o[16];
-    tmem_ld16(o, tm_o + lane_base + q);
+#pragma unroll 2
+  for (int q = half * 16; q < np; q += 64) {  // two groups of 16 columns at a time
+    const bool two = q + 32 < np;
+    uint32_t o[2][16];
+    tmem_ld16(o[0], tm_o + lane_base + q);
+    if (two) tmem_ld16(o[1], tm_o + lane_base + q + 32);
     tmem_wait_ld();
 #pragma unroll
-    for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * win);
-    tmem_st16(tm_o + lane_base + q, o);
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int e = 0; e < 16; ++e) o[x][e] = __float_as_uint(__uint_as_float(o[x][e]) * win);
+    tmem_st16(tm_o + lane_base + q, o[0]);
+    if (two) tmem_st16(tm_o + lane_base + q + 32, o[1]);
   }
   tmem_wait_st();
   tmem_fence_before();
-  cp_async_wait<0>();
+  cp_async_wait<1>();  // V
   fence_proxy_async_smem();
   __syncthreads();
   if (tid == 0) {
@@ -364,17 +377,23 @@ __global__ void __launch_bounds__(ML_THREADS, VB > 2 ? 1 : 2) mlstm_tc_chunk_out
   __syncwarp();
   tmem_fence_after();
   float ss = 0.f;
-  for (int q = half * 16; q < np; q += 32) {
-    uint32_t o[16];
-    tmem_ld16(o, tm_o + lane_base + q);
+#pragma unroll 2
+  for (int q = half * 16; q < np; q += 64) {
+    const bool two = q + 32 < np;
+    uint32_t o[2][16];
+    tmem_ld16(o[0], tm_o + lane_base + q);
+    if (two) tmem_ld16(o[1], tm_o + lane_base + q + 32);
     tmem_wait_ld();
 #pragma unroll
-    for (int e = 0; e < 16; ++e) {
-      const float x = __uint_as_float(o[e]) * inv;  // (columns past the end are zero)
-      ss = fmaf(x, x, ss);
-    }
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int e = 0; e < 16; ++e) {
+        const float v = x == 0 || two ? __uint_as_float(o[x][e]) * inv : 0.f;  // (columns past the end are zero)
+        ss = fmaf(v, v, ss);
+      }
   }
-  __syncthreads();  // everybody has read exch
+  cp_async_wait<0>();  // the gates
+  __syncthreads();     // everybody has read exch
   exch[half][r] = ss;
   __syncthreads();
   float tot = exch[0][r] + exch[1][r];
@@ -387,30 +406,35 @@ __global__ void __launch_bounds__(ML_THREADS, VB > 2 ? 1 : 2) mlstm_tc_chunk_out
     for (int x = 0; x < nvt; ++x) tot += ssq[x][r];
   }
   const float rn = inv / sqrtf(tot / (float)dv + a.eps);
-  bf16 *out = static_cast<bf16 *>(a.out) + (((size_t)b * a.n + t0 + r) * a.H + h) * dv + v0;
-  const float *norm = a.norm + (size_t)h * dv + v0;
+  // results go over their gates in shared memory, and out of there row by row
+  unsigned char *io = base + 2 * KB * MT_BLOCK + (VBUF ^ 1) * BUF;
+#pragma unroll 2
   for (int q = half * 16; q < np; q += 32) {
     uint32_t o[16];
     tmem_ld16(o, tm_o + lane_base + q);
     tmem_wait_ld();
-    if (r < cl) {
 #pragma unroll
-      for (int e = 0; e < 16; e += 8) {
-        if (q + e < vn) {
-          float z[8], f[8];
-          unpack_chunk<bf16>(*reinterpret_cast<const uint4 *>(gate + q + e), z);
+    for (int e = 0; e < 16; e += 8) {
+      uint4 *p = reinterpret_cast<uint4 *>(io + sw128_offset(MT_C, r, (q + e) / 8));
+      float z[8], f[8];
+      unpack_chunk<bf16>(*p, z);
 #pragma unroll
-          for (int x = 0; x < 8; ++x) f[x] = __uint_as_float(o[e + x]) * rn * norm[q + e + x] * sigmoid_f(z[x]);
-          uint4 v;
-          v.x = pack_bf16(f[0], f[1]);
-          v.y = pack_bf16(f[2], f[3]);
-          v.z = pack_bf16(f[4], f[5]);
-          v.w = pack_bf16(f[6], f[7]);
-          *reinterpret_cast<uint4 *>(out + q + e) = v;
-        }
-      }
+      for (int x = 0; x < 8; ++x)
+        f[x] = __uint_as_float(o[e + x]) * rn * norm_s[q + e + x] * __fdividef(1.f, 1.f + __expf(-z[x]));
+      uint4 v;
+      v.x = pack_bf16(f[0], f[1]);
+      v.y = pack_bf16(f[2], f[3]);
+      v.z = pack_bf16(f[4], f[5]);
+      v.w = pack_bf16(f[6], f[7]);
+      *p = v;
     }
-    __syncwarp();
+  }
+  __syncthreads();
+  bf16 *out = static_cast<bf16 *>(a.out) + (((size_t)b * a.n + t0) * a.H + h) * dv + v0;
+  for (int i = tid; i < cl * VB * 8; i += ML_THREADS) {
+    const int t = i / (VB * 8), ch = i - t * (VB * 8);
+    if (ch * 8 < vn)
+      *reinterpret_cast<uint4 *>(out + (size_t)t * a.H * dv + ch * 8) = *reinterpret_cast<const uint4 *>(io + sw128_offset(MT_C, t, ch));
   }
   if (dead && tid == 0) atomicAdd(&g_mlstm_timeouts, 1u);
   tmem_fence_before();
@@ -426,6 +450,12 @@ static int out_vb(int dk, int dv) {
 
 bool mlstm_tc_supported(int dtype, int dk, int dv) {
   return dtype == DJV_DTYPE_BF16 && dk % 8 == 0 && dv % 8 == 0 && dk <= 256 && ceil_div(dv, out_vb(dk, dv) * 64) <= MT_MAX_TILES;
+}
+
+int mlstm_tc_gates(const MlstmArgs &a, cudaStream_t st) {
+  djv::launch_kernel(mlstm_tc_gates_kernel, dim3(ceil_div(a.nc, MG_WARPS), a.H, a.B), dim3(MG_WARPS * WARP), 0, st, a);
+  count_launch();
+  return check_launch("mlstm_prefill");
 }
 
 int mlstm_tc_chunk_state(const MlstmArgs &a, cudaStream_t st) {

@@ -68,7 +68,10 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
   const int h = blockIdx.x, b = blockIdx.z, g = h / (a.H / a.G);
   const int t0 = (int)(gridDim.y - 1 - blockIdx.y) * WP_TILE;
   unsigned char *base = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-  const uint32_t q_sm = smem_u32(base), k_sm = q_sm + KT, v_sm = k_sm + KT;
+  // with three blocks per key, values go over their keys: two thread blocks fit a multiprocessor that way, and each loads
+  // while the other computes
+  constexpr bool OVER = KB == 3 && VB <= 2;
+  const uint32_t q_sm = smem_u32(base), k_sm = q_sm + KT, v_sm = OVER ? k_sm : k_sm + KT;
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   asm volatile("griddepcontrol.wait;" ::: "memory");
 
@@ -176,6 +179,7 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
       if (!dead) dead = !mbar_wait(&bar_o, (i - 1) & 1);
       __syncwarp();  // (TMEM accesses are whole-warp instructions)
       tmem_fence_after();
+      if (OVER) load(k_sm, j0, kr, a.dk, k_new, a.ldk, own, kb);
     }
     cp_async_wait<0>();
     fence_proxy_async_smem();
@@ -189,8 +193,9 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
       }
       mma_commit(&bar_s);
     }
-    load(v_sm, j0, vr, a.dv, v_new, a.ldv, a.dv, vb);
+    if (!OVER) load(v_sm, j0, vr, a.dv, v_new, a.ldv, a.dv, vb);
     if (!dead) dead = !mbar_wait(&bar_s, i & 1);
+    if (OVER) load(v_sm, j0, vr, a.dv, v_new, a.ldv, a.dv, vb);
     __syncwarp();
     tmem_fence_after();
     __syncwarp();
@@ -297,7 +302,7 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
         mma_ts(tm_o, tm_s + 64 + k * 8, v_desc + (uint64_t)(k * 128), idesc_o, true);
       mma_commit(&bar_o);
     }
-    if (i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, a.ldk, own, kb);  // behind the values' products
+    if (!OVER && i + 1 < tiles) load(k_sm, j0 + WP_TILE, kr, a.dk, k_new, a.ldk, own, kb);  // behind the values' products
   }
   if (!dead) dead = !mbar_wait(&bar_o, (tiles - 1) & 1);
   __syncwarp();
@@ -344,7 +349,7 @@ __global__ void __launch_bounds__(WP_THREADS, VB > 2 ? 1 : 2) window_prefill_ker
 
 template <int KB, int VB>
 static int launch_window_prefill(const WindowArgs &a, cudaStream_t st) {
-  size_t smem = 1024 + (size_t)(2 * KB + VB) * WP_TILE * 128;
+  size_t smem = 1024 + (size_t)(2 * KB + (KB == 3 && VB <= 2 ? 0 : VB)) * WP_TILE * 128;
   // as many blocks per multiprocessor as TMEM has room for: two, or one with wide values
   const size_t least = (VB > 2 ? 120 : 80) * 1024;
   if (smem < least) smem = least;

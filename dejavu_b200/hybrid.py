@@ -5,6 +5,7 @@ from __future__ import annotations
 import torch
 import torch.nn as nn
 
+from . import _lib
 from .generation import GenerationMixin, InferenceParams
 from .gpt import CausalLMOutput, _randn_big, _stable_hash
 from .mixers import Linear, _empty
@@ -19,6 +20,7 @@ class HybridDecoder(nn.Module, GenerationMixin):
 
     selects_logit_rows = True  # forward(logit_rows=...) computes logits at those tokens only
     takes_portions = True      # a prompt may arrive in portions of any size
+    load_kernels = staticmethod(_lib.load_hybrid)  # the library that has the design's kernels
 
     def __init__(self, config, device=None, dtype=torch.bfloat16):
         super().__init__()
@@ -86,6 +88,8 @@ class HybridDecoder(nn.Module, GenerationMixin):
     def allocate_cache(self, batch_size: int, max_seqlen: int, device) -> dict:
         """Per layer run: the window's rings or the recurrent state. Nothing needs clearing between requests: a sequence
         that starts at position 0 reads neither."""
+        if torch.device(device).type == "cuda":
+            self.load_kernels()
         return {r: self.layers[i].mixer.new_cache(batch_size, max_seqlen, device, self.dtype)
                 for r, i in enumerate(self.runs)}
 

@@ -14,7 +14,7 @@ from types import SimpleNamespace
 import torch
 import torch.nn as nn
 
-from . import ops
+from . import _lib, ops
 from .hybrid import HybridDecoder
 from .mixers import GatedMLP, LatentAttention, MatrixMemory, MixtureOfExperts, SplitSum, _empty
 
@@ -70,6 +70,8 @@ class TifosunLayer(nn.Module):
 
 
 class TifosunForCausalLM(HybridDecoder):
+    load_kernels = staticmethod(_lib.load_routed)
+
     def __init__(self, config: dict, device=None, dtype=torch.bfloat16):
         """`config` is the parsed config.json."""
         cfg = parse_config(config)

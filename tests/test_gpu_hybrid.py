@@ -129,7 +129,7 @@ def test_rotary(dtype, rot, dim, heads):
 
 # heads, kv heads, dk, dv, window: groups of 1 to 16, sizes that are and are not multiples of 8 / 16 / 64
 WINDOWS = [(4, 2, 64, 64, 45), (3, 3, 18, 10, 3), (8, 1, 128, 64, 150), (6, 2, 48, 96, 64), (16, 1, 32, 40, 7), (4, 4, 128, 128, 300),
-           (5, 1, 80, 256, 33), (2, 1, 256, 80, 129), (2, 2, 64, 130, 20), (12, 4, 96, 192, 64), (1, 1, 16, 16, 1)]
+           (5, 1, 80, 256, 33), (2, 1, 256, 80, 129), (2, 2, 64, 130, 20), (12, 4, 96, 192, 64), (1, 1, 16, 16, 1), (4, 2, 160, 64, 70), (2, 1, 192, 128, 140)]
 
 
 def spiky(g, n, heads, kv, dk, dv, dtype, window):
