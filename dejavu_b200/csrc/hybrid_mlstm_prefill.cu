@@ -5,8 +5,8 @@
 // Outputs: S = Q K^T (TMEM); P_ts = S_ts e^(a_s - M_t) for s <= t goes back to TMEM over S, as hi + lo; O (TMEM) = Q S_in, S_in
 // in hi + lo, scaled by e^(m_in - M_t) row by row, then += P_hi V + P_lo V. The denominator takes the fp32 sums of P and
 // q . n_in. Norm and gate run on the way out. The incoming state streams through two buffers of 64 channels; V takes the one
-// that is free first, the output gates the other. A block has 256 threads, two per row of TMEM, and up to 256 value columns; wider heads are a cluster of
-// blocks that exchange their sums of squares.
+// that is free first, the output gates the other. A block has 256 threads, two per row of TMEM, and up to 256 value
+// columns; wider heads are a cluster of blocks that exchange their sums of squares.
 #include <cooperative_groups.h>
 
 #include "../../include/dejavu_b200_routed.h"
